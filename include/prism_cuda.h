@@ -324,7 +324,8 @@ int prism_cuda_engine_bind_by_keys(prism_cuda_engine *eng, const char *key_prefi
 /* PrismEngine::load: reads a reference-format .cimage (src/quantization/cimage.rs:242-277),
  * uploads every palettized tensor and binds it. */
 int prism_cuda_engine_load_cimage(prism_cuda_engine *eng, const char *path, const char *key_prefix);
-/* Fills every weight of the model with seeded synthetic tensors on the device. */
+/* Fills every weight of the model with seeded synthetic tensors on the device (layered engines: bf16 N(0, sigma),
+ * norm weights N(1, sigma)). */
 int prism_cuda_engine_synth_weights(prism_cuda_engine *eng, uint64_t seed, float sigma);
 /* PrismEngine::generate for `batch` sequences at once: prompts is
  * [batch][n_prompt] token ids, out_tokens receives [batch][max_new].  Prefill is
@@ -355,6 +356,60 @@ double prism_cuda_engine_last_device_ms(prism_cuda_engine *eng);
 uint32_t prism_cuda_engine_position(prism_cuda_engine *eng);
 /* Kernels one step launches (counted when the step was first enqueued). */
 uint32_t prism_cuda_engine_kernels_per_step(prism_cuda_engine *eng);
+/* ---- models described layer by layer (not in the reference; dense bf16 weights) ------------------------
+ * The same engine object -- create / generate / step / decode / reset, CUDA-graph step, greedy argmax --
+ * over a list of layers instead of the Llama/Qwen2 node order: every layer names its mixer and its sizes.
+ * Residual, norms, attention scores and weights, positions and recurrent state are fp32; linears and
+ * activations are bf16 with fp32 accumulation, or everything is fp32 (dtype). */
+enum { PRISM_MIXER_LIGHTNING = 0, PRISM_MIXER_LATENT_ATTENTION = 1 };
+enum { PRISM_DTYPE_BF16 = 0, PRISM_DTYPE_F32 = 1 };
+
+typedef struct prism_layer_config {
+    uint32_t mixer;            /* PRISM_MIXER_* */
+    uint32_t heads, dim, vdim; /* per head: key size (latent: its unrotated part), value size */
+    const float *decay;        /* lightning: [heads] decay of the state per token */
+    uint32_t q_rank, kv_rank;  /* latent: sizes of the query latent and of the cached latent */
+    uint32_t rot_dim;          /* latent: rotated part of queries and of the shared key */
+    uint32_t rot_pairs;        /* latent: pairs (i, i + rot_pairs) of it that turn; the rest passes */
+    const float *rot_freq;     /* latent: [rot_pairs] angle per position */
+    float rot_mul;             /* latent: factor of cos and sin */
+    float scale;               /* latent: factor of the scores */
+    uint32_t window;           /* latent: positions i - window + 1 .. i are visible; 0: all up to i */
+    uint32_t ff;               /* dense feed-forward size; 0: none */
+} prism_layer_config;
+
+typedef struct prism_layered_config {
+    uint32_t vocab, width, num_layers;
+    float norm_eps, residual_mult, logit_scale;
+    uint32_t dtype;            /* PRISM_DTYPE_* */
+    uint32_t max_seq, max_batch;
+} prism_layered_config;
+
+/* The arrays inside the layer configs are copied.  Prompt portions go through the layers in chunks of the
+ * context's "prefill_chunk" option at the time of this call (windowed caches are sized by it). */
+int prism_cuda_engine_create_layered(prism_cuda_ctx *ctx, const prism_layered_config *cfg, const prism_layer_config *layers,
+                                     prism_cuda_engine **out);
+/* Sets one tensor by its checkpoint name ("embed", "l0.norm1", "l0.mix.q", "l0.mlp.up.b", "final.norm", "head",
+ * ...) from bf16 bit patterns, row-major; a vector is rows x 1 (or 1 x n).  PRISM_E_NOTFOUND for a name the
+ * configuration has no place for. */
+int prism_cuda_engine_set_tensor(prism_cuda_engine *eng, const char *name, const uint16_t *bf16, uint64_t rows, uint64_t cols);
+/* Every tensor of a .safetensors file (bf16) into the engine; fails when a tensor has no place, a wrong shape
+ * or another type, or when one the model needs is missing. */
+int prism_cuda_engine_load_safetensors(prism_cuda_engine *eng, const char *path);
+/* Sequences of a layered engine (at most max_batch at a time): open gives a slot whose state is empty, close
+ * gives it back.  reset() and generate() close all of them and use slots 0 .. batch-1. */
+int prism_cuda_engine_seq_open(prism_cuda_engine *eng, uint32_t *seq);
+int prism_cuda_engine_seq_close(prism_cuda_engine *eng, uint32_t seq);
+int prism_cuda_engine_seq_position(prism_cuda_engine *eng, uint32_t seq, uint32_t *pos);
+/* One step over `n` open sequences: entry i appends n_tokens[i] tokens (taken one entry after the other from
+ * `tokens`) where its sequence stands.  Entries of one token run together as a decode step, longer ones as
+ * prompt portions.  want lists, entry by entry, n_want[i] ascending places inside the entry's tokens whose
+ * fp32 logits go to `logits` ([sum n_want][vocab], host); next_tokens (optional) gets the greedy token
+ * after each entry.  A sequence may appear once per call. */
+int prism_cuda_engine_extend(prism_cuda_engine *eng, uint32_t n, const uint32_t *seqs, const uint32_t *n_tokens,
+                             const uint32_t *tokens, const uint32_t *n_want, const uint32_t *want, float *logits,
+                             uint32_t *next_tokens);
+
 /* ---- tensor parallelism (not in the reference; column/row-sharded linears
  *      with an all-reduce after each row-parallel matmul) ------------------- */
 

@@ -9,3 +9,4 @@ from .backend import (QWEN25_0P5B, QWEN25_7B, QWEN25_72B, CudaBackend, PrismEngi
                       model_config)
 from .cimage import CImageReader, CImageWriter  # noqa: F401
 from .graph import ModelGraph, UnifiedConfig, generate_plan  # noqa: F401
+from .models import LayeredConfig, load_model, read_config  # noqa: F401

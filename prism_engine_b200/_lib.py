@@ -36,6 +36,27 @@ class ModelConfig(C.Structure):
     ]
 
 
+class LayerConfig(C.Structure):
+    """Mirror of ``prism_layer_config``."""
+
+    _fields_ = [
+        ("mixer", C.c_uint32), ("heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32),
+        ("decay", C.POINTER(C.c_float)), ("q_rank", C.c_uint32), ("kv_rank", C.c_uint32), ("rot_dim", C.c_uint32),
+        ("rot_pairs", C.c_uint32), ("rot_freq", C.POINTER(C.c_float)), ("rot_mul", C.c_float), ("scale", C.c_float),
+        ("window", C.c_uint32), ("ff", C.c_uint32),
+    ]
+
+
+class LayeredModelConfig(C.Structure):
+    """Mirror of ``prism_layered_config``."""
+
+    _fields_ = [
+        ("vocab", C.c_uint32), ("width", C.c_uint32), ("num_layers", C.c_uint32), ("norm_eps", C.c_float),
+        ("residual_mult", C.c_float), ("logit_scale", C.c_float), ("dtype", C.c_uint32), ("max_seq", C.c_uint32),
+        ("max_batch", C.c_uint32),
+    ]
+
+
 class CImagePlan(C.Structure):
     """Mirror of ``prism_cimage_plan``."""
 
@@ -86,6 +107,13 @@ SIGNATURES = {
     "prism_cuda_argmax": (C.c_int, [_vp, _vp, _u32, _pu32]),
     "prism_cuda_engine_create": (C.c_int, [_vp, C.POINTER(ModelConfig), C.POINTER(_vp)]),
     "prism_cuda_engine_destroy": (None, [_vp]),
+    "prism_cuda_engine_create_layered": (C.c_int, [_vp, C.POINTER(LayeredModelConfig), C.POINTER(LayerConfig), C.POINTER(_vp)]),
+    "prism_cuda_engine_set_tensor": (C.c_int, [_vp, _cp, _vp, _u64, _u64]),
+    "prism_cuda_engine_load_safetensors": (C.c_int, [_vp, _cp]),
+    "prism_cuda_engine_seq_open": (C.c_int, [_vp, _pu32]),
+    "prism_cuda_engine_seq_close": (C.c_int, [_vp, _u32]),
+    "prism_cuda_engine_seq_position": (C.c_int, [_vp, _u32, _pu32]),
+    "prism_cuda_engine_extend": (C.c_int, [_vp, _u32, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
     "prism_cuda_engine_bind": (C.c_int, [_vp, _u32, _u32, _i32]),
     "prism_cuda_engine_bind_by_keys": (C.c_int, [_vp, _cp]),
     "prism_cuda_engine_load_cimage": (C.c_int, [_vp, _cp, _cp]),

@@ -381,14 +381,24 @@ QWEN25_7B = dict(num_layers=28, hidden_size=3584, num_heads=28, num_kv_heads=4, 
 
 
 class PrismEngine:
-    """Mirror of ``PrismEngine`` (src/lut/engine_impl.rs:503-512) with every op on the device."""
+    """Mirror of ``PrismEngine`` (src/lut/engine_impl.rs:503-512) with every op on the device.
 
-    def __init__(self, backend: CudaBackend, cfg: ModelConfig):
+    ``cfg`` is a ``ModelConfig`` (palettized Llama/Qwen2 family) or a ``LayeredConfig`` (a model described
+    layer by layer, models.py) together with ``dtype``, ``max_seq`` and ``max_batch``."""
+
+    def __init__(self, backend: CudaBackend, cfg, dtype: str = "bfloat16", max_seq: int = 4096, max_batch: int = 1):
         self.be = backend
         self.cfg = cfg
         self.L = backend.L
         h = C.c_void_p()
-        check(backend.ctx, self.L.prism_cuda_engine_create(backend.ctx, C.byref(cfg), C.byref(h)))
+        if isinstance(cfg, ModelConfig):
+            check(backend.ctx, self.L.prism_cuda_engine_create(backend.ctx, C.byref(cfg), C.byref(h)))
+            self.vocab = cfg.vocab_size
+        else:
+            mc, layers, keep = cfg.to_c(dtype, max_seq, max_batch)
+            check(backend.ctx, self.L.prism_cuda_engine_create_layered(backend.ctx, C.byref(mc), layers, C.byref(h)))
+            del keep  # the library has copied the arrays
+            self.vocab = cfg.vocab
         self.h = h
         backend._engines.add(self)
 
@@ -419,6 +429,45 @@ class PrismEngine:
     def bind_by_keys(self, prefix: str = "model") -> None:
         self._ck(self.L.prism_cuda_engine_bind_by_keys(self.h, prefix.encode()))
 
+    # -- models described layer by layer ---------------------------------------------------------------
+    def set_tensor(self, name: str, bits) -> None:
+        """One weight by its checkpoint name, as bf16 bit patterns (uint16, matrix or vector)."""
+        a = _u16(bits)
+        if a.ndim not in (1, 2):
+            raise PrismCudaError(_lib.E_ARG, f"set_tensor: {name} must be a vector or a matrix")
+        self._ck(self.L.prism_cuda_engine_set_tensor(self.h, name.encode(), _ptr(a), a.shape[0], a.shape[1] if a.ndim == 2 else 1))
+
+    def load_safetensors(self, path: str) -> None:
+        self._ck(self.L.prism_cuda_engine_load_safetensors(self.h, path.encode()))
+
+    def open_sequence(self) -> int:
+        s = C.c_uint32()
+        self._ck(self.L.prism_cuda_engine_seq_open(self.h, C.byref(s)))
+        return s.value
+
+    def close_sequence(self, seq: int) -> None:
+        self._ck(self.L.prism_cuda_engine_seq_close(self.h, seq))
+
+    def sequence_position(self, seq: int) -> int:
+        p = C.c_uint32()
+        self._ck(self.L.prism_cuda_engine_seq_position(self.h, seq, C.byref(p)))
+        return p.value
+
+    def extend(self, entries, want_next: bool = False):
+        """One step over open sequences: ``entries`` is a list of ``(sequence, tokens, wanted places)``.
+        Returns fp32 logits ``[wanted, vocab]`` in that order (with ``want_next`` also the greedy token after
+        each entry)."""
+        seqs = np.array([e[0] for e in entries], np.uint32)
+        lens = np.array([len(e[1]) for e in entries], np.uint32)
+        toks = np.concatenate([np.asarray(e[1], np.uint32).reshape(-1) for e in entries]) if entries else np.empty(0, np.uint32)
+        nw = np.array([len(e[2]) for e in entries], np.uint32)
+        want = np.concatenate([np.asarray(e[2], np.uint32).reshape(-1) for e in entries]) if entries else np.empty(0, np.uint32)
+        lg = np.empty((int(nw.sum()), self.vocab), np.float32)
+        nxt = np.empty(len(entries), np.uint32)
+        self._ck(self.L.prism_cuda_engine_extend(self.h, len(entries), _ptr(seqs), _ptr(lens), _ptr(toks), _ptr(nw), _ptr(want),
+                                                 _ptr(lg), _ptr(nxt) if want_next else None))
+        return (lg, nxt) if want_next else lg
+
     def synth_weights(self, seed: int = 0, sigma: float = 0.02) -> None:
         self._ck(self.L.prism_cuda_engine_synth_weights(self.h, seed, sigma))
 
@@ -430,7 +479,7 @@ class PrismEngine:
             p = p[None, :]
         batch, n = p.shape
         out = np.empty((batch, max_new), np.uint32)
-        lg = np.empty((batch, self.cfg.vocab_size), np.uint16) if return_logits else None
+        lg = np.empty((batch, self.vocab), np.uint16) if return_logits else None
         self._ck(self.L.prism_cuda_engine_generate(self.h, _ptr(p), batch, n, max_new, _ptr(out),
                                                    _ptr(lg) if lg is not None else None))
         if single:
@@ -444,7 +493,7 @@ class PrismEngine:
     def step(self, tokens, want_logits: bool = False):
         t = np.ascontiguousarray(np.atleast_1d(tokens), dtype=np.uint32)
         nxt = np.empty(t.size, np.uint32)
-        lg = np.empty((t.size, self.cfg.vocab_size), np.uint16) if want_logits else None
+        lg = np.empty((t.size, self.vocab), np.uint16) if want_logits else None
         self._ck(self.L.prism_cuda_engine_step(self.h, _ptr(t), _ptr(nxt), _ptr(lg) if lg is not None else None))
         return (nxt, lg) if want_logits else nxt
 

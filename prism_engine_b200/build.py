@@ -17,7 +17,7 @@ def _stale() -> bool:
     if not os.path.exists(LIB):
         return True
     t = os.path.getmtime(LIB)
-    srcs = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cuh", ".h", "Makefile"))]
+    srcs = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cuh", ".hpp", ".h", "Makefile"))]
     srcs.append(os.path.join(HERE, "..", "include", "prism_cuda.h"))
     return any(os.path.getmtime(s) > t for s in srcs)
 

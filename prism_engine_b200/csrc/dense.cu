@@ -1,0 +1,415 @@
+// Dense bf16 linears for few rows, the same linears in 32-bit, and the element-wise kernels around
+// them: weight packing, RMS norm with a weight, embedding gather, fp32 argmax.
+#include <algorithm>
+
+#include "dense.cuh"
+
+namespace prism {
+
+// ---- weights -------------------------------------------------------------------------------------
+
+int dense_alloc(prism_cuda_ctx *ctx, DenseLinear &l, uint32_t k_pad, uint32_t n_tiles) {
+    l.k_pad = k_pad;
+    l.n_tiles = n_tiles;
+    PRISM_CUDA_TRY(ctx, cudaMalloc((void **)&l.w, l.bytes()));
+    PRISM_CUDA_TRY(ctx, cudaMemsetAsync(l.w, 0, l.bytes(), ctx->stream));
+    return PRISM_OK;
+}
+
+__global__ void dense_pack_kernel(const bf16 *__restrict__ src, uint32_t rows, uint32_t cols, bf16 *__restrict__ w, uint32_t k_pad,
+                                  uint32_t row0, uint32_t k0) {
+    const size_t n = (size_t)rows * cols;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const uint32_t r = row0 + (uint32_t)(i / cols), k = k0 + (uint32_t)(i % cols);
+        w[(((size_t)(r >> 7) * (k_pad / 8) + (k >> 3)) * 128 + (r & 127)) * 8 + (k & 7)] = src[i];
+    }
+}
+int launch_dense_pack(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 *src, uint32_t rows, uint32_t cols, uint32_t row0,
+                      uint32_t k0) {
+    const size_t n = (size_t)rows * cols;
+    dense_pack_kernel<<<(unsigned)std::min<size_t>((n + 255) / 256, 65535), 256, 0, ctx->stream>>>(src, rows, cols, l.w, l.k_pad, row0, k0);
+    return after_launch(ctx, "dense_pack_kernel");
+}
+
+__global__ void bf16_to_f32_kernel(const bf16 *__restrict__ src, float *__restrict__ dst, size_t n) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) dst[i] = __bfloat162float(src[i]);
+}
+int launch_bf16_to_f32(prism_cuda_ctx *ctx, const bf16 *src, float *dst, size_t n) {
+    bf16_to_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(src, dst, n);
+    return after_launch(ctx, "bf16_to_f32_kernel");
+}
+
+__global__ void bf16_pitch_copy_kernel(const bf16 *__restrict__ src, bf16 *__restrict__ dst, uint32_t rows, uint32_t cols, uint32_t pitch) {
+    const size_t n = (size_t)rows * pitch;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const uint32_t r = (uint32_t)(i / pitch), c = (uint32_t)(i % pitch);
+        dst[i] = c < cols ? src[(size_t)r * cols + c] : __float2bfloat16_rn(0.0f);
+    }
+}
+int launch_bf16_pitch_copy(prism_cuda_ctx *ctx, const bf16 *src, bf16 *dst, uint32_t rows, uint32_t cols, uint32_t dst_pitch) {
+    const size_t n = (size_t)rows * dst_pitch;
+    bf16_pitch_copy_kernel<<<(unsigned)std::min<size_t>((n + 255) / 256, 65535), 256, 0, ctx->stream>>>(src, dst, rows, cols, dst_pitch);
+    return after_launch(ctx, "bf16_pitch_copy_kernel");
+}
+
+// Seeded values N(mean, sigma) of a benchmark model (Box-Muller over a counter hash).
+__device__ __forceinline__ uint32_t mix32(uint64_t z) {
+    z += 0x9E3779B97F4A7C15ull;
+    z = (z ^ (z >> 30)) * 0xBF58476D1CE4E5B9ull;
+    z = (z ^ (z >> 27)) * 0x94D049BB133111EBull;
+    return (uint32_t)(z ^ (z >> 31));
+}
+__global__ void dense_synth_kernel(bf16 *__restrict__ dst, size_t n, uint64_t seed, float mean, float sigma) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const float u1 = ((float)mix32(seed * 0x100000001B3ull + 2 * i) + 1.0f) * 2.3283064e-10f;
+        const float u2 = (float)mix32(seed * 0x100000001B3ull + 2 * i + 1) * 2.3283064e-10f;
+        dst[i] = __float2bfloat16_rn(mean + sigma * sqrtf(-2.0f * logf(fminf(u1, 1.0f))) * cospif(2.0f * u2));
+    }
+}
+int launch_dense_synth(prism_cuda_ctx *ctx, bf16 *dst, size_t n, uint64_t seed, float mean, float sigma) {
+    dense_synth_kernel<<<(unsigned)std::min<size_t>((n + 255) / 256, 65535), 256, 0, ctx->stream>>>(dst, n, seed, mean, sigma);
+    return after_launch(ctx, "dense_synth_kernel");
+}
+
+DenseEpi dense_epi(const DenseLinear &l, const DenseOut *outs) {
+    DenseEpi e{};
+    e.n = l.n_segs;
+    for (uint32_t i = 0; i < l.n_segs; i++)
+        e.s[i] = DenseEpiSeg{l.seg[i].row0, l.seg[i].rows, l.seg[i].act, outs[i].store, outs[i].pitch, l.seg[i].mul, l.seg[i].bias, outs[i].p};
+    return e;
+}
+
+// ---- few rows: mma.sync straight from the weight units ----------------------------------------------
+// A CTA takes 32 weight rows at a time; its eight warps share the k range in steps of 32.  In a step lane
+// (g, t) = (lane / 4, lane % 4) loads the units (row g + 8 i, k/8 = 4 step + t): eight consecutive k of four
+// rows, and the same eight k of token g of the input.  The order of k inside a dot product is free as long
+// as both operands agree, so these registers ARE the fragments of two m16n8k16 products per 16 rows: no
+// conversion, no shuffles, and any batch of 1..8 costs the same.  The sums of the warps meet in shared
+// memory in a fixed order.
+struct GemvArgs {
+    const uint4 *w;
+    uint32_t k8, n_groups, rows;
+    const void *x;
+    uint32_t pitch, f32;
+    const float *norm_w;
+    const bf16 *gate;
+    uint32_t gate_pitch, n_norm, norm_pad;  // norm_pad: n_norm rounded up to 64
+    float eps;
+    DenseEpi epi;
+};
+constexpr int GV_THREADS = 256, GV_WARPS = 8, GV_U = 4;
+
+// RMS norm (times weight, times gate) of the first n_norm entries of every row into shared memory as bf16.
+__device__ __forceinline__ void gemv_stage_norm(const GemvArgs &a, bf16 *xs, float *sh) {
+    const uint32_t R = a.rows;
+    const uint32_t tpr = R == 1 ? 256 : R == 2 ? 128 : R <= 4 ? 64 : 32;  // threads per row
+    const uint32_t r = threadIdx.x / tpr, i0 = threadIdx.x % tpr;
+    const bool on = r < R;
+    const float *xf = reinterpret_cast<const float *>(a.x) + (size_t)r * a.pitch;
+    const bf16 *xh = reinterpret_cast<const bf16 *>(a.x) + (size_t)r * a.pitch;
+    float ss = 0.0f;
+    if (on)
+        for (uint32_t i = i0; i < a.n_norm; i += tpr) {
+            const float v = a.f32 ? xf[i] : __bfloat162float(xh[i]);
+            ss += v * v;
+        }
+    ss = warp_sum_f(ss);
+    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    if (on) {
+        const uint32_t w0 = r * (tpr / 32);
+        float s = 0.0f;
+        for (uint32_t w = 0; w < tpr / 32; w++) s += sh[w0 + w];
+        const float inv = 1.0f / sqrtf(s / (float)a.n_norm + a.eps);
+        for (uint32_t i = i0; i < a.norm_pad; i += tpr) {
+            float v = 0.0f;
+            if (i < a.n_norm) {
+                v = (a.f32 ? xf[i] : __bfloat162float(xh[i])) * inv * __ldg(a.norm_w + i);
+                if (a.gate) v *= __bfloat162float(a.gate[(size_t)r * a.gate_pitch + i]);
+            }
+            xs[(size_t)r * a.norm_pad + i] = __float2bfloat16_rn(v);
+        }
+    }
+    __syncthreads();
+}
+
+template <bool NORM>
+__global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArgs a) {
+    extern __shared__ __align__(16) uint8_t dsm[];
+    __shared__ float red[GV_WARPS][8][33];
+    __shared__ float sh[32];
+    bf16 *xs = reinterpret_cast<bf16 *>(dsm);
+    pdl_launch_dependents();
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g8 = lane >> 2, t4 = lane & 3;
+    const uint32_t steps = a.k8 / 4, norm8 = NORM ? a.norm_pad / 8 : 0;
+    const bool tok_on = g8 < a.rows;
+    const uint4 *xg = reinterpret_cast<const uint4 *>(reinterpret_cast<const bf16 *>(a.x) + (size_t)g8 * a.pitch);
+    const uint4 *xl = reinterpret_cast<const uint4 *>(xs + (size_t)g8 * a.norm_pad);
+    uint4 w[GV_U][4];
+    auto locate = [&](uint32_t grp, uint32_t &sg, uint32_t &rb) -> const uint4 * {  // segment, block of 32 rows inside it, first unit
+        sg = 0;
+        rb = grp;
+        while (sg + 1 < a.epi.n && rb >= (a.epi.s[sg].rows + 31) / 32) {
+            rb -= (a.epi.s[sg].rows + 31) / 32;
+            sg++;
+        }
+        const uint32_t row = a.epi.s[sg].row0 + rb * 32;
+        return a.w + (size_t)(row >> 7) * a.k8 * 128 + (row & 127) + g8;
+    };
+    auto load = [&](const uint4 *wt, uint32_t s0) {
+#pragma unroll
+        for (int u = 0; u < GV_U; u++) {
+            const uint32_t s = s0 + u * GV_WARPS;
+            if (s < steps) {
+                const uint4 *p = wt + (size_t)(4 * s + t4) * 128;
+#pragma unroll
+                for (int i = 0; i < 4; i++) w[u][i] = __ldg(p + 8 * i);
+            }
+        }
+    };
+    uint32_t sg, rb;
+    const uint4 *wt = locate(blockIdx.x, sg, rb);
+    load(wt, warp);  // weights do not depend on the previous kernel; the input does
+    pdl_wait();
+    if (NORM) gemv_stage_norm(a, xs, sh);
+    bool loaded = true;
+    for (uint32_t grp = blockIdx.x; grp < a.n_groups; grp += gridDim.x) {
+        if (!loaded) wt = locate(grp, sg, rb);
+        float acc[2][4] = {};
+        for (uint32_t s0 = warp; s0 < steps; s0 += GV_WARPS * GV_U) {
+            if (!loaded) load(wt, s0);
+            loaded = false;
+#pragma unroll
+            for (int u = 0; u < GV_U; u++) {
+                const uint32_t s = s0 + u * GV_WARPS;
+                if (s < steps) {
+                    const uint32_t k8 = 4 * s + t4;
+                    uint4 x = make_uint4(0, 0, 0, 0);
+                    if (tok_on) x = NORM && k8 < norm8 ? xl[k8] : xg[k8];
+#pragma unroll
+                    for (int m = 0; m < 2; m++) {
+                        const uint4 lo = w[u][2 * m], hi = w[u][2 * m + 1];
+                        const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+                        mma_bf16(acc[m], a0, x.x, x.y);
+                        mma_bf16(acc[m], a1, x.z, x.w);
+                    }
+                }
+            }
+        }
+        loaded = false;
+#pragma unroll
+        for (int m = 0; m < 2; m++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) red[warp][2 * t4 + (i & 1)][16 * m + g8 + 8 * (i >> 1)] = acc[m][i];
+        __syncthreads();
+        const uint32_t t = threadIdx.x >> 5, rl = rb * 32 + lane;
+        if (t < a.rows && rl < a.epi.s[sg].rows) {
+            float v = 0.0f;
+#pragma unroll
+            for (int w = 0; w < GV_WARPS; w++) v += red[w][t][lane];
+            dense_store<bf16>(a.epi.s[sg], rl, t, v);
+        }
+        __syncthreads();
+    }
+}
+
+static size_t gemv_smem(const DenseIn &in, uint32_t rows) {
+    return in.norm_w ? (size_t)rows * round_up_u32(in.n_norm, 64) * 2 : 0;
+}
+constexpr size_t GV_SMEM_MAX = 160 * 1024;
+
+bool dense_gemv_ok(const DenseLinear &l, const DenseIn &in, uint32_t rows) {
+    (void)l;
+    return rows <= DENSE_GEMV_ROWS && gemv_smem(in, rows) <= GV_SMEM_MAX && (in.norm_w || !in.f32) && (in.f32 || in.pitch % 8 == 0);
+}
+
+int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows) {
+    GemvArgs a{};
+    a.w = reinterpret_cast<const uint4 *>(l.w);
+    a.k8 = l.k_pad / 8;
+    a.rows = rows;
+    a.x = in.x; a.pitch = in.pitch; a.f32 = in.f32;
+    a.norm_w = in.norm_w; a.n_norm = in.n_norm; a.norm_pad = round_up_u32(in.n_norm, 64); a.eps = in.eps;
+    a.gate = reinterpret_cast<const bf16 *>(in.gate); a.gate_pitch = in.gate_pitch;
+    a.epi = dense_epi(l, outs);
+    for (uint32_t s = 0; s < l.n_segs; s++) a.n_groups += (l.seg[s].rows + 31) / 32;
+    const size_t smem = gemv_smem(in, rows);
+    const uint32_t grid = std::min(a.n_groups, 2u * (uint32_t)ctx->sm_count);
+    if (in.norm_w) {
+        static bool configured[PRISM_MAX_DEVICES] = {false};
+        if (!configured[ctx->device]) {
+            PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemv_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GV_SMEM_MAX));
+            configured[ctx->device] = true;
+        }
+        launch_pdl(ctx, "dense_gemv_kernel", dense_gemv_kernel<true>, grid, GV_THREADS, smem, a);
+    } else {
+        launch_pdl(ctx, "dense_gemv_kernel", dense_gemv_kernel<false>, grid, GV_THREADS, 0, a);
+    }
+    return after_launch(ctx, "dense_gemv_kernel");
+}
+
+// ---- 32-bit ------------------------------------------------------------------------------------------
+// 64 weight rows x 64 input rows per CTA, 4 x 4 per thread, plain fp32 multiply-adds.
+struct F32Args {
+    const bf16 *w;
+    uint32_t k_pad, rows;
+    const float *x;
+    uint32_t pitch;
+    DenseEpi epi;
+};
+constexpr int F32_BK = 16;
+__global__ void __launch_bounds__(256) dense_f32_kernel(const F32Args a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float ws[F32_BK][68], xs[F32_BK][68];
+    const uint32_t tid = threadIdx.x, row0 = blockIdx.x * 64, t0 = blockIdx.y * 64;
+    uint32_t sg = 0;
+    while (sg + 1 < a.epi.n && row0 >= a.epi.s[sg + 1].row0) sg++;
+    if (row0 >= a.epi.s[sg].row0 + a.epi.s[sg].rows) return;  // padding
+    const uint32_t tx = tid & 15, ty = tid >> 4;              // rows tx*4.., tokens ty*4..
+    float acc[4][4] = {};
+    for (uint32_t k0 = 0; k0 < a.k_pad; k0 += F32_BK) {
+        for (uint32_t i = tid; i < 64 * F32_BK; i += 256) {
+            const uint32_t r = i / F32_BK, k = i % F32_BK;
+            const uint32_t row = row0 + r, kk = k0 + k;
+            ws[k][r] = __bfloat162float(a.w[(((size_t)(row >> 7) * (a.k_pad / 8) + (kk >> 3)) * 128 + (row & 127)) * 8 + (kk & 7)]);
+            xs[k][r] = t0 + r < a.rows && kk < a.pitch ? a.x[(size_t)(t0 + r) * a.pitch + kk] : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < F32_BK; k++) {
+            float w[4], x[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) { w[i] = ws[k][tx * 4 + i]; x[i] = xs[k][ty * 4 + i]; }
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(w[i], x[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    for (int j = 0; j < 4; j++)
+        for (int i = 0; i < 4; i++) {
+            const uint32_t rl = row0 + tx * 4 + i - a.epi.s[sg].row0, t = t0 + ty * 4 + j;
+            if (rl < a.epi.s[sg].rows && t < a.rows) dense_store<float>(a.epi.s[sg], rl, t, acc[i][j]);
+        }
+}
+int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const float *x, uint32_t pitch, const DenseOut *outs, uint32_t rows) {
+    F32Args a{l.w, l.k_pad, rows, x, pitch, dense_epi(l, outs)};
+    launch_pdl(ctx, "dense_f32_kernel", dense_f32_kernel, dim3(l.n_tiles * 2, (rows + 63) / 64), 256, 0, a);
+    return after_launch(ctx, "dense_f32_kernel");
+}
+
+// ---- element-wise ------------------------------------------------------------------------------------
+template <typename TX, typename TA>
+__global__ void __launch_bounds__(256) dense_norm_kernel(const TX *__restrict__ x, uint32_t pitch, const float *__restrict__ w, const TA *__restrict__ gate,
+                                                         uint32_t gate_pitch, uint32_t n, float eps, TA *y, uint32_t y_pitch) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float sh[32];
+    const uint32_t r = blockIdx.x;
+    const TX *xr = x + (size_t)r * pitch;
+    float ss = 0.0f;
+    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = ld_act(xr + i);
+        ss += v * v;
+    }
+    ss = block_sum_f(ss, sh);
+    const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+        float v = ld_act(xr + i) * inv * __ldg(w + i);
+        if (gate) v *= ld_act(gate + (size_t)r * gate_pitch + i);
+        st_act(y + (size_t)r * y_pitch + i, v);
+    }
+}
+int launch_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t y_pitch, uint32_t rows, bool act32) {
+    if (act32)
+        launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<float, float>, rows, 256, 0, (const float *)in.x, in.pitch, in.norm_w,
+                   (const float *)in.gate, in.gate_pitch, in.n_norm, in.eps, (float *)y, y_pitch);
+    else if (in.f32)
+        launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<float, bf16>, rows, 256, 0, (const float *)in.x, in.pitch, in.norm_w,
+                   (const bf16 *)in.gate, in.gate_pitch, in.n_norm, in.eps, (bf16 *)y, y_pitch);
+    else
+        launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<bf16, bf16>, rows, 256, 0, (const bf16 *)in.x, in.pitch, in.norm_w,
+                   (const bf16 *)in.gate, in.gate_pitch, in.n_norm, in.eps, (bf16 *)y, y_pitch);
+    return after_launch(ctx, "dense_norm_kernel");
+}
+
+__global__ void dense_embed_kernel(const bf16 *__restrict__ table, uint32_t width, uint32_t vocab, const uint32_t *__restrict__ tokens,
+                                   float *__restrict__ x) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t tok = min(tokens[blockIdx.x], vocab - 1);  // the host rejects larger ids before the launch
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x)
+        x[(size_t)blockIdx.x * width + i] = __bfloat162float(table[(size_t)tok * width + i]);
+}
+int launch_dense_embed(prism_cuda_ctx *ctx, const bf16 *table, uint32_t width, uint32_t vocab, const uint32_t *tokens, uint32_t rows, float *x) {
+    launch_pdl(ctx, "dense_embed_kernel", dense_embed_kernel, rows, 256, 0, table, width, vocab, tokens, x);
+    return after_launch(ctx, "dense_embed_kernel");
+}
+
+__global__ void gather_rows_f32_kernel(const float *__restrict__ x, const uint32_t *__restrict__ idx, uint32_t width, float *__restrict__ y) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const float *s = x + (size_t)idx[blockIdx.x] * width;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) y[(size_t)blockIdx.x * width + i] = s[i];
+}
+int launch_gather_rows_f32(prism_cuda_ctx *ctx, const float *x, const uint32_t *idx, uint32_t n, uint32_t width, float *y) {
+    launch_pdl(ctx, "gather_rows_f32_kernel", gather_rows_f32_kernel, n, 256, 0, x, idx, width, y);
+    return after_launch(ctx, "gather_rows_f32_kernel");
+}
+
+// First index of the strictly greatest value; NaN never wins (the rule of the fp16 argmax).
+__global__ void __launch_bounds__(1024) argmax_f32_kernel(const float *__restrict__ logits, uint32_t n, uint32_t stride, uint32_t *__restrict__ out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float sv[32];
+    __shared__ uint32_t si[32];
+    const float *lg = logits + (size_t)blockIdx.x * stride;
+    float bv = -INFINITY;
+    uint32_t bi = 0xFFFFFFFFu;
+    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+        const float f = lg[i];
+        if (f > bv) {
+            bv = f;
+            bi = i;
+        }
+    }
+    auto take = [&](float ov, uint32_t oi) {
+        if (ov > bv || (ov == bv && oi < bi)) {
+            bv = ov;
+            bi = oi;
+        }
+    };
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, o);
+        const uint32_t oi = __shfl_xor_sync(0xFFFFFFFFu, bi, o);
+        take(ov, oi);
+    }
+    if ((threadIdx.x & 31) == 0) {
+        sv[threadIdx.x >> 5] = bv;
+        si[threadIdx.x >> 5] = bi;
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        for (uint32_t w = 1; w < (blockDim.x >> 5); w++) take(sv[w], si[w]);
+        out[blockIdx.x] = bi == 0xFFFFFFFFu ? 0u : bi;
+    }
+}
+int launch_argmax_f32(prism_cuda_ctx *ctx, const float *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev) {
+    launch_pdl(ctx, "argmax_f32_kernel", argmax_f32_kernel, batch, 1024, 0, logits, n, stride, out_dev);
+    return after_launch(ctx, "argmax_f32_kernel");
+}
+
+__global__ void f32_to_f16_kernel(const float *__restrict__ x, uint32_t n, uint32_t stride, uint16_t *__restrict__ y, uint32_t y_stride) {
+    const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) y[(size_t)blockIdx.y * y_stride + i] = __half_as_ushort(__float2half_rn(x[(size_t)blockIdx.y * stride + i]));
+}
+int launch_f32_to_f16(prism_cuda_ctx *ctx, const float *x, uint32_t rows, uint32_t n, uint32_t stride, uint16_t *y, uint32_t y_stride) {
+    f32_to_f16_kernel<<<dim3((n + 255) / 256, rows), 256, 0, ctx->stream>>>(x, n, stride, y, y_stride);
+    return after_launch(ctx, "f32_to_f16_kernel");
+}
+
+}  // namespace prism

@@ -1,0 +1,242 @@
+// Dense bf16 linears and the element-wise pieces of the layer-list models: weight layout, epilogue
+// (shared by the tensor-core GEMM, the small-batch kernel and the 32-bit kernel) and launchers.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace prism {
+
+using bf16 = __nv_bfloat16;
+
+// ---------------------------------------------------------------------------
+// Device layout of a dense weight: bf16, rows padded to 128 and k to 64 with zeros,
+//   w : [row tile of 128][k/8][128 rows][8 k]
+// i.e. 16-byte units of eight consecutive k of one row.  64 k of a row tile are one contiguous 16 KB
+// run that already has the K-major core-matrix order of a tcgen05 shared-memory operand (one bulk copy
+// per pipeline stage), and eight rows of one k/8 are one contiguous 128-byte line for the small-batch
+// kernel, whose lanes hold mma fragments straight from these units.
+//
+// Several linears of the same input are stacked along the rows (each "segment" starts on a row tile and
+// has its own epilogue); two linears that are added together can be stacked along k instead.
+// ---------------------------------------------------------------------------
+enum DenseAct : uint32_t { ACT_NONE = 0, ACT_SILU = 1, ACT_SIGMOID = 2, ACT_GELU_TANH = 3 };
+enum DenseStore : uint32_t { ST_ACT = 0, ST_F32 = 1, ST_RESID = 2 };  // activation type, fp32, fp32 +=
+constexpr uint32_t DENSE_MAX_SEGS = 6;
+
+struct DenseSeg {
+    uint32_t row0 = 0, rows = 0;  // first row in the stacked weight (multiple of 128), valid rows
+    uint32_t act = ACT_NONE;
+    float mul = 1.0f;             // y = act(W x + bias) * mul
+    const float *bias = nullptr;  // fp32 [rows] or null
+};
+struct DenseLinear {
+    bf16 *w = nullptr;
+    uint32_t k_pad = 0, n_tiles = 0, n_segs = 0;
+    DenseSeg seg[DENSE_MAX_SEGS];
+    size_t bytes() const { return (size_t)n_tiles * 128 * k_pad * 2; }
+    uint64_t valid_rows() const {
+        uint64_t r = 0;
+        for (uint32_t s = 0; s < n_segs; s++) r += seg[s].rows;
+        return r;
+    }
+};
+// Where a segment's output goes: rows `pitch` elements apart.
+struct DenseOut {
+    void *p = nullptr;
+    uint32_t pitch = 0;
+    uint32_t store = ST_ACT;
+};
+
+// Input rows of a linear.  With norm_w the first n_norm entries of a row are RMS-normalised together (times
+// norm_w, and times gate when given); the rest of the row is taken as it is.
+struct DenseIn {
+    const void *x = nullptr;      // activation type, or fp32 when f32 is set
+    uint32_t pitch = 0;           // elements between rows
+    uint32_t f32 = 0;
+    const float *norm_w = nullptr;
+    uint32_t n_norm = 0;
+    float eps = 0.0f;
+    const void *gate = nullptr;   // activation type
+    uint32_t gate_pitch = 0;
+};
+
+struct DenseEpiSeg {
+    uint32_t row0, rows, act, store, pitch;
+    float mul;
+    const float *bias;
+    void *p;
+};
+struct DenseEpi {
+    uint32_t n;
+    DenseEpiSeg s[DENSE_MAX_SEGS];
+};
+
+#ifdef __CUDACC__
+__device__ __forceinline__ float ld_act(const bf16 *p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float ld_act(const float *p) { return *p; }
+__device__ __forceinline__ void st_act(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void st_act(float *p, float v) { *p = v; }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float dense_act(uint32_t act, float z) {
+    switch (act) {
+    case ACT_SILU: return z * sigmoid_f(z);
+    case ACT_SIGMOID: return sigmoid_f(z);
+    case ACT_GELU_TANH: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    default: return z;
+    }
+}
+// Stores output `row` (inside the segment) of token t.
+template <typename TA>
+__device__ __forceinline__ void dense_store(const DenseEpiSeg &s, uint32_t row, uint32_t t, float acc) {
+    const float v = dense_act(s.act, acc + (s.bias ? __ldg(s.bias + row) : 0.0f)) * s.mul;
+    const size_t at = (size_t)t * s.pitch + row;
+    if (s.store == ST_ACT) st_act(reinterpret_cast<TA *>(s.p) + at, v);
+    else if (s.store == ST_F32) reinterpret_cast<float *>(s.p)[at] = v;
+    else reinterpret_cast<float *>(s.p)[at] += v;
+}
+__device__ __forceinline__ float warp_sum_f(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+    return v;
+}
+__device__ __forceinline__ float warp_max_f(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xFFFFFFFFu, v, o));
+    return v;
+}
+// Block-wide sum of a value per thread; sh holds 32 floats; every thread gets the result, summed in a fixed order.
+__device__ __forceinline__ float block_sum_f(float v, float *sh) {
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    v = warp_sum_f(v);
+    __syncthreads();
+    if (lane == 0) sh[warp] = v;
+    __syncthreads();
+    float r = 0.0f;
+    for (uint32_t i = 0; i < nw; i++) r += sh[i];
+    return r;
+}
+// D += A * B, m16n8k16, bf16 operands, fp32 accumulate.
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x2(uint32_t (&r)[2], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x2_t(uint32_t (&r)[2], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+// Two floats as a bf16 pair (first in the low half), and what that rounding left over as another pair:
+// hi + lo carries 16 bits of each value, so a product with a bf16 operand keeps fp32-like accuracy.
+__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
+    const __nv_bfloat162 p = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t *>(&p);
+}
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t &hi, uint32_t &lo) {
+    const float ah = __bfloat162float(__float2bfloat16_rn(a)), bh = __bfloat162float(__float2bfloat16_rn(b));
+    hi = pack_bf16(ah, bh);
+    lo = pack_bf16(a - ah, b - bh);
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
+#endif
+
+// The rows of a step: (state slot, position) of each row.  Device arrays in a decode step (a captured graph
+// reads them at every replay); slot == nullptr: consecutive tokens of one slot from position pos0.
+struct RowMap {
+    const int32_t *slot = nullptr, *pos = nullptr;
+    int32_t slot0 = 0, pos0 = 0;
+#ifdef __CUDACC__
+    __device__ __forceinline__ int32_t slot_of(uint32_t r) const { return slot ? slot[r] : slot0; }
+    __device__ __forceinline__ int32_t pos_of(uint32_t r) const { return slot ? pos[r] : pos0 + (int32_t)r; }
+#endif
+};
+
+// dense.cu
+int dense_alloc(prism_cuda_ctx *ctx, DenseLinear &l, uint32_t k_pad, uint32_t n_tiles);
+// rows x cols bf16 (row-major, device) into rows row0.., columns k0.. of the stacked layout
+int launch_dense_pack(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 *src, uint32_t rows, uint32_t cols, uint32_t row0,
+                      uint32_t k0);
+int launch_bf16_to_f32(prism_cuda_ctx *ctx, const bf16 *src, float *dst, size_t n);
+// dst rows `dst_pitch` apart, columns cols..dst_pitch-1 zero
+int launch_bf16_pitch_copy(prism_cuda_ctx *ctx, const bf16 *src, bf16 *dst, uint32_t rows, uint32_t cols, uint32_t dst_pitch);
+int launch_dense_synth(prism_cuda_ctx *ctx, bf16 *dst, size_t n, uint64_t seed, float mean, float sigma);
+DenseEpi dense_epi(const DenseLinear &l, const DenseOut *outs);
+// Small batch (bf16, at most DENSE_GEMV_ROWS rows): mma.sync straight from the weight units, the input's norm folded in.
+constexpr uint32_t DENSE_GEMV_ROWS = 8;
+bool dense_gemv_ok(const DenseLinear &l, const DenseIn &in, uint32_t rows);
+int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows);
+// 32-bit activations and fp32 products (the weights are exact in fp32): any number of rows, plain input
+int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const float *x, uint32_t pitch, const DenseOut *outs, uint32_t rows);
+// dense_gemm_tc5.cu: tcgen05/TMEM GEMM, bf16 activations, plain input, pitch a multiple of 8
+int launch_dense_gemm_tc5(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 *x, uint32_t pitch, const DenseOut *outs, uint32_t rows);
+// y[r][0..n) = rms(x[r][0..n)) * w (* gate); y may be x.  f32 says whether x is fp32; act32 whether the activation type is fp32.
+int launch_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t y_pitch, uint32_t rows, bool act32);
+int launch_dense_embed(prism_cuda_ctx *ctx, const bf16 *table, uint32_t width, uint32_t vocab, const uint32_t *tokens, uint32_t rows, float *x);
+int launch_gather_rows_f32(prism_cuda_ctx *ctx, const float *x, const uint32_t *idx, uint32_t n, uint32_t width, float *y);
+int launch_argmax_f32(prism_cuda_ctx *ctx, const float *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev);
+int launch_f32_to_f16(prism_cuda_ctx *ctx, const float *x, uint32_t rows, uint32_t n, uint32_t stride, uint16_t *y, uint32_t y_stride);
+
+// lightning.cu
+struct LightningArgs {
+    const void *q, *k, *v;        // activation type, rows `pitch` apart, head-major
+    uint32_t pitch;
+    void *o;                      // [rows] o_pitch apart, heads * vdim
+    uint32_t o_pitch;
+    float *state;                 // [slot][heads][dim][vdim]
+    const float *decay;           // [heads]
+    uint32_t heads, dim, vdim, rows;
+};
+// One token per row, every row another sequence (decode).
+int launch_lightning_step(prism_cuda_ctx *ctx, const LightningArgs &a, const RowMap &rows, bool act32);
+// The rows are consecutive tokens of one sequence (rows.slot0).
+int launch_lightning_seq(prism_cuda_ctx *ctx, const LightningArgs &a, const RowMap &rows, bool act32);
+
+// latent_attn.cu
+struct LatentCache {
+    void *rows = nullptr;         // activation type: [slot][ring][pitch], a row = kv_rank latent | rot_dim rotated key | zeros
+    uint32_t ring = 0, pitch = 0; // position p lives in row p % ring
+};
+struct LatentArgs {
+    uint32_t heads, dim, rot_dim, rot_pairs, vdim, kv_rank, window;  // window 0: every earlier position
+    float scale, eps, rot_mul;
+    const float *rot_freq;        // [rot_pairs] angle per position
+    const float *dkv_norm;        // [kv_rank]
+    const bf16 *uk, *uv;          // row-major [heads*dim][uk_pitch] / [heads*vdim][uk_pitch]
+    uint32_t uk_pitch;
+    LatentCache cache;
+};
+// Normalises and rotates the rows of W_dkv h and appends them to the cache.
+int launch_latent_append(prism_cuda_ctx *ctx, const LatentArgs &a, const void *dkv, uint32_t pitch, const RowMap &rows, uint32_t n_rows, bool act32);
+// Rows against the cached latents themselves (W_uk folded into the query, W_uv applied to the weighted latent):
+// decode, short portions, and everything in 32-bit.  n_keys bounds the keys a row can see.
+struct LatentRowsScratch { float *qa; float *part; float *ml; size_t rows_cap; uint32_t splits; };
+size_t latent_rows_scratch_floats(const LatentArgs &a, uint32_t splits, size_t *qa, size_t *part, size_t *ml);
+uint32_t latent_rows_splits(const LatentArgs &a, uint32_t max_seq);
+int launch_latent_rows(prism_cuda_ctx *ctx, const LatentArgs &a, const LatentRowsScratch &s, const void *q, uint32_t q_pitch, const void *gate,
+                       uint32_t gate_pitch, void *out, uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32);
+// Prompt portion of one sequence (bf16): keys and values expanded for positions [lo, pos0 + n_rows).
+bool latent_expand_ok(const LatentArgs &a);
+int launch_latent_gather(prism_cuda_ctx *ctx, const LatentArgs &a, int32_t slot, uint32_t lo, uint32_t n, bf16 *lat, uint32_t lat_pitch, bf16 *krot);
+int launch_latent_prefill(prism_cuda_ctx *ctx, const LatentArgs &a, const bf16 *q, uint32_t q_pitch, const bf16 *kx, uint32_t kx_pitch,
+                          const bf16 *vx, uint32_t vx_pitch, const bf16 *krot, uint32_t lo, const bf16 *gate, uint32_t gate_pitch, bf16 *out,
+                          uint32_t out_pitch, uint32_t pos0, uint32_t n_rows);
+
+}  // namespace prism

@@ -1,0 +1,231 @@
+// Dense bf16 GEMM on tcgen05 / TMEM with the segment epilogues of dense.cuh:
+//   y[t][n] = epilogue( sum_k x[t][k] * W[n][k] ),  fp32 accumulate.
+//
+// A persistent CTA computes tiles of 128 weight rows x NT rows of x.  One warp loads: the weights of a
+// 64-k stage are one contiguous 16 KB run (dense.cuh), fetched by a 1-D bulk copy straight into the
+// unswizzled core-matrix order of the A operand; the rows of x come through a tensor map with the
+// 128-byte swizzle of the B operand (rows past the end are filled with zeros).  One thread issues the
+// tcgen05.mma; four warps read the accumulators back, apply the epilogue of the tile's segment and store
+// -- two accumulator buffers in TMEM, so that an epilogue overlaps the products of the next tile.
+// Every mbarrier wait is bounded; one that gives up raises the context's device error word.
+#include <cuda.h>
+
+#include <algorithm>
+
+#include "dense.cuh"
+#include "tc5_ptx.cuh"
+
+namespace prism {
+
+constexpr int DG_THREADS = 192;               // loader warp, MMA warp, four epilogue warps
+constexpr int DG_A_BYTES = 128 * 64 * 2;      // weights of a stage
+template <int NT>
+struct DgCfg {
+    static constexpr int B_BYTES = NT * 128;
+    static constexpr int STAGE = DG_A_BYTES + B_BYTES;
+    static constexpr int S = (200 * 1024 / STAGE) < 8 ? (200 * 1024 / STAGE) : 8;
+    static constexpr int TMEM_COLS = 2 * NT < 32 ? 32 : 2 * NT;
+    static constexpr int BAR_OFF = S * STAGE;
+    static constexpr size_t SMEM = BAR_OFF + 8 * (2 * S + 4) + 64 + 1024;  // + slack for the 1 KB alignment of the stages
+};
+
+struct DgArgs {
+    const uint8_t *w;
+    uint32_t kb;              // 64-k stages per row
+    uint32_t n_rt, n_tt, rt_group;  // row tiles, token tiles, row tiles per group of the walk
+    uint32_t rows;            // rows of x
+    unsigned int *err;
+    DenseEpi epi;
+};
+
+__device__ __forceinline__ void tma_2d(uint32_t dst, const CUtensorMap *map, int32_t x, int32_t y, uint32_t mbar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(dst),
+                 "l"(map), "r"(x), "r"(y), "r"(mbar)
+                 : "memory");
+}
+__device__ __forceinline__ void mma_ss(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}\n" ::"r"(d_tmem),
+        "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+// K-major operand with the 128-byte swizzle: rows of 128 bytes, eight-row groups 1024 bytes apart.
+__device__ __forceinline__ uint64_t desc_sw128(uint32_t addr) {
+    return (uint64_t)((addr & 0x3FFFFu) >> 4) | (uint64_t)1 << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+
+// Walk of the tiles: groups of rt_group row tiles over all token tiles, so that the CTAs of one wave share a
+// few weights and a few rows of x in L2.
+__device__ __forceinline__ void dg_item(const DgArgs &a, uint32_t w, uint32_t &rt, uint32_t &tt) {
+    const uint32_t per = a.rt_group * a.n_tt, g = w / per, rem = w % per;
+    const uint32_t gr = min(a.rt_group, a.n_rt - g * a.rt_group);
+    rt = g * a.rt_group + rem % gr;
+    tt = rem / gr;
+}
+
+template <int NT>
+__global__ void __launch_bounds__(DG_THREADS, 1) dense_gemm_tc5_kernel(const DgArgs a, const __grid_constant__ CUtensorMap xmap) {
+    using C = DgCfg<NT>;
+    extern __shared__ uint8_t dg_smem_raw[];
+    uint8_t *smem = dg_smem_raw + (1024 - ((uint32_t)__cvta_generic_to_shared(dg_smem_raw) & 1023u)) % 1024;
+    const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
+    pdl_launch_dependents();
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const uint32_t b_full = base + C::BAR_OFF, b_empty = b_full + 8 * C::S, b_dfull = b_empty + 8 * C::S, b_dempty = b_dfull + 16;
+    const uint32_t state = C::BAR_OFF + 8 * (2 * C::S + 4);
+    volatile uint32_t *err_flag = reinterpret_cast<volatile uint32_t *>(smem + state);
+    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(smem + state + 8);
+    const uint32_t n_items = a.n_rt * a.n_tt;
+    if (tid == 0) {
+        for (int s = 0; s < C::S; s++) { t5::mbar_init(b_full + 8 * s, 1); t5::mbar_init(b_empty + 8 * s, 1); }
+        for (int b = 0; b < 2; b++) { t5::mbar_init(b_dfull + 8 * b, 1); t5::mbar_init(b_dempty + 8 * b, 4); }
+        *err_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+    }
+    if (warp == 1) t5::tmem_alloc(base + state + 8, C::TMEM_COLS);
+    t5::fence_before();
+    __syncthreads();
+    t5::fence_after();
+    const uint32_t tmem = *tmem_slot;
+    pdl_wait();  // before any bounded wait: the kernel before this one may still be at work
+
+    if (warp == 0) {
+        if (lane == 0) {
+            uint32_t n = 0;
+            for (uint32_t w = blockIdx.x; w < n_items; w += gridDim.x) {
+                uint32_t rt, tt;
+                dg_item(a, w, rt, tt);
+                const uint8_t *wsrc = a.w + (size_t)rt * a.kb * DG_A_BYTES;
+                for (uint32_t k = 0; k < a.kb; k++, n++) {
+                    const uint32_t s = n % C::S, ph = (n / C::S) & 1, dst = base + s * C::STAGE;
+                    t5::mbar_wait_bounded(b_empty + 8 * s, ph ^ 1, err_flag);
+                    t5::mbar_arrive_expect_tx(b_full + 8 * s, C::STAGE);
+                    t5::bulk_g2s(dst, wsrc + (size_t)k * DG_A_BYTES, DG_A_BYTES, b_full + 8 * s);
+                    tma_2d(dst + DG_A_BYTES, &xmap, (int32_t)(k * 64), (int32_t)(tt * NT), b_full + 8 * s);
+                }
+            }
+            // every copy in flight lands before the CTA leaves (a stage's last use is committed to its empty barrier)
+            for (uint32_t i = 0; i < (uint32_t)C::S && i < n; i++) {
+                const uint32_t m = n - 1 - i, s = m % C::S;
+                t5::mbar_wait_bounded(b_full + 8 * s, (m / C::S) & 1, err_flag);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc = t5::idesc_f16(128, NT) | (1u << 7) | (1u << 10);  // A and B bf16
+            uint32_t n = 0, ti = 0;
+            for (uint32_t w = blockIdx.x; w < n_items; w += gridDim.x, ti++) {
+                const uint32_t b = ti & 1, d = tmem + b * NT;
+                t5::mbar_wait_bounded(b_dempty + 8 * b, ((ti >> 1) & 1) ^ 1, err_flag);
+                t5::fence_after();
+                for (uint32_t k = 0; k < a.kb; k++, n++) {
+                    const uint32_t s = n % C::S, ph = (n / C::S) & 1, sa = base + s * C::STAGE, sb = sa + DG_A_BYTES;
+                    t5::mbar_wait_bounded(b_full + 8 * s, ph, err_flag);
+                    t5::fence_after();
+#pragma unroll
+                    for (int j = 0; j < 4; j++)  // 16 k each: two k/8 slabs of 2 KB in A, 32 bytes inside the swizzled rows of B
+                        mma_ss(d, t5::smem_desc(sa + j * 4096, 2048, 128), desc_sw128(sb + j * 32), idesc, (k | j) != 0);
+                    t5::commit(b_empty + 8 * s);
+                }
+                t5::commit(b_dfull + 8 * b);
+            }
+        }
+    } else {
+        const uint32_t q = warp & 3;  // the TMEM lanes a warp may read
+        uint32_t ti = 0;
+        for (uint32_t w = blockIdx.x; w < n_items; w += gridDim.x, ti++) {
+            uint32_t rt, tt;
+            dg_item(a, w, rt, tt);
+            const uint32_t b = ti & 1;
+            uint32_t sg = 0;
+            while (sg + 1 < a.epi.n && rt * 128 >= a.epi.s[sg + 1].row0) sg++;
+            const DenseEpiSeg &seg = a.epi.s[sg];
+            const uint32_t row = rt * 128 + q * 32 + lane - seg.row0;
+            const bool row_ok = row < seg.rows;
+            t5::mbar_wait_warp(b_dfull + 8 * b, (ti >> 1) & 1, err_flag);
+            t5::fence_after();
+#pragma unroll 1
+            for (int g = 0; g < NT / 16; g++) {
+                uint32_t v[16];
+                t5::ld16(tmem + ((q * 32) << 16) + b * NT + g * 16, v);
+                t5::wait_ld();
+                const uint32_t t0 = tt * NT + g * 16;
+                if (row_ok && t0 < a.rows) {
+#pragma unroll
+                    for (int i = 0; i < 16; i++)
+                        if (t0 + i < a.rows) dense_store<bf16>(seg, row, t0 + i, __uint_as_float(v[i]));
+                }
+            }
+            t5::fence_before();
+            __syncwarp();
+            if (lane == 0) t5::mbar_arrive(b_dempty + 8 * b);
+        }
+    }
+    t5::fence_before();
+    __syncthreads();
+    t5::fence_after();
+    if (warp == 1) t5::tmem_dealloc(tmem, C::TMEM_COLS);
+    if (tid == 0 && *err_flag) atomicExch(a.err, 5u);
+}
+
+// ---- host side ---------------------------------------------------------------------------------
+typedef CUresult (*TensorMapEncode)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
+                                    const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                    CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+static TensorMapEncode tensor_map_encode() {
+    static TensorMapEncode fn = [] {
+        void *p = nullptr;
+        cudaDriverEntryPointQueryResult st;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &st) != cudaSuccess || st != cudaDriverEntryPointSuccess)
+            p = nullptr;
+        return reinterpret_cast<TensorMapEncode>(p);
+    }();
+    return fn;
+}
+
+template <int NT>
+static int launch_dg(prism_cuda_ctx *ctx, const DenseLinear &l, DgArgs &a, const bf16 *x, uint32_t pitch) {
+    using C = DgCfg<NT>;
+    static bool configured[PRISM_MAX_DEVICES] = {false};
+    if (!configured[ctx->device]) {
+        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemm_tc5_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+        configured[ctx->device] = true;
+    }
+    TensorMapEncode enc = tensor_map_encode();
+    if (!enc) return fail(ctx, PRISM_E_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
+    CUtensorMap map;
+    const cuuint64_t dims[2] = {l.k_pad, a.rows}, strides[1] = {(cuuint64_t)pitch * 2};
+    const cuuint32_t box[2] = {64, NT}, estr[2] = {1, 1};
+    const CUresult rc = enc(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16 *>(x), dims, strides, box, estr,
+                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (rc != CUDA_SUCCESS) return fail(ctx, PRISM_E_CUDA, "cuTensorMapEncodeTiled failed: " + std::to_string((int)rc));
+    a.n_tt = (a.rows + NT - 1) / NT;
+    const uint32_t G = (uint32_t)ctx->sm_count;
+    a.rt_group = std::min(a.n_rt, std::max(1u, (G + a.n_tt - 1) / a.n_tt));
+    const uint32_t grid = std::min(G, a.n_rt * a.n_tt);
+    launch_pdl(ctx, "dense_gemm_tc5_kernel", dense_gemm_tc5_kernel<NT>, dim3(grid), dim3(DG_THREADS), C::SMEM, a, map);
+    return after_launch(ctx, "dense_gemm_tc5_kernel");
+}
+
+int launch_dense_gemm_tc5(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 *x, uint32_t pitch, const DenseOut *outs, uint32_t rows) {
+    if ((reinterpret_cast<uintptr_t>(x) & 15) || pitch % 8 || pitch < l.k_pad || l.k_pad % 64)
+        return fail(ctx, PRISM_E_ARG, "dense gemm: input rows must be 16-byte aligned and hold the padded k range");
+    DgArgs a{};
+    a.w = reinterpret_cast<const uint8_t *>(l.w);
+    a.kb = l.k_pad / 64;
+    a.n_rt = l.n_tiles;
+    a.rows = rows;
+    a.err = ctx->dev_err;
+    a.epi = dense_epi(l, outs);
+    // token tile: as small as the batch allows, and small enough that the tiles cover the GPU
+    if (rows <= 16) return launch_dg<16>(ctx, l, a, x, pitch);
+    if (rows <= 32) return launch_dg<32>(ctx, l, a, x, pitch);
+    if (rows <= 64 || a.n_rt * ((rows + 127) / 128) < (uint32_t)ctx->sm_count) return launch_dg<64>(ctx, l, a, x, pitch);
+    if (rows <= 128 || a.n_rt * ((rows + 255) / 256) < (uint32_t)ctx->sm_count) return launch_dg<128>(ctx, l, a, x, pitch);
+    return launch_dg<256>(ctx, l, a, x, pitch);
+}
+
+}  // namespace prism

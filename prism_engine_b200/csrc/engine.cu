@@ -12,59 +12,7 @@
 #include <cstring>
 
 #include "../../include/prism_cuda_bench.h"
-#include "common.cuh"
-
-namespace prism {
-int synth_shard(prism_cuda_ctx *ctx, const char *name, uint32_t rows, uint32_t cols, uint32_t bits,
-                uint64_t seed, float sigma, uint32_t row0, uint32_t col0, int32_t *handle);
-}  // namespace prism
-
-struct prism_cuda_engine {
-    prism_cuda_ctx *ctx = nullptr;
-    prism_model_config cfg{};
-    int T = 1, rank = 0;
-    // local (per-rank) dimensions
-    uint32_t H = 0, nh_l = 0, nkv_l = 0, hd = 0, qd_l = 0, kvd_l = 0, I_l = 0, V_l = 0;
-    uint32_t head0 = 0, kvhead0 = 0, i0 = 0, v0 = 0;  // first local q head / kv head / inter row / vocab row
-    std::vector<int32_t> wq, wk, wv, wo, wg, wu, wd;
-    std::vector<int32_t> wqkv;   // q, k, v rows stacked into one tensor (one launch instead of three)
-    bool fused_ready = false;
-    uint16_t *gu = nullptr;      // [2][B][max(I_l, H)] scratch of the batched (GEMM) path
-    uint16_t *qkv = nullptr;     // [B][qkv_stride]: q | k | v of a sequence side by side
-    uint32_t qkv_stride = 0;
-    int32_t embed = -1, lm_head = -1;
-    // activations
-    uint16_t *h = nullptr, *xn = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *att = nullptr,
-             *act = nullptr, *logits = nullptr;
-    float *part = nullptr;       // [B][H] fp32 partial sums of row-parallel matmuls (TP)
-    uint32_t *tok = nullptr, *next = nullptr, *out_tokens = nullptr, *prompts = nullptr;
-    uint64_t *pairs_send = nullptr, *pairs_recv = nullptr;  // TP argmax: (value bits << 32 | ~index)
-    int32_t *scalars = nullptr;  // [0] pos, [1] step, [2] record
-    size_t prompts_cap = 0;
-    uint32_t act_stride = 0, out_cap = 0;
-    void *kc = nullptr, *vc = nullptr;
-    size_t kv_layer_bytes = 0;
-    uint64_t kv_seq_stride = 0;  // fp16: elements, int8: bytes
-    uint32_t kv_slots = 0;       // positions a layer slot can hold
-    uint32_t batch = 0, pos = 0;
-    bool guard_skip = false;     // down_guard && inter != hidden
-    // paged KV cache (cfg.kv_page_size > 0): page table on the device and its host mirror, free pages
-    int32_t *page_tbl = nullptr;             // [max_batch][pages_per_seq]
-    std::vector<int32_t> page_tbl_host, free_pages;
-    std::vector<uint32_t> seq_pages;         // pages each sequence holds
-    uint32_t page_shift = 0, pages_per_seq = 0, pool_pages = 0;
-    // batched prefill scratch (one chunk of prompt tokens of one sequence), grown on demand
-    uint16_t *pf_x = nullptr, *pf_xn = nullptr, *pf_qkv = nullptr, *pf_att = nullptr, *pf_g = nullptr, *pf_u = nullptr,
-             *pf_act = nullptr;
-    uint32_t *pf_tok = nullptr;
-    uint32_t pf_cap = 0;         // tokens the buffers hold
-    cudaGraphExec_t graph = nullptr;
-    uint32_t graph_batch = 0;
-    uint64_t graph_epoch = ~0ull;  // option epoch of the context when the graph (or its eager warm-up) was made
-    cudaEvent_t ev0 = nullptr, ev1 = nullptr, ev2 = nullptr, ev3 = nullptr;
-    double last_ms = 0.0, last_device_ms = 0.0;
-    uint32_t kernels_per_step = 0;
-};
+#include "engine.hpp"
 
 namespace prism {
 
@@ -87,9 +35,10 @@ __global__ void round_add_resid_kernel(const float *__restrict__ sum, uint16_t *
 }
 
 // End of a step: pos += 1; when recording, out_tokens[b][step] = next[b],
-// tok[b] = next[b] (the greedy token feeds the next step), step += 1.
+// tok[b] = next[b] (the greedy token feeds the next step), step += 1.  row_pos (layered models: a position per
+// row) advances with it.
 __global__ void advance_kernel(int32_t *scalars, const uint32_t *__restrict__ next, uint32_t *__restrict__ tok,
-                               uint32_t *__restrict__ out_tokens, uint32_t batch, uint32_t out_cap) {
+                               uint32_t *__restrict__ out_tokens, uint32_t batch, uint32_t out_cap, int32_t *row_pos) {
     pdl_launch_dependents();
     pdl_wait();
     const int32_t step = scalars[1], record = scalars[2];
@@ -100,6 +49,8 @@ __global__ void advance_kernel(int32_t *scalars, const uint32_t *__restrict__ ne
             if ((uint32_t)step < out_cap) out_tokens[(size_t)b * out_cap + step] = t;
         }
     }
+    if (row_pos)
+        for (uint32_t b = threadIdx.x; b < batch; b += blockDim.x) row_pos[b] += 1;
     __syncthreads();
     if (threadIdx.x == 0) {
         scalars[0] += 1;
@@ -224,7 +175,13 @@ static int enqueue_attention(prism_cuda_engine *e, uint32_t l, uint32_t li) {
     return launch_attention(ctx, aa);
 }
 
+int enqueue_advance(prism_cuda_engine *e, int32_t *row_pos) {
+    launch_pdl(e->ctx, "advance_kernel", advance_kernel, 1, 64, 0, e->scalars, e->next, e->tok, e->out_tokens, e->batch, e->out_cap, row_pos);
+    return after_launch(e->ctx, "advance_kernel");
+}
+
 static int enqueue_step(prism_cuda_engine *e) {
+    if (e->lm) return layered_enqueue_step(e);
     prism_cuda_ctx *ctx = e->ctx;
     const prism_model_config &c = e->cfg;
     const uint32_t B = e->batch, H = e->H;
@@ -311,8 +268,7 @@ static int enqueue_step(prism_cuda_engine *e) {
     } else {
         PRISM_TRY(launch_argmax(ctx, e->logits, e->V_l, lstride, B, e->next));
     }
-    launch_pdl(ctx, "advance_kernel", advance_kernel, 1, 64, 0, e->scalars, e->next, e->tok, e->out_tokens, B, e->out_cap);
-    return after_launch(ctx, "advance_kernel");
+    return enqueue_advance(e, nullptr);
 }
 
 // Stacks the rows of q, k and v of a layer into one tensor (device-to-device copies of
@@ -344,6 +300,7 @@ static int build_fused_qkv(prism_cuda_engine *e) {
 }
 
 static int check_bound(prism_cuda_engine *e) {
+    if (e->lm) return layered_check_bound(e);
     if (e->embed < 0) return fail(e->ctx, PRISM_E_STATE, "emb miss: no embedding tensor bound");
     for (uint32_t l = 0; l < e->cfg.num_layers; l++) {
         if (e->wq[l] < 0 || e->wk[l] < 0 || e->wv[l] < 0 || e->wo[l] < 0 || e->wg[l] < 0 || e->wu[l] < 0 ||
@@ -388,6 +345,11 @@ static void release_pages(prism_cuda_engine *e) {
     std::fill(e->seq_pages.begin(), e->seq_pages.end(), 0u);
 }
 
+// Entry points that only the palettized step has.
+static int palettized_only(prism_cuda_engine *e) {
+    return e->lm ? fail(e->ctx, PRISM_E_STATE, "not available for a model described layer by layer") : PRISM_OK;
+}
+
 static int capacity_ok(prism_cuda_engine *e, uint32_t steps) {
     const uint64_t need = e->guard_skip ? (uint64_t)(e->pos + steps) * e->cfg.num_layers : (uint64_t)e->pos + steps;
     if (need > e->kv_slots)
@@ -398,7 +360,7 @@ static int capacity_ok(prism_cuda_engine *e, uint32_t steps) {
 // Runs one step: the first call per (batch, options) runs eagerly (this sizes
 // every scratch buffer and sets kernel attributes), the second captures the
 // graph, later ones replay it.
-static int run_step(prism_cuda_engine *e) {
+int run_step(prism_cuda_engine *e) {
     prism_cuda_ctx *ctx = e->ctx;
     // every option can change which kernels a step launches, so a graph is good for one option epoch
     const bool same_cfg = e->graph_batch == e->batch && e->graph_epoch == ctx->option_epoch;
@@ -441,8 +403,6 @@ static int run_step(prism_cuda_engine *e) {
     ctx->launches += 1;
     return PRISM_OK;
 }
-
-static int set_scalars(prism_cuda_engine *e, int32_t pos, int32_t step, int32_t record);
 
 // ---- batched prefill -------------------------------------------------------------------------------
 // The reference prefills with one step() per prompt token (prefill_cpu, engine_impl.rs:1046-1053) and
@@ -544,12 +504,35 @@ static int prefill_batched(prism_cuda_engine *e, uint32_t batch, uint32_t n_prom
     return set_scalars(e, (int32_t)n_prompt, 0, 0);
 }
 
-static int set_scalars(prism_cuda_engine *e, int32_t pos, int32_t step, int32_t record) {
+int set_scalars(prism_cuda_engine *e, int32_t pos, int32_t step, int32_t record) {
     int32_t v[3] = {pos, step, record};
     // pageable source: the copy is complete on return, `v` may go out of scope
     PRISM_CUDA_TRY(e->ctx, cudaMemcpyAsync(e->scalars, v, sizeof v, cudaMemcpyHostToDevice, e->ctx->stream));
     PRISM_CUDA_TRY(e->ctx, cudaStreamSynchronize(e->ctx->stream));
     return PRISM_OK;
+}
+
+// What every engine has whatever its model: tokens in and out, the step's scalars, events.
+int engine_alloc_common(prism_cuda_engine *e, uint32_t B) {
+    prism_cuda_ctx *ctx = e->ctx;
+    auto A = [&](void **p, size_t bytes) { return cudaMalloc(p, (bytes + 255) / 256 * 256); };
+    cudaError_t ce = A((void **)&e->tok, (size_t)B * 4);
+    if (ce == cudaSuccess) ce = A((void **)&e->next, (size_t)B * 4);
+    if (ce == cudaSuccess) ce = A((void **)&e->out_tokens, (size_t)B * e->out_cap * 4);
+    if (ce == cudaSuccess) ce = A((void **)&e->scalars, 64);
+    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev0);
+    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev1);
+    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev2);
+    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev3);
+    if (ce == cudaSuccess) ce = cudaMemsetAsync(e->scalars, 0, 64, ctx->stream);
+    return ce == cudaSuccess ? PRISM_OK : cuda_fail(ctx, ce, "engine allocation");
+}
+
+void engine_drop_graph(prism_cuda_engine *e) {
+    if (!e->graph) return;
+    cudaGraphExecDestroy(e->graph);
+    e->graph = nullptr;
+    e->graph_batch = 0;
 }
 
 }  // namespace prism
@@ -641,12 +624,8 @@ int prism_cuda_engine_create(prism_cuda_ctx *ctx, const prism_model_config *cfg,
     ALLOC(e->act, (size_t)B * e->act_stride * 2);
     ALLOC(e->logits, (size_t)B * round_up_u32(e->V_l, 8) * 2);
     ALLOC(e->part, (size_t)B * e->H * 4);
-    ALLOC(e->tok, (size_t)B * 4);
-    ALLOC(e->next, (size_t)B * 4);
-    ALLOC(e->out_tokens, (size_t)B * e->out_cap * 4);
     ALLOC(e->pairs_send, (size_t)B * 8);
     ALLOC(e->pairs_recv, (size_t)B * 8 * T);
-    ALLOC(e->scalars, 64);
     if (c.kv_page_size) ALLOC(e->page_tbl, (size_t)B * e->pages_per_seq * sizeof(int32_t));
     ALLOC(e->kc, e->kv_layer_bytes * kv_layers);
     ALLOC(e->vc, e->kv_layer_bytes * kv_layers);
@@ -654,15 +633,15 @@ int prism_cuda_engine_create(prism_cuda_ctx *ctx, const prism_model_config *cfg,
     e->q = e->qkv;
     e->k = e->qkv ? e->qkv + e->qd_l : nullptr;
     e->v = e->qkv ? e->qkv + e->qd_l + e->kvd_l : nullptr;
-    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev0);
-    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev1);
-    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev2);
-    if (ce == cudaSuccess) ce = cudaEventCreate(&e->ev3);
     if (ce == cudaSuccess) ce = cudaMemsetAsync(e->act, 0, (size_t)B * e->act_stride * 2, ctx->stream);
-    if (ce == cudaSuccess) ce = cudaMemsetAsync(e->scalars, 0, 64, ctx->stream);
     if (ce != cudaSuccess) {
         prism_cuda_engine_destroy(e);
         return cuda_fail(ctx, ce, "engine allocation");
+    }
+    const int rc_common = engine_alloc_common(e, B);
+    if (rc_common != PRISM_OK) {
+        prism_cuda_engine_destroy(e);
+        return rc_common;
     }
     e->batch = 1;
     if (e->page_tbl) {
@@ -678,6 +657,7 @@ void prism_cuda_engine_destroy(prism_cuda_engine *e) {
     cudaSetDevice(e->ctx->device);
     cudaStreamSynchronize(e->ctx->stream);
     if (e->graph) cudaGraphExecDestroy(e->graph);
+    if (e->lm) layered_destroy(e);
     for (int32_t h : e->wqkv)
         if (h >= 0) prism_cuda_free_tensor(e->ctx, h);
     void *ptrs[] = {e->page_tbl, e->pf_x, e->pf_xn, e->pf_qkv, e->pf_att, e->pf_g, e->pf_u, e->pf_act, e->pf_tok, e->gu, e->h, e->xn, e->qkv, e->att, e->act, e->logits, e->part, e->tok, e->next,
@@ -692,6 +672,7 @@ void prism_cuda_engine_destroy(prism_cuda_engine *e) {
 
 int prism_cuda_engine_bind(prism_cuda_engine *e, uint32_t role, uint32_t layer, int32_t handle) {
     if (!e) return PRISM_E_NULL;
+    PRISM_TRY(palettized_only(e));
     prism_cuda_ctx *ctx = e->ctx;
     LutTensor *t = get_tensor(ctx, handle);
     if (!t) return PRISM_E_NOTFOUND;
@@ -724,16 +705,13 @@ int prism_cuda_engine_bind(prism_cuda_engine *e, uint32_t role, uint32_t layer, 
     }
     else if (role == PRISM_ROLE_EMBED) e->embed = handle;
     else e->lm_head = handle;
-    if (e->graph) {  // pointers baked into the graph are stale
-        cudaGraphExecDestroy(e->graph);
-        e->graph = nullptr;
-        e->graph_batch = 0;
-    }
+    engine_drop_graph(e);  // pointers baked into the graph are stale
     return PRISM_OK;
 }
 
 int prism_cuda_engine_bind_by_keys(prism_cuda_engine *e, const char *key_prefix) {
     if (!e) return PRISM_E_NULL;
+    PRISM_TRY(palettized_only(e));
     prism_cuda_ctx *ctx = e->ctx;
     if (e->T > 1) return fail(ctx, PRISM_E_STATE, "bind_by_keys binds whole tensors; shard and bind explicitly under tensor parallelism");
     const std::string p = key_prefix && *key_prefix ? key_prefix : "model";
@@ -762,6 +740,7 @@ int prism_cuda_engine_bind_by_keys(prism_cuda_engine *e, const char *key_prefix)
 
 int prism_cuda_engine_synth_weights(prism_cuda_engine *e, uint64_t seed, float sigma) {
     if (!e) return PRISM_E_NULL;
+    if (e->lm) return layered_synth(e, seed, sigma);
     prism_cuda_ctx *ctx = e->ctx;
     const prism_model_config &c = e->cfg;
     const uint32_t H = e->H, bits = c.bits;
@@ -797,6 +776,7 @@ int prism_cuda_engine_reset(prism_cuda_engine *e, uint32_t batch) {
     e->batch = batch;
     e->pos = 0;
     release_pages(e);  // a reset returns every page to the pool
+    if (e->lm) PRISM_TRY(layered_reset(e, batch));
     return set_scalars(e, 0, 0, 0);
 }
 
@@ -807,12 +787,16 @@ int prism_cuda_engine_step(prism_cuda_engine *e, const uint32_t *tokens, uint32_
     PRISM_TRY(check_bound(e));
     PRISM_TRY(capacity_ok(e, 1));
     PRISM_TRY(set_scalars(e, (int32_t)e->pos, 0, 0));
+    if (e->lm) PRISM_TRY(layered_set_rows(e, e->pos));
     PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(e->tok, tokens, (size_t)e->batch * 4, cudaMemcpyHostToDevice, ctx->stream));
     PRISM_TRY(run_step(e));
     e->pos += 1;
+    if (e->lm) layered_advance(e, 1);
     if (next_tokens)
         PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(next_tokens, e->next, (size_t)e->batch * 4, cudaMemcpyDeviceToHost, ctx->stream));
-    if (logits) {
+    if (logits && e->lm) {
+        PRISM_TRY(layered_logits_f16(e, logits));
+    } else if (logits) {
         if (e->T > 1) return fail(ctx, PRISM_E_STATE, "logits are sharded under tensor parallelism");
         const uint32_t ls = round_up_u32(e->V_l, 8);
         PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(logits, (size_t)e->V_l * 2, e->logits, (size_t)ls * 2, (size_t)e->V_l * 2,
@@ -833,12 +817,14 @@ int prism_cuda_engine_decode(prism_cuda_engine *e, const uint32_t *tokens_in, ui
     if (n_steps > e->out_cap) return fail(ctx, PRISM_E_ARG, "n_steps exceeds max_seq");
     PRISM_TRY(capacity_ok(e, n_steps));
     PRISM_TRY(set_scalars(e, (int32_t)e->pos, 0, 1));
+    if (e->lm) PRISM_TRY(layered_set_rows(e, e->pos));
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev0, ctx->stream));
     PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(e->tok, tokens_in, (size_t)e->batch * 4, cudaMemcpyHostToDevice, ctx->stream));
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev2, ctx->stream));
     for (uint32_t i = 0; i < n_steps; i++) PRISM_TRY(run_step(e));
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev3, ctx->stream));
     e->pos += n_steps;
+    if (e->lm) layered_advance(e, n_steps);
     PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(out_tokens, (size_t)n_steps * 4, e->out_tokens, (size_t)e->out_cap * 4,
                                           (size_t)n_steps * 4, e->batch, cudaMemcpyDeviceToHost, ctx->stream));
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev1, ctx->stream));
@@ -861,7 +847,10 @@ int prism_cuda_engine_generate(prism_cuda_engine *e, const uint32_t *prompts, ui
     PRISM_TRY(check_bound(e));
     PRISM_TRY(prism_cuda_engine_reset(e, batch));
     if (max_new > e->out_cap) return fail(ctx, PRISM_E_ARG, "max_new exceeds max_seq");
-    PRISM_TRY(capacity_ok(e, n_prompt + max_new));
+    // The layered models predict from the last prompt token where it stands; the reference's loop feeds it a second time.
+    if (e->lm && n_prompt == 0) return fail(ctx, PRISM_E_ARG, "generate needs at least one prompt token");
+    const uint32_t n_pre = e->lm ? n_prompt - 1 : n_prompt;
+    PRISM_TRY(capacity_ok(e, n_pre + max_new));
     // prompts -> device, position-major so a step's tokens are contiguous
     const size_t need = (size_t)std::max<uint32_t>(n_prompt, 1) * batch;
     if (need > e->prompts_cap) {
@@ -878,7 +867,13 @@ int prism_cuda_engine_generate(prism_cuda_engine *e, const uint32_t *prompts, ui
     PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(e->prompts, tr.data(), need * 4, cudaMemcpyHostToDevice, ctx->stream));
     PRISM_CUDA_TRY(ctx, cudaStreamSynchronize(ctx->stream));
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev0, ctx->stream));
-    if (n_prompt >= 2 && prefill_batched_ok(e)) {
+    if (e->lm) {
+        for (uint32_t b = 0; b < batch && n_pre; b++) PRISM_TRY(layered_prefill(e, b, prompts + (size_t)b * n_prompt, n_pre));
+        PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(e->tok, e->prompts + (size_t)(n_prompt - 1) * batch, (size_t)batch * 4,
+                                            cudaMemcpyDeviceToDevice, ctx->stream));
+        PRISM_TRY(set_scalars(e, (int32_t)n_pre, 0, 0));
+        PRISM_TRY(layered_set_rows(e, n_pre));
+    } else if (n_prompt >= 2 && prefill_batched_ok(e)) {
         PRISM_TRY(prefill_batched(e, batch, n_prompt));
     } else {
         // prefill_cpu (engine_impl.rs:1046-1053): one step per prompt token
@@ -888,7 +883,7 @@ int prism_cuda_engine_generate(prism_cuda_engine *e, const uint32_t *prompts, ui
             PRISM_TRY(run_step(e));
         }
     }
-    e->pos = n_prompt;
+    e->pos = n_pre;
     // decode: `nt = *prompt.last().unwrap_or(&0)` (engine_impl.rs:1015) is fed first
     if (n_prompt == 0) PRISM_CUDA_TRY(ctx, cudaMemsetAsync(e->tok, 0, (size_t)batch * 4, ctx->stream));
     {
@@ -899,11 +894,14 @@ int prism_cuda_engine_generate(prism_cuda_engine *e, const uint32_t *prompts, ui
     for (uint32_t i = 0; i < max_new; i++) PRISM_TRY(run_step(e));
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev3, ctx->stream));
     e->pos += max_new;
+    if (e->lm) layered_advance(e, max_new);
     PRISM_CUDA_TRY(ctx, cudaEventRecord(e->ev1, ctx->stream));
     if (max_new)
         PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(out_tokens, (size_t)max_new * 4, e->out_tokens, (size_t)e->out_cap * 4,
                                               (size_t)max_new * 4, batch, cudaMemcpyDeviceToHost, ctx->stream));
-    if (last_logits) {
+    if (last_logits && e->lm) {
+        PRISM_TRY(layered_logits_f16(e, last_logits));
+    } else if (last_logits) {
         if (e->T > 1) return fail(ctx, PRISM_E_STATE, "logits are sharded under tensor parallelism");
         const uint32_t ls = round_up_u32(e->V_l, 8);
         PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(last_logits, (size_t)e->V_l * 2, e->logits, (size_t)ls * 2,
@@ -922,6 +920,7 @@ int prism_cuda_engine_generate(prism_cuda_engine *e, const uint32_t *prompts, ui
 
 uint64_t prism_cuda_engine_step_bytes(prism_cuda_engine *e) {
     if (!e) return 0;
+    if (e->lm) return layered_step_bytes(e);
     prism_cuda_ctx *ctx = e->ctx;
     uint64_t bytes = 0;
     auto add = [&](int32_t h) {
@@ -949,6 +948,7 @@ uint32_t prism_cuda_engine_kernels_per_step(prism_cuda_engine *e) { return e ? e
 extern "C" int prism_cuda_engine_profile_gemv(prism_cuda_engine *e, uint32_t reps, double *ms_out, uint64_t *bytes_out,
                                    uint32_t *launches_out) {
     if (!e || !ms_out) return fail(e ? e->ctx : nullptr, PRISM_E_NULL, "null argument");
+    PRISM_TRY(palettized_only(e));
     prism_cuda_ctx *ctx = e->ctx;
     PRISM_CUDA_TRY(ctx, cudaSetDevice(ctx->device));
     PRISM_TRY(check_bound(e));
@@ -1000,6 +1000,7 @@ extern "C" int prism_cuda_engine_profile_gemv(prism_cuda_engine *e, uint32_t rep
 extern "C" int prism_cuda_engine_profile_part(prism_cuda_engine *e, uint32_t part, uint32_t reps, double *ms_out,
                                               uint32_t *launches_out) {
     if (!e || !ms_out) return fail(e ? e->ctx : nullptr, PRISM_E_NULL, "null argument");
+    PRISM_TRY(palettized_only(e));
     prism_cuda_ctx *ctx = e->ctx;
     if (part != 1 && part != 2) return fail(ctx, PRISM_E_ARG, "profile_part: 1 = attention, 2 = tensor-parallel reductions");
     PRISM_CUDA_TRY(ctx, cudaSetDevice(ctx->device));
