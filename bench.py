@@ -25,6 +25,10 @@ clocks:
   lut_gemv_decode_shapes N = 1: the five GEMV launch shapes of the workload's decode step, each timed alone
   cpu_baseline      N = 1: the CPU restatement of the reference's path on the host cores (a sample)
 
+`--workload mefipel-*` runs a model described layer by layer (lightning and latent attention
+layers in turn, bf16 random weights): prefill of 2048 tokens and decode at batch 1 and 8, beside
+the palettized model of the same width, feed-forward, depth and vocabulary (`sizes` in the line).
+
 `--impl reference` times the CPU restatement of the reference's own path (the
 oracle) on the host cores for the same workload; each of its steps is a bounded
 SAMPLE of a decode step, extrapolated, and the line says so.
@@ -54,6 +58,16 @@ WORKLOADS = {
     "qwen2.5-0.5b-decode": ("QWEN25_0P5B", 128),
     # prefill: the palettized linears of one Qwen2.5-7B layer on M = 2048 tokens (tensor-core GEMM)
     "qwen2.5-7b-prefill-gemm": ("QWEN25_7B", 2048),
+}
+# Models described layer by layer (bf16), each beside the palettized model of the same width, feed-forward, depth and
+# vocabulary: name -> (palettized architecture, layers (0: all of it), mixer sizes)
+LAYERED_WORKLOADS = {
+    "mefipel-0.5b": ("QWEN25_0P5B", 0, dict(lightning=dict(heads=14, dim=64, vdim=64),
+                                            latent=dict(heads=14, dim=64, rot_dim=32, vdim=64, q_rank=448, kv_rank=256, window=1024))),
+    "mefipel-7b": ("QWEN25_7B", 0, dict(lightning=dict(heads=28, dim=128, vdim=128),
+                                        latent=dict(heads=28, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=2048))),
+    "mefipel-72b-8-layers": ("QWEN25_72B", 8, dict(lightning=dict(heads=64, dim=128, vdim=128),
+                                                   latent=dict(heads=64, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=2048))),
 }
 METRIC = "decode_tokens_per_s"
 UNIT = "tok/s"
@@ -639,6 +653,97 @@ def run_gemm(args):
     return 0
 
 
+def layered_raw(name):
+    """config.json of a layered workload: lightning and latent attention layers in turn."""
+    import prism_engine_b200 as p
+
+    arch_name, n_layers, mix = LAYERED_WORKLOADS[name]
+    arch = dict(getattr(p, arch_name))
+    if n_layers:
+        arch["num_layers"] = n_layers
+    li, la = mix["lightning"], mix["latent"]
+    decay = [1.0 - 2.0 ** (-4.0 - 6.0 * h / li["heads"]) for h in range(li["heads"])]
+    lightning = {"type": "lightning", "mixer": dict(li, decay=decay)}
+    latent = {"type": "latent_attention", "mixer": dict(
+        {k: v for k, v in la.items() if k != "window"}, mask={"size": la["window"]}, scale=(la["dim"] + la["rot_dim"]) ** -0.5,
+        rot={"base": 1e6, "dims": la["rot_dim"], "scaling": {"factor": 4.0, "fast": 32.0, "original": 4096, "slow": 1.0}})}
+    layers = [dict(latent if i % 2 else lightning, mlp={"kind": "dense", "ff": arch["intermediate_size"]})
+              for i in range(arch["num_layers"])]
+    raw = {"architecture": "Mefipel", "layers": layers, "logit_scale": 1.0, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+           "vocab": arch["vocab_size"], "width": arch["hidden_size"]}
+    return raw, arch
+
+
+def linear_flops_per_token(cfg):
+    """2 x weights of every linear a prompt token goes through (no head; keys and values expanded once per token)."""
+    return 2.0 * sum(float(np.prod(s)) for n, s in cfg.tensor_shapes().items() if len(s) == 2 and n not in ("embed", "head"))
+
+
+def measure_layered(env, be, name, batches, steps, warmup, ctx_len, n_prompt):
+    import prism_engine_b200 as p
+    from prism_engine_b200 import synth
+
+    raw, arch = layered_raw(name)
+    cfg = p.LayeredConfig.from_dict(raw)
+    peak, _ = measured_peaks()
+    sustained, _, _ = measured_tensor_peak()
+    H, I, L = arch["hidden_size"], arch["intermediate_size"], arch["num_layers"]
+    qkv = (arch["num_heads"] + 2 * arch["num_kv_heads"]) * arch["head_dim"]
+    pal_flops = 2.0 * L * (qkv * H + H * arch["num_heads"] * arch["head_dim"] + 3 * H * I)
+    max_seq = max(ctx_len + 40 + 2 * (warmup + steps), n_prompt) + 16
+    out = {}
+    for kind in ("layered", "palettized"):
+        if kind == "layered":
+            eng = p.PrismEngine(be, cfg, max_seq=max_seq, max_batch=max(batches))
+        else:
+            eng = p.PrismEngine(be, p.model_config(**arch, max_seq=max_seq, max_batch=max(batches), profile="baseline"))
+        eng.synth_weights(seed=1)
+        prompt = synth.make_prompt(n_prompt, arch["vocab_size"], seed=3)
+        for _ in range(2):
+            eng.generate(prompt, 0)
+        reps = 5
+        ms = 0.0
+        for _ in range(reps):
+            eng.generate(prompt, 0)
+            ms += eng.last_ms()
+        ms /= reps
+        flops = (linear_flops_per_token(cfg) if kind == "layered" else pal_flops) * n_prompt
+        res = {"prefill": {"tokens": n_prompt, "ms": ms, "tok_s": n_prompt / ms * 1e3, "linear_tflops": flops / ms / 1e9,
+                           "frac_of_sustained": flops / ms / 1e9 / sustained}}
+        for b in batches:
+            m, _ = measure_decode(env, be, eng, arch, b, ctx_len, steps, warmup)
+            res[f"decode_batch{b}"] = m
+        res["weights"] = "bf16" if kind == "layered" else "4-bit palettized"
+        out[kind] = res
+        eng.close()
+    return out
+
+
+def run_layered(args):
+    """Prefill and decode of a model described layer by layer beside the palettized model of equal size."""
+    import prism_engine_b200 as p
+
+    env = Env(args)
+    if env.world > 1:
+        raise SystemExit("layered models run on one GPU")
+    be = p.CudaBackend(device=env.local)
+    for kv in args.option:
+        key, val = kv.split("=")
+        be.set_option(key, int(val))
+    ctx_len = 512 if args.ctx < 0 else args.ctx
+    res = measure_layered(env, be, args.workload, sorted({1, 8, args.batch}), args.steps, args.warmup, ctx_len, 2048)
+    main = res["layered"][f"decode_batch{args.batch}"]
+    emit({"metric": METRIC, "value": main["value"], "unit": UNIT, "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+          "ms_per_step": main["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+          "dtype": "bf16 weights and activations / f32 residual, state and accumulate", "data": "synthetic",
+          "config": {"workload": f"{args.workload}: batch {args.batch}, {ctx_len}-token context, greedy", "model": args.workload,
+                     "l2_policy": "every step streams all weights of the model (larger than L2) from HBM"},
+          "step_roofline": main["step_roofline"], "e2e": main["e2e"], "gpu_launches": main["kernels_per_step"] * args.steps,
+          "clocks": main["clocks"], "sizes": res})
+    be.close()
+    return 0
+
+
 _RESULT_FD = None
 
 
@@ -664,7 +769,7 @@ def main():
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="qwen2.5-72b-decode", choices=sorted(WORKLOADS))
+    ap.add_argument("--workload", default="qwen2.5-72b-decode", choices=sorted(WORKLOADS) + sorted(LAYERED_WORKLOADS))
     ap.add_argument("--batch", type=int, default=1)
     ap.add_argument("--bits", type=int, default=4, choices=[2, 4], help="palette width of the prefill-GEMM workload")
     ap.add_argument("--layers", type=int, default=0, help="override the layer count (profiling/debugging only)")
@@ -678,6 +783,11 @@ def main():
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
+    if args.workload in LAYERED_WORKLOADS:
+        if args.impl == "reference":
+            emit({"impl": "reference", "unavailable": "the reference has no model of this design"})
+            return 0
+        return run_layered(args)
     if args.workload.endswith("prefill-gemm"):
         if args.impl == "reference":
             emit({"impl": "reference", "unavailable": "the reference arm times decode; run the decode workloads"})

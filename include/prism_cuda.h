@@ -89,6 +89,7 @@ int prism_cuda_synchronize(prism_cuda_ctx *ctx);
  * "prefill_chunk" (default 512: prism_cuda_engine_generate puts up to this many prompt tokens of a sequence
  * through the layers at once -- tensor-core GEMMs, causal attention over the cache, no LM head -- instead of
  * one step per token as the reference's prefill_cpu does; 0 = one step per token.  Single GPU, fp16 KV),
+ * "layered_chunk" (default 2048: the same for models described layer by layer; read when the engine is created),
  * "tp_fused_ar" (batch-1 tensor-parallel decode, how the partial sums of a row-parallel matmul are reduced:
  * 0 = the GEMV leaves fp32 partial sums, one kernel pushes them to the peers and reduces; 1 = the GEMV's epilogue
  * stores its sums into every rank's receive area, a small kernel publishes flags, waits and reduces; 2 = flags,
@@ -386,7 +387,7 @@ typedef struct prism_layered_config {
 } prism_layered_config;
 
 /* The arrays inside the layer configs are copied.  Prompt portions go through the layers in chunks of the
- * context's "prefill_chunk" option at the time of this call (windowed caches are sized by it). */
+ * context's "layered_chunk" option at the time of this call (windowed caches are sized by it). */
 int prism_cuda_engine_create_layered(prism_cuda_ctx *ctx, const prism_layered_config *cfg, const prism_layer_config *layers,
                                      prism_cuda_engine **out);
 /* Sets one tensor by its checkpoint name ("embed", "l0.norm1", "l0.mix.q", "l0.mlp.up.b", "final.norm", "head",
@@ -397,7 +398,7 @@ int prism_cuda_engine_set_tensor(prism_cuda_engine *eng, const char *name, const
  * or another type, or when one the model needs is missing. */
 int prism_cuda_engine_load_safetensors(prism_cuda_engine *eng, const char *path);
 /* Sequences of a layered engine (at most max_batch at a time): open gives a slot whose state is empty, close
- * gives it back.  reset() and generate() close all of them and use slots 0 .. batch-1. */
+ * gives it back.  reset() and generate() close all of them and use slots 0 .. batch-1 (reset(0) only closes). */
 int prism_cuda_engine_seq_open(prism_cuda_engine *eng, uint32_t *seq);
 int prism_cuda_engine_seq_close(prism_cuda_engine *eng, uint32_t seq);
 int prism_cuda_engine_seq_position(prism_cuda_engine *eng, uint32_t seq, uint32_t *pos);

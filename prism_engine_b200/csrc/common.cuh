@@ -84,6 +84,7 @@ struct prism_cuda_ctx {
     int gemm_reuse_x = 0;    // set by a caller for the second of two GEMMs over the same activations: skip the re-lay
     int pdl = 1;  // programmatic dependent launch between the kernels of the decode chain
     int prefill_chunk = 512;  // prompt tokens generate() puts through the layers at once (tensor-core GEMMs); 0: one step per token
+    int layered_chunk = 2048;  // layered models: most prompt tokens of a sequence that go through the layers at once (read at engine creation)
     int cimage_cache = 0;  // engine_load_cimage keeps / uses the cache of the re-laid image beside the file
     // Upper bound, in polls, of the device-side waits on something outside the waiting CTA (a peer
     // GPU's flag, a grid-wide arrival); a wait that runs out sets the device error word and the
@@ -319,6 +320,7 @@ int launch_silu_mul(prism_cuda_ctx *ctx, uint16_t *out, const uint16_t *g, const
 int launch_softmax(prism_cuda_ctx *ctx, const uint16_t *in, uint16_t *out, uint32_t n);
 int launch_argmax(prism_cuda_ctx *ctx, const uint16_t *logits, uint32_t n, uint32_t stride, uint32_t batch,
                   uint32_t *out_dev);
+int launch_argmax(prism_cuda_ctx *ctx, const float *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev);
 struct AttnArgs {
     const uint16_t *q;      // [batch] rows of nh*hd, q_stride halfs apart
     uint32_t q_stride;

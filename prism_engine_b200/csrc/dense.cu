@@ -1,8 +1,12 @@
 // Dense bf16 linears for few rows, the same linears in 32-bit, and the element-wise kernels around
 // them: weight packing, RMS norm with a weight, embedding gather, fp32 argmax.
+#include <cooperative_groups.h>
+
 #include <algorithm>
 
 #include "dense.cuh"
+
+namespace cg = cooperative_groups;
 
 namespace prism {
 
@@ -86,10 +90,11 @@ DenseEpi dense_epi(const DenseLinear &l, const DenseOut *outs) {
 // rows, and the same eight k of token g of the input.  The order of k inside a dot product is free as long
 // as both operands agree, so these registers ARE the fragments of two m16n8k16 products per 16 rows: no
 // conversion, no shuffles, and any batch of 1..8 costs the same.  The sums of the warps meet in shared
-// memory in a fixed order.
+// memory in a fixed order.  When there are too few row blocks for the GPU a cluster of `ks` CTAs shares the
+// k range of a block; the sums of ranks 1.. travel to rank 0 through distributed shared memory.
 struct GemvArgs {
     const uint4 *w;
-    uint32_t k8, n_groups, rows;
+    uint32_t k8, n_groups, rows, ks;
     const void *x;
     uint32_t pitch, f32;
     const float *norm_w;
@@ -98,7 +103,7 @@ struct GemvArgs {
     float eps;
     DenseEpi epi;
 };
-constexpr int GV_THREADS = 256, GV_WARPS = 8, GV_U = 4;
+constexpr int GV_THREADS = 256, GV_WARPS = 8, GV_U = 4, GV_KS_MAX = 4;
 
 // RMS norm (times weight, times gate) of the first n_norm entries of every row into shared memory as bf16.
 __device__ __forceinline__ void gemv_stage_norm(const GemvArgs &a, bf16 *xs, float *sh) {
@@ -138,11 +143,16 @@ template <bool NORM>
 __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArgs a) {
     extern __shared__ __align__(16) uint8_t dsm[];
     __shared__ float red[GV_WARPS][8][33];
+    __shared__ float peer[GV_KS_MAX][8][32];  // rank 0: sums of the other ranks
     __shared__ float sh[32];
     bf16 *xs = reinterpret_cast<bf16 *>(dsm);
     pdl_launch_dependents();
+    cg::cluster_group cluster = cg::this_cluster();
+    const uint32_t rank = a.ks > 1 ? cluster.block_rank() : 0;
+    if (a.ks > 1) asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");  // met before the first remote store
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g8 = lane >> 2, t4 = lane & 3;
-    const uint32_t steps = a.k8 / 4, norm8 = NORM ? a.norm_pad / 8 : 0;
+    const uint32_t all_steps = a.k8 / 4, norm8 = NORM ? a.norm_pad / 8 : 0;
+    const uint32_t first = all_steps * rank / a.ks, steps = all_steps * (rank + 1) / a.ks;  // this rank's k range
     const bool tok_on = g8 < a.rows;
     const uint4 *xg = reinterpret_cast<const uint4 *>(reinterpret_cast<const bf16 *>(a.x) + (size_t)g8 * a.pitch);
     const uint4 *xl = reinterpret_cast<const uint4 *>(xs + (size_t)g8 * a.norm_pad);
@@ -169,15 +179,16 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
         }
     };
     uint32_t sg, rb;
-    const uint4 *wt = locate(blockIdx.x, sg, rb);
-    load(wt, warp);  // weights do not depend on the previous kernel; the input does
+    const uint32_t grp0 = blockIdx.x / a.ks;
+    const uint4 *wt = locate(grp0, sg, rb);
+    load(wt, first + warp);  // weights do not depend on the previous kernel; the input does
     pdl_wait();
     if (NORM) gemv_stage_norm(a, xs, sh);
     bool loaded = true;
-    for (uint32_t grp = blockIdx.x; grp < a.n_groups; grp += gridDim.x) {
+    for (uint32_t grp = grp0; grp < a.n_groups; grp += gridDim.x / a.ks) {
         if (!loaded) wt = locate(grp, sg, rb);
         float acc[2][4] = {};
-        for (uint32_t s0 = warp; s0 < steps; s0 += GV_WARPS * GV_U) {
+        for (uint32_t s0 = first + warp; s0 < steps; s0 += GV_WARPS * GV_U) {
             if (!loaded) load(wt, s0);
             loaded = false;
 #pragma unroll
@@ -204,12 +215,17 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
             for (int i = 0; i < 4; i++) red[warp][2 * t4 + (i & 1)][16 * m + g8 + 8 * (i >> 1)] = acc[m][i];
         __syncthreads();
         const uint32_t t = threadIdx.x >> 5, rl = rb * 32 + lane;
-        if (t < a.rows && rl < a.epi.s[sg].rows) {
-            float v = 0.0f;
+        float v = 0.0f;
 #pragma unroll
-            for (int w = 0; w < GV_WARPS; w++) v += red[w][t][lane];
-            dense_store<bf16>(a.epi.s[sg], rl, t, v);
+        for (int w = 0; w < GV_WARPS; w++) v += red[w][t][lane];
+        if (a.ks > 1) {  // one block per cluster (the grid is n_groups * ks)
+            asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
+            if (rank) *cluster.map_shared_rank(&peer[rank][t][lane], 0) = v;
+            cluster.sync();
+            if (rank) return;
+            for (uint32_t r = 1; r < a.ks; r++) v += peer[r][t][lane];
         }
+        if (t < a.rows && rl < a.epi.s[sg].rows) dense_store<bf16>(a.epi.s[sg], rl, t, v);
         __syncthreads();
     }
 }
@@ -218,10 +234,11 @@ static size_t gemv_smem(const DenseIn &in, uint32_t rows) {
     return in.norm_w ? (size_t)rows * round_up_u32(in.n_norm, 64) * 2 : 0;
 }
 constexpr size_t GV_SMEM_MAX = 160 * 1024;
+constexpr uint32_t GV_FOLD_ROWS = 2;  // more rows: every CTA norming all of them costs more than a norm kernel does
 
-bool dense_gemv_ok(const DenseLinear &l, const DenseIn &in, uint32_t rows) {
-    (void)l;
-    return rows <= DENSE_GEMV_ROWS && gemv_smem(in, rows) <= GV_SMEM_MAX && (in.norm_w || !in.f32) && (in.f32 || in.pitch % 8 == 0);
+bool dense_gemv_ok(const DenseIn &in, uint32_t rows) {
+    return rows <= DENSE_GEMV_ROWS && (in.norm_w ? rows <= GV_FOLD_ROWS && gemv_smem(in, rows) <= GV_SMEM_MAX : !in.f32) &&
+           (in.f32 || in.pitch % 8 == 0);
 }
 
 int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows) {
@@ -234,17 +251,21 @@ int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &
     a.gate = reinterpret_cast<const bf16 *>(in.gate); a.gate_pitch = in.gate_pitch;
     a.epi = dense_epi(l, outs);
     for (uint32_t s = 0; s < l.n_segs; s++) a.n_groups += (l.seg[s].rows + 31) / 32;
+    // few row blocks and a long k: share a block's k range inside a cluster, at least GV_WARPS * GV_U steps each
+    const uint32_t slots = 2u * (uint32_t)ctx->sm_count;
+    a.ks = 1;
+    while (a.ks < GV_KS_MAX && a.n_groups * a.ks * 2 <= slots + slots / 2 && a.k8 / 4 >= a.ks * 2 * GV_WARPS * GV_U) a.ks *= 2;
     const size_t smem = gemv_smem(in, rows);
-    const uint32_t grid = std::min(a.n_groups, 2u * (uint32_t)ctx->sm_count);
+    const uint32_t grid = a.ks > 1 ? a.n_groups * a.ks : std::min(a.n_groups, slots);
     if (in.norm_w) {
         static bool configured[PRISM_MAX_DEVICES] = {false};
         if (!configured[ctx->device]) {
             PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemv_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GV_SMEM_MAX));
             configured[ctx->device] = true;
         }
-        launch_pdl(ctx, "dense_gemv_kernel", dense_gemv_kernel<true>, grid, GV_THREADS, smem, a);
+        launch_cluster_pdl(ctx, dense_gemv_kernel<true>, grid, GV_THREADS, smem, a.ks, a);
     } else {
-        launch_pdl(ctx, "dense_gemv_kernel", dense_gemv_kernel<false>, grid, GV_THREADS, 0, a);
+        launch_cluster_pdl(ctx, dense_gemv_kernel<false>, grid, GV_THREADS, 0, a.ks, a);
     }
     return after_launch(ctx, "dense_gemv_kernel");
 }
@@ -302,37 +323,76 @@ int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const float *x, 
 }
 
 // ---- element-wise ------------------------------------------------------------------------------------
+// Four consecutive values of a row.
+__device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 ld4(const bf16 *p) {
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void st4(bf16 *p, float4 v) { *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+
+constexpr int DN_THREADS = 256, DN_U = 8;  // a row of up to 8192 values is read once and kept in registers
 template <typename TX, typename TA>
-__global__ void __launch_bounds__(256) dense_norm_kernel(const TX *__restrict__ x, uint32_t pitch, const float *__restrict__ w, const TA *__restrict__ gate,
-                                                         uint32_t gate_pitch, uint32_t n, float eps, TA *y, uint32_t y_pitch) {
+__global__ void __launch_bounds__(DN_THREADS) dense_norm_kernel(const TX *__restrict__ x, uint32_t pitch, const float *__restrict__ w,
+                                                                const TA *__restrict__ gate, uint32_t gate_pitch, uint32_t n, float eps, TA *y,
+                                                                uint32_t y_pitch, uint32_t vec) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float sh[32];
     const uint32_t r = blockIdx.x;
     const TX *xr = x + (size_t)r * pitch;
+    const TA *gr = gate ? gate + (size_t)r * gate_pitch : nullptr;
+    TA *yr = y + (size_t)r * y_pitch;
     float ss = 0.0f;
-    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+    if (vec) {
+        float4 v[DN_U];
+#pragma unroll
+        for (int u = 0; u < DN_U; u++) {
+            const uint32_t i = (threadIdx.x + u * DN_THREADS) * 4;
+            v[u] = i < n ? ld4(xr + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+        }
+        ss = block_sum_f(ss, sh);
+        const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+        for (int u = 0; u < DN_U; u++) {
+            const uint32_t i = (threadIdx.x + u * DN_THREADS) * 4;
+            if (i >= n) break;
+            const float4 wv = ld4(w + i);
+            float4 o = make_float4(v[u].x * inv * wv.x, v[u].y * inv * wv.y, v[u].z * inv * wv.z, v[u].w * inv * wv.w);
+            if (gr) {
+                const float4 g = ld4(gr + i);
+                o = make_float4(o.x * g.x, o.y * g.y, o.z * g.z, o.w * g.w);
+            }
+            st4(yr + i, o);
+        }
+        return;
+    }
+    for (uint32_t i = threadIdx.x; i < n; i += DN_THREADS) {
         const float v = ld_act(xr + i);
         ss += v * v;
     }
     ss = block_sum_f(ss, sh);
     const float inv = 1.0f / sqrtf(ss / (float)n + eps);
-    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+    for (uint32_t i = threadIdx.x; i < n; i += DN_THREADS) {
         float v = ld_act(xr + i) * inv * __ldg(w + i);
-        if (gate) v *= ld_act(gate + (size_t)r * gate_pitch + i);
-        st_act(y + (size_t)r * y_pitch + i, v);
+        if (gr) v *= ld_act(gr + i);
+        st_act(yr + i, v);
     }
 }
+template <typename TX, typename TA>
+static void run_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t y_pitch, uint32_t rows) {
+    const uintptr_t p = reinterpret_cast<uintptr_t>(in.x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(in.gate) | reinterpret_cast<uintptr_t>(in.norm_w);
+    const uint32_t vec = !(p & 15) && !((in.pitch | y_pitch | in.n_norm | (in.gate ? in.gate_pitch : 0)) & 3) && in.n_norm <= DN_THREADS * DN_U * 4;
+    launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<TX, TA>, rows, DN_THREADS, 0, (const TX *)in.x, in.pitch, in.norm_w, (const TA *)in.gate,
+               in.gate_pitch, in.n_norm, in.eps, (TA *)y, y_pitch, vec);
+}
 int launch_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t y_pitch, uint32_t rows, bool act32) {
-    if (act32)
-        launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<float, float>, rows, 256, 0, (const float *)in.x, in.pitch, in.norm_w,
-                   (const float *)in.gate, in.gate_pitch, in.n_norm, in.eps, (float *)y, y_pitch);
-    else if (in.f32)
-        launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<float, bf16>, rows, 256, 0, (const float *)in.x, in.pitch, in.norm_w,
-                   (const bf16 *)in.gate, in.gate_pitch, in.n_norm, in.eps, (bf16 *)y, y_pitch);
-    else
-        launch_pdl(ctx, "dense_norm_kernel", dense_norm_kernel<bf16, bf16>, rows, 256, 0, (const bf16 *)in.x, in.pitch, in.norm_w,
-                   (const bf16 *)in.gate, in.gate_pitch, in.n_norm, in.eps, (bf16 *)y, y_pitch);
+    if (act32) run_dense_norm<float, float>(ctx, in, y, y_pitch, rows);
+    else if (in.f32) run_dense_norm<float, bf16>(ctx, in, y, y_pitch, rows);
+    else run_dense_norm<bf16, bf16>(ctx, in, y, y_pitch, rows);
     return after_launch(ctx, "dense_norm_kernel");
 }
 
@@ -358,49 +418,6 @@ __global__ void gather_rows_f32_kernel(const float *__restrict__ x, const uint32
 int launch_gather_rows_f32(prism_cuda_ctx *ctx, const float *x, const uint32_t *idx, uint32_t n, uint32_t width, float *y) {
     launch_pdl(ctx, "gather_rows_f32_kernel", gather_rows_f32_kernel, n, 256, 0, x, idx, width, y);
     return after_launch(ctx, "gather_rows_f32_kernel");
-}
-
-// First index of the strictly greatest value; NaN never wins (the rule of the fp16 argmax).
-__global__ void __launch_bounds__(1024) argmax_f32_kernel(const float *__restrict__ logits, uint32_t n, uint32_t stride, uint32_t *__restrict__ out) {
-    pdl_launch_dependents();
-    pdl_wait();
-    __shared__ float sv[32];
-    __shared__ uint32_t si[32];
-    const float *lg = logits + (size_t)blockIdx.x * stride;
-    float bv = -INFINITY;
-    uint32_t bi = 0xFFFFFFFFu;
-    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
-        const float f = lg[i];
-        if (f > bv) {
-            bv = f;
-            bi = i;
-        }
-    }
-    auto take = [&](float ov, uint32_t oi) {
-        if (ov > bv || (ov == bv && oi < bi)) {
-            bv = ov;
-            bi = oi;
-        }
-    };
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, o);
-        const uint32_t oi = __shfl_xor_sync(0xFFFFFFFFu, bi, o);
-        take(ov, oi);
-    }
-    if ((threadIdx.x & 31) == 0) {
-        sv[threadIdx.x >> 5] = bv;
-        si[threadIdx.x >> 5] = bi;
-    }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        for (uint32_t w = 1; w < (blockDim.x >> 5); w++) take(sv[w], si[w]);
-        out[blockIdx.x] = bi == 0xFFFFFFFFu ? 0u : bi;
-    }
-}
-int launch_argmax_f32(prism_cuda_ctx *ctx, const float *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev) {
-    launch_pdl(ctx, "argmax_f32_kernel", argmax_f32_kernel, batch, 1024, 0, logits, n, stride, out_dev);
-    return after_launch(ctx, "argmax_f32_kernel");
 }
 
 __global__ void f32_to_f16_kernel(const float *__restrict__ x, uint32_t n, uint32_t stride, uint16_t *__restrict__ y, uint32_t y_stride) {

@@ -35,7 +35,7 @@ struct DenseLinear {
     bf16 *w = nullptr;
     uint32_t k_pad = 0, n_tiles = 0, n_segs = 0;
     DenseSeg seg[DENSE_MAX_SEGS];
-    size_t bytes() const { return (size_t)n_tiles * 128 * k_pad * 2; }
+    size_t bytes() const { return (size_t)((n_tiles + 1) / 2 * 2) * 128 * k_pad * 2; }  // whole pairs of row tiles
     uint64_t valid_rows() const {
         uint64_t r = 0;
         for (uint32_t s = 0; s < n_segs; s++) r += seg[s].rows;
@@ -181,7 +181,7 @@ int launch_dense_synth(prism_cuda_ctx *ctx, bf16 *dst, size_t n, uint64_t seed, 
 DenseEpi dense_epi(const DenseLinear &l, const DenseOut *outs);
 // Small batch (bf16, at most DENSE_GEMV_ROWS rows): mma.sync straight from the weight units, the input's norm folded in.
 constexpr uint32_t DENSE_GEMV_ROWS = 8;
-bool dense_gemv_ok(const DenseLinear &l, const DenseIn &in, uint32_t rows);
+bool dense_gemv_ok(const DenseIn &in, uint32_t rows);
 int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows);
 // 32-bit activations and fp32 products (the weights are exact in fp32): any number of rows, plain input
 int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const float *x, uint32_t pitch, const DenseOut *outs, uint32_t rows);
@@ -191,7 +191,6 @@ int launch_dense_gemm_tc5(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 
 int launch_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t y_pitch, uint32_t rows, bool act32);
 int launch_dense_embed(prism_cuda_ctx *ctx, const bf16 *table, uint32_t width, uint32_t vocab, const uint32_t *tokens, uint32_t rows, float *x);
 int launch_gather_rows_f32(prism_cuda_ctx *ctx, const float *x, const uint32_t *idx, uint32_t n, uint32_t width, float *y);
-int launch_argmax_f32(prism_cuda_ctx *ctx, const float *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev);
 int launch_f32_to_f16(prism_cuda_ctx *ctx, const float *x, uint32_t rows, uint32_t n, uint32_t stride, uint16_t *y, uint32_t y_stride);
 
 // lightning.cu
@@ -226,12 +225,12 @@ struct LatentArgs {
 // Normalises and rotates the rows of W_dkv h and appends them to the cache.
 int launch_latent_append(prism_cuda_ctx *ctx, const LatentArgs &a, const void *dkv, uint32_t pitch, const RowMap &rows, uint32_t n_rows, bool act32);
 // Rows against the cached latents themselves (W_uk folded into the query, W_uv applied to the weighted latent):
-// decode, short portions, and everything in 32-bit.  n_keys bounds the keys a row can see.
+// decode, short portions, and everything in 32-bit.  Appends the rows' latents (dkv) to the cache first.
 struct LatentRowsScratch { float *qa; float *part; float *ml; size_t rows_cap; uint32_t splits; };
 size_t latent_rows_scratch_floats(const LatentArgs &a, uint32_t splits, size_t *qa, size_t *part, size_t *ml);
 uint32_t latent_rows_splits(const LatentArgs &a, uint32_t max_seq);
-int launch_latent_rows(prism_cuda_ctx *ctx, const LatentArgs &a, const LatentRowsScratch &s, const void *q, uint32_t q_pitch, const void *gate,
-                       uint32_t gate_pitch, void *out, uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32);
+int launch_latent_rows(prism_cuda_ctx *ctx, const LatentArgs &a, const LatentRowsScratch &s, const void *q, uint32_t q_pitch, const void *dkv,
+                       uint32_t dkv_pitch, const void *gate, uint32_t gate_pitch, void *out, uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32);
 // Prompt portion of one sequence (bf16): keys and values expanded for positions [lo, pos0 + n_rows).
 bool latent_expand_ok(const LatentArgs &a);
 int launch_latent_gather(prism_cuda_ctx *ctx, const LatentArgs &a, int32_t slot, uint32_t lo, uint32_t n, bf16 *lat, uint32_t lat_pitch, bf16 *krot);

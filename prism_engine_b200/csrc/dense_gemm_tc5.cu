@@ -1,12 +1,14 @@
 // Dense bf16 GEMM on tcgen05 / TMEM with the segment epilogues of dense.cuh:
 //   y[t][n] = epilogue( sum_k x[t][k] * W[n][k] ),  fp32 accumulate.
 //
-// A persistent CTA computes tiles of 128 weight rows x NT rows of x.  One warp loads: the weights of a
+// A persistent CTA computes tiles of RT x 128 weight rows x NT rows of x (RT = 2 reads x once for two row tiles:
+// a 128-row tile needs more operand bytes per cycle than L2 delivers to all SMs).  One warp loads: the weights of a
 // 64-k stage are one contiguous 16 KB run (dense.cuh), fetched by a 1-D bulk copy straight into the
 // unswizzled core-matrix order of the A operand; the rows of x come through a tensor map with the
 // 128-byte swizzle of the B operand (rows past the end are filled with zeros).  One thread issues the
-// tcgen05.mma; four warps read the accumulators back, apply the epilogue of the tile's segment and store
-// -- two accumulator buffers in TMEM, so that an epilogue overlaps the products of the next tile.
+// tcgen05.mma; four warps per accumulator read it back, apply the epilogue of the tile's segment and store.
+// Two accumulators in TMEM: successive tiles alternate between them (RT = 1) or each row tile has its own
+// (RT = 2), so that an epilogue overlaps the loads and, for RT = 1, the products of the next tile.
 // Every mbarrier wait is bounded; one that gives up raises the context's device error word.
 #include <cuda.h>
 
@@ -17,12 +19,12 @@
 
 namespace prism {
 
-constexpr int DG_THREADS = 192;               // loader warp, MMA warp, four epilogue warps
-constexpr int DG_A_BYTES = 128 * 64 * 2;      // weights of a stage
-template <int NT>
+constexpr int DG_A_BYTES = 128 * 64 * 2;      // weights of a stage and row tile
+template <int NT, int RT>
 struct DgCfg {
-    static constexpr int B_BYTES = NT * 128;
-    static constexpr int STAGE = DG_A_BYTES + B_BYTES;
+    static constexpr int THREADS = 64 + 128 * RT;  // loader warp, MMA warp, four epilogue warps per row tile
+    static constexpr int A_BYTES = RT * DG_A_BYTES, B_BYTES = NT * 128;
+    static constexpr int STAGE = A_BYTES + B_BYTES;
     static constexpr int S = (200 * 1024 / STAGE) < 8 ? (200 * 1024 / STAGE) : 8;
     static constexpr int TMEM_COLS = 2 * NT < 32 ? 32 : 2 * NT;
     static constexpr int BAR_OFF = S * STAGE;
@@ -32,7 +34,7 @@ struct DgCfg {
 struct DgArgs {
     const uint8_t *w;
     uint32_t kb;              // 64-k stages per row
-    uint32_t n_rt, n_tt, rt_group;  // row tiles, token tiles, row tiles per group of the walk
+    uint32_t n_rt, n_tt, rt_group;  // row tiles (of RT x 128), token tiles, row tiles per group of the walk
     uint32_t rows;            // rows of x
     unsigned int *err;
     DenseEpi epi;
@@ -65,9 +67,9 @@ __device__ __forceinline__ void dg_item(const DgArgs &a, uint32_t w, uint32_t &r
     tt = rem / gr;
 }
 
-template <int NT>
-__global__ void __launch_bounds__(DG_THREADS, 1) dense_gemm_tc5_kernel(const DgArgs a, const __grid_constant__ CUtensorMap xmap) {
-    using C = DgCfg<NT>;
+template <int NT, int RT>
+__global__ void __launch_bounds__(DgCfg<NT, RT>::THREADS, 1) dense_gemm_tc5_kernel(const DgArgs a, const __grid_constant__ CUtensorMap xmap) {
+    using C = DgCfg<NT, RT>;
     extern __shared__ uint8_t dg_smem_raw[];
     uint8_t *smem = dg_smem_raw + (1024 - ((uint32_t)__cvta_generic_to_shared(dg_smem_raw) & 1023u)) % 1024;
     const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
@@ -97,13 +99,15 @@ __global__ void __launch_bounds__(DG_THREADS, 1) dense_gemm_tc5_kernel(const DgA
             for (uint32_t w = blockIdx.x; w < n_items; w += gridDim.x) {
                 uint32_t rt, tt;
                 dg_item(a, w, rt, tt);
-                const uint8_t *wsrc = a.w + (size_t)rt * a.kb * DG_A_BYTES;
+                const uint8_t *wsrc = a.w + (size_t)rt * RT * a.kb * DG_A_BYTES;
                 for (uint32_t k = 0; k < a.kb; k++, n++) {
                     const uint32_t s = n % C::S, ph = (n / C::S) & 1, dst = base + s * C::STAGE;
                     t5::mbar_wait_bounded(b_empty + 8 * s, ph ^ 1, err_flag);
                     t5::mbar_arrive_expect_tx(b_full + 8 * s, C::STAGE);
-                    t5::bulk_g2s(dst, wsrc + (size_t)k * DG_A_BYTES, DG_A_BYTES, b_full + 8 * s);
-                    tma_2d(dst + DG_A_BYTES, &xmap, (int32_t)(k * 64), (int32_t)(tt * NT), b_full + 8 * s);
+#pragma unroll
+                    for (int r = 0; r < RT; r++)
+                        t5::bulk_g2s(dst + r * DG_A_BYTES, wsrc + ((size_t)r * a.kb + k) * DG_A_BYTES, DG_A_BYTES, b_full + 8 * s);
+                    tma_2d(dst + C::A_BYTES, &xmap, (int32_t)(k * 64), (int32_t)(tt * NT), b_full + 8 * s);
                 }
             }
             // every copy in flight lands before the CTA leaves (a stage's last use is committed to its empty barrier)
@@ -117,34 +121,48 @@ __global__ void __launch_bounds__(DG_THREADS, 1) dense_gemm_tc5_kernel(const DgA
             const uint32_t idesc = t5::idesc_f16(128, NT) | (1u << 7) | (1u << 10);  // A and B bf16
             uint32_t n = 0, ti = 0;
             for (uint32_t w = blockIdx.x; w < n_items; w += gridDim.x, ti++) {
-                const uint32_t b = ti & 1, d = tmem + b * NT;
-                t5::mbar_wait_bounded(b_dempty + 8 * b, ((ti >> 1) & 1) ^ 1, err_flag);
-                t5::fence_after();
+                if (RT == 1) {
+                    t5::mbar_wait_bounded(b_dempty + 8 * (ti & 1), ((ti >> 1) & 1) ^ 1, err_flag);
+                    t5::fence_after();
+                }
                 for (uint32_t k = 0; k < a.kb; k++, n++) {
-                    const uint32_t s = n % C::S, ph = (n / C::S) & 1, sa = base + s * C::STAGE, sb = sa + DG_A_BYTES;
+                    const uint32_t s = n % C::S, ph = (n / C::S) & 1, sa = base + s * C::STAGE, sb = sa + C::A_BYTES;
                     t5::mbar_wait_bounded(b_full + 8 * s, ph, err_flag);
                     t5::fence_after();
 #pragma unroll
-                    for (int j = 0; j < 4; j++)  // 16 k each: two k/8 slabs of 2 KB in A, 32 bytes inside the swizzled rows of B
-                        mma_ss(d, t5::smem_desc(sa + j * 4096, 2048, 128), desc_sw128(sb + j * 32), idesc, (k | j) != 0);
+                    for (int r = 0; r < RT; r++) {
+                        if (RT == 2 && k == 0) {
+                            t5::mbar_wait_bounded(b_dempty + 8 * r, (ti & 1) ^ 1, err_flag);
+                            t5::fence_after();
+                        }
+                        const uint32_t d = tmem + (RT == 1 ? ti & 1 : r) * NT;
+#pragma unroll
+                        for (int j = 0; j < 4; j++)  // 16 k each: two k/8 slabs of 2 KB in A, 32 bytes inside the swizzled rows of B
+                            mma_ss(d, t5::smem_desc(sa + r * DG_A_BYTES + j * 4096, 2048, 128), desc_sw128(sb + j * 32), idesc, (k | j) != 0);
+                    }
                     t5::commit(b_empty + 8 * s);
                 }
-                t5::commit(b_dfull + 8 * b);
+                if (RT == 1) {
+                    t5::commit(b_dfull + 8 * (ti & 1));
+                } else {
+                    t5::commit(b_dfull);
+                    t5::commit(b_dfull + 8);
+                }
             }
         }
     } else {
-        const uint32_t q = warp & 3;  // the TMEM lanes a warp may read
+        const uint32_t q = warp & 3, er = (warp - 2) >> 2;  // the TMEM lanes a warp may read; its row tile
         uint32_t ti = 0;
         for (uint32_t w = blockIdx.x; w < n_items; w += gridDim.x, ti++) {
             uint32_t rt, tt;
             dg_item(a, w, rt, tt);
-            const uint32_t b = ti & 1;
+            const uint32_t b = RT == 1 ? ti & 1 : er, ph = RT == 1 ? (ti >> 1) & 1 : ti & 1, row0 = (rt * RT + er) * 128;
             uint32_t sg = 0;
-            while (sg + 1 < a.epi.n && rt * 128 >= a.epi.s[sg + 1].row0) sg++;
+            while (sg + 1 < a.epi.n && row0 >= a.epi.s[sg + 1].row0) sg++;
             const DenseEpiSeg &seg = a.epi.s[sg];
-            const uint32_t row = rt * 128 + q * 32 + lane - seg.row0;
+            const uint32_t row = row0 + q * 32 + lane - seg.row0;
             const bool row_ok = row < seg.rows;
-            t5::mbar_wait_warp(b_dfull + 8 * b, (ti >> 1) & 1, err_flag);
+            t5::mbar_wait_warp(b_dfull + 8 * b, ph, err_flag);
             t5::fence_after();
 #pragma unroll 1
             for (int g = 0; g < NT / 16; g++) {
@@ -185,12 +203,12 @@ static TensorMapEncode tensor_map_encode() {
     return fn;
 }
 
-template <int NT>
+template <int NT, int RT>
 static int launch_dg(prism_cuda_ctx *ctx, const DenseLinear &l, DgArgs &a, const bf16 *x, uint32_t pitch) {
-    using C = DgCfg<NT>;
+    using C = DgCfg<NT, RT>;
     static bool configured[PRISM_MAX_DEVICES] = {false};
     if (!configured[ctx->device]) {
-        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemm_tc5_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemm_tc5_kernel<NT, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
         configured[ctx->device] = true;
     }
     TensorMapEncode enc = tensor_map_encode();
@@ -202,11 +220,12 @@ static int launch_dg(prism_cuda_ctx *ctx, const DenseLinear &l, DgArgs &a, const
                             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (rc != CUDA_SUCCESS) return fail(ctx, PRISM_E_CUDA, "cuTensorMapEncodeTiled failed: " + std::to_string((int)rc));
+    a.n_rt = (l.n_tiles + RT - 1) / RT;
     a.n_tt = (a.rows + NT - 1) / NT;
     const uint32_t G = (uint32_t)ctx->sm_count;
     a.rt_group = std::min(a.n_rt, std::max(1u, (G + a.n_tt - 1) / a.n_tt));
     const uint32_t grid = std::min(G, a.n_rt * a.n_tt);
-    launch_pdl(ctx, "dense_gemm_tc5_kernel", dense_gemm_tc5_kernel<NT>, dim3(grid), dim3(DG_THREADS), C::SMEM, a, map);
+    launch_pdl(ctx, "dense_gemm_tc5_kernel", dense_gemm_tc5_kernel<NT, RT>, dim3(grid), dim3(C::THREADS), C::SMEM, a, map);
     return after_launch(ctx, "dense_gemm_tc5_kernel");
 }
 
@@ -216,16 +235,35 @@ int launch_dense_gemm_tc5(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 
     DgArgs a{};
     a.w = reinterpret_cast<const uint8_t *>(l.w);
     a.kb = l.k_pad / 64;
-    a.n_rt = l.n_tiles;
     a.rows = rows;
     a.err = ctx->dev_err;
     a.epi = dense_epi(l, outs);
-    // token tile: as small as the batch allows, and small enough that the tiles cover the GPU
-    if (rows <= 16) return launch_dg<16>(ctx, l, a, x, pitch);
-    if (rows <= 32) return launch_dg<32>(ctx, l, a, x, pitch);
-    if (rows <= 64 || a.n_rt * ((rows + 127) / 128) < (uint32_t)ctx->sm_count) return launch_dg<64>(ctx, l, a, x, pitch);
-    if (rows <= 128 || a.n_rt * ((rows + 255) / 256) < (uint32_t)ctx->sm_count) return launch_dg<128>(ctx, l, a, x, pitch);
-    return launch_dg<256>(ctx, l, a, x, pitch);
+    // Tile shape with the least estimated time: waves x cycles of a 64-k stage, which the tensor core bounds by
+    // 2 NT RT and the loads by what L2 delivers to the CTAs at work (about 6000 bytes per cycle in all).
+    struct Shape { uint32_t nt, rt; };
+    static const Shape shapes[] = {{256, 2}, {128, 2}, {64, 2}, {256, 1}, {128, 1}, {64, 1}, {32, 1}, {16, 1}};
+    const uint32_t G = (uint32_t)ctx->sm_count;
+    Shape best = shapes[0];
+    double best_t = 1e30;
+    for (const Shape &s : shapes) {
+        const uint64_t items = (uint64_t)((l.n_tiles + s.rt - 1) / s.rt) * ((rows + s.nt - 1) / s.nt);
+        const double bytes = s.rt * DG_A_BYTES + s.nt * 128.0, act = (double)std::min<uint64_t>(items, G);
+        const double t = (double)((items + G - 1) / G) * std::max({2.0 * s.nt * s.rt, bytes * act / 6000.0, bytes / 100.0});
+        if (t < best_t * 0.999) {
+            best_t = t;
+            best = s;
+        }
+    }
+    switch (best.nt * 4 + best.rt) {
+    case 256 * 4 + 2: return launch_dg<256, 2>(ctx, l, a, x, pitch);
+    case 128 * 4 + 2: return launch_dg<128, 2>(ctx, l, a, x, pitch);
+    case 64 * 4 + 2: return launch_dg<64, 2>(ctx, l, a, x, pitch);
+    case 256 * 4 + 1: return launch_dg<256, 1>(ctx, l, a, x, pitch);
+    case 128 * 4 + 1: return launch_dg<128, 1>(ctx, l, a, x, pitch);
+    case 64 * 4 + 1: return launch_dg<64, 1>(ctx, l, a, x, pitch);
+    case 32 * 4 + 1: return launch_dg<32, 1>(ctx, l, a, x, pitch);
+    default: return launch_dg<16, 1>(ctx, l, a, x, pitch);
+    }
 }
 
 }  // namespace prism

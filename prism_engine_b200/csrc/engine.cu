@@ -771,9 +771,9 @@ int prism_cuda_engine_synth_weights(prism_cuda_engine *e, uint64_t seed, float s
 
 int prism_cuda_engine_reset(prism_cuda_engine *e, uint32_t batch) {
     if (!e) return PRISM_E_NULL;
-    if (batch == 0 || batch > e->cfg.max_batch) return fail(e->ctx, PRISM_E_ARG, "batch outside [1, max_batch]");
+    if ((batch == 0 && !e->lm) || batch > e->cfg.max_batch) return fail(e->ctx, PRISM_E_ARG, "batch outside [1, max_batch]");
     PRISM_CUDA_TRY(e->ctx, cudaSetDevice(e->ctx->device));
-    e->batch = batch;
+    e->batch = batch ? batch : 1;  // 0 (layered models): every sequence slot is given back
     e->pos = 0;
     release_pages(e);  // a reset returns every page to the pool
     if (e->lm) PRISM_TRY(layered_reset(e, batch));

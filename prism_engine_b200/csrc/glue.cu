@@ -196,8 +196,8 @@ int launch_softmax(prism_cuda_ctx *ctx, const uint16_t *in, uint16_t *out, uint3
 // argmax (engine_impl.rs:1448-1459): first index holding the strictly greatest
 // value; NaN never wins; an all-NaN/-inf vector gives 0.  A cluster of ARGMAX_CTAS
 // blocks per sequence: each scans a slice with 16-byte loads, rank 0 merges the
-// slices' winners through distributed shared memory.  Rows of `logits` are
-// `stride` apart and 16-byte aligned.
+// slices' winners through distributed shared memory.  Rows of `logits` (fp16, or fp32 for the
+// layered models) are `stride` apart and 16-byte aligned.
 constexpr int ARGMAX_CTAS = 8;
 constexpr int ARGMAX_THREADS = 512;
 __device__ __forceinline__ void argmax_take(float &bv, uint32_t &bi, float ov, uint32_t oi) {
@@ -206,8 +206,12 @@ __device__ __forceinline__ void argmax_take(float &bv, uint32_t &bi, float ov, u
         bi = oi;
     }
 }
-__global__ void __launch_bounds__(ARGMAX_THREADS) argmax_kernel(const uint16_t *__restrict__ logits, uint32_t n,
+__device__ __forceinline__ float logit_value(uint16_t v) { return h2f(v); }
+__device__ __forceinline__ float logit_value(float v) { return v; }
+template <typename T>
+__global__ void __launch_bounds__(ARGMAX_THREADS) argmax_kernel(const T *__restrict__ logits, uint32_t n,
                                                                 uint32_t stride, uint32_t *__restrict__ out) {
+    constexpr uint32_t V = 16 / sizeof(T);  // values of a 16-byte load
     pdl_launch_dependents();
     pdl_wait();
     cg::cluster_group cluster = cg::this_cluster();
@@ -217,20 +221,20 @@ __global__ void __launch_bounds__(ARGMAX_THREADS) argmax_kernel(const uint16_t *
     __shared__ float win_v;
     __shared__ uint32_t win_i;
     const uint32_t seq = blockIdx.x / R;
-    const uint16_t *lg = logits + (size_t)seq * stride;
-    // slice of this block, in groups of 8 values
-    const uint32_t groups = (n + 7) / 8, per = (groups + R - 1) / R;
+    const T *lg = logits + (size_t)seq * stride;
+    // slice of this block, in groups of V values
+    const uint32_t groups = (n + V - 1) / V, per = (groups + R - 1) / R;
     const uint32_t g0 = min(groups, rank * per), g1 = min(groups, g0 + per);
     float bv = -INFINITY;
     uint32_t bi = 0xFFFFFFFFu;
     for (uint32_t g = g0 + threadIdx.x; g < g1; g += ARGMAX_THREADS) {
-        const uint32_t i0 = g * 8;
-        if (i0 + 8 <= n) {
+        const uint32_t i0 = g * V;
+        if (i0 + V <= n) {
             const uint4 v = *reinterpret_cast<const uint4 *>(lg + i0);
-            const uint16_t *e = reinterpret_cast<const uint16_t *>(&v);
+            const T *e = reinterpret_cast<const T *>(&v);
 #pragma unroll
-            for (int k = 0; k < 8; k++) {
-                const float f = h2f(e[k]);
+            for (uint32_t k = 0; k < V; k++) {
+                const float f = logit_value(e[k]);
                 if (f > bv) {  // ascending index per thread: keeps the first maximum
                     bv = f;
                     bi = i0 + k;
@@ -238,7 +242,7 @@ __global__ void __launch_bounds__(ARGMAX_THREADS) argmax_kernel(const uint16_t *
             }
         } else {
             for (uint32_t i = i0; i < n; i++) {
-                const float f = h2f(lg[i]);
+                const float f = logit_value(lg[i]);
                 if (f > bv) {
                     bv = f;
                     bi = i;
@@ -272,13 +276,19 @@ __global__ void __launch_bounds__(ARGMAX_THREADS) argmax_kernel(const uint16_t *
     }
     cluster.sync();  // peers keep their shared memory alive until rank 0 has read it
 }
-int launch_argmax(prism_cuda_ctx *ctx, const uint16_t *logits, uint32_t n, uint32_t stride, uint32_t batch,
-                  uint32_t *out_dev) {
-    if ((reinterpret_cast<uintptr_t>(logits) & 15) || (batch > 1 && stride % 8))
+template <typename T>
+static int run_argmax(prism_cuda_ctx *ctx, const T *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev) {
+    if ((reinterpret_cast<uintptr_t>(logits) & 15) || (batch > 1 && stride % (16 / sizeof(T))))
         return fail(ctx, PRISM_E_ARG, "argmax: rows must be 16-byte aligned");
-    launch_cluster_pdl(ctx, argmax_kernel, dim3(ARGMAX_CTAS * batch), dim3(ARGMAX_THREADS), 0, ARGMAX_CTAS, logits, n,
+    launch_cluster_pdl(ctx, argmax_kernel<T>, dim3(ARGMAX_CTAS * batch), dim3(ARGMAX_THREADS), 0, ARGMAX_CTAS, logits, n,
                        stride, out_dev);
     return after_launch(ctx, "argmax_kernel");
+}
+int launch_argmax(prism_cuda_ctx *ctx, const uint16_t *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev) {
+    return run_argmax(ctx, logits, n, stride, batch, out_dev);
+}
+int launch_argmax(prism_cuda_ctx *ctx, const float *logits, uint32_t n, uint32_t stride, uint32_t batch, uint32_t *out_dev) {
+    return run_argmax(ctx, logits, n, stride, batch, out_dev);
 }
 
 // KV append.  fp16 mode stores the GEMV outputs verbatim at [slot][kvd].

@@ -30,12 +30,9 @@ __device__ __forceinline__ void rotate_pair(const LatentArgs &a, int32_t pos, ui
 }
 
 // ---- append ------------------------------------------------------------------------------------------
+// By a whole block: row r of W_dkv h, its latent normed, its rotated part turned, into the cache.  sh: 32 floats.
 template <typename TA>
-__global__ void __launch_bounds__(128) latent_append_kernel(const LatentArgs a, const TA *__restrict__ dkv, uint32_t pitch, const RowMap rows) {
-    pdl_launch_dependents();
-    pdl_wait();
-    __shared__ float sh[32];
-    const uint32_t r = blockIdx.x;
+__device__ __forceinline__ void append_row(const LatentArgs &a, const TA *__restrict__ dkv, uint32_t pitch, const RowMap &rows, uint32_t r, float *sh) {
     const int32_t pos = rows.pos_of(r);
     const TA *x = dkv + (size_t)r * pitch;
     TA *y = reinterpret_cast<TA *>(a.cache.rows) + cache_row(a.cache, rows.slot_of(r), pos);
@@ -57,6 +54,13 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const LatentArgs a, 
     }
     for (uint32_t i = 2 * a.rot_pairs + threadIdx.x; i < a.rot_dim; i += blockDim.x) y[i] = x[i];
 }
+template <typename TA>
+__global__ void __launch_bounds__(128) latent_append_kernel(const LatentArgs a, const TA *__restrict__ dkv, uint32_t pitch, const RowMap rows) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float sh[32];
+    append_row(a, dkv, pitch, rows, blockIdx.x, sh);
+}
 int launch_latent_append(prism_cuda_ctx *ctx, const LatentArgs &a, const void *dkv, uint32_t pitch, const RowMap &rows, uint32_t n_rows, bool act32) {
     if (act32) launch_pdl(ctx, "latent_append_kernel", latent_append_kernel<float>, n_rows, 128, 0, a, (const float *)dkv, pitch, rows);
     else launch_pdl(ctx, "latent_append_kernel", latent_append_kernel<bf16>, n_rows, 128, 0, a, (const bf16 *)dkv, pitch, rows);
@@ -64,23 +68,34 @@ int launch_latent_append(prism_cuda_ctx *ctx, const LatentArgs &a, const void *d
 }
 
 // ---- rows: query against the latents -------------------------------------------------------------------
-// qa[r][h] = [W_uk[h]^T q_unrotated | rotated q | zeros], fp32.  Grid: (head, 128 latent columns, 4 rows).
-constexpr int LQ_ROWS = 4;
+// qa[r][h] = [W_uk[h]^T q_unrotated | rotated q | zeros], fp32.  Grid: (head, 128 latent columns, 4 rows).  One
+// more block along x appends the rows to the cache meanwhile.
+constexpr int LQ_ROWS = 4, LQ_PRE = 8;  // weight units a thread requests before the dependency wait
 template <typename TA>
-__global__ void __launch_bounds__(256) latent_query_kernel(const LatentArgs a, const TA *__restrict__ q, uint32_t q_pitch, const RowMap rows,
-                                                           uint32_t n_rows, float *__restrict__ qa) {
+__global__ void __launch_bounds__(256) latent_query_kernel(const LatentArgs a, const TA *__restrict__ q, uint32_t q_pitch,
+                                                           const TA *__restrict__ dkv, uint32_t dkv_pitch, const RowMap rows, uint32_t n_rows,
+                                                           float *__restrict__ qa) {
     __shared__ float red[16][LQ_ROWS][130];
     pdl_launch_dependents();
     const uint32_t h = blockIdx.x, c8 = threadIdx.x & 15, dg = threadIdx.x >> 4, col = blockIdx.y * 128 + c8 * 8, r0 = blockIdx.z * LQ_ROWS;
     const uint32_t hq = a.dim + a.rot_dim, L = a.cache.pitch;
+    if (h == a.heads) {
+        pdl_wait();
+        if (blockIdx.y == 0)
+            for (uint32_t r = r0; r < min(n_rows, r0 + LQ_ROWS); r++) append_row(a, dkv, dkv_pitch, rows, r, &red[0][0][0]);
+        return;
+    }
     const bool on = col < a.uk_pitch;
     const bf16 *wk = a.uk + (size_t)h * a.dim * a.uk_pitch + col;
+    uint4 pre[LQ_PRE];
+#pragma unroll
+    for (int i = 0; i < LQ_PRE; i++) {
+        pre[i] = make_uint4(0, 0, 0, 0);
+        if (on && dg + 16 * i < a.dim) pre[i] = __ldg(reinterpret_cast<const uint4 *>(wk + (size_t)(dg + 16 * i) * a.uk_pitch));
+    }
     pdl_wait();
     float acc[LQ_ROWS][8] = {};
-#pragma unroll 4
-    for (uint32_t d = dg; d < a.dim; d += 16) {
-        uint4 w4 = make_uint4(0, 0, 0, 0);
-        if (on) w4 = __ldg(reinterpret_cast<const uint4 *>(wk + (size_t)d * a.uk_pitch));
+    auto add = [&](uint32_t d, const uint4 &w4) {
         const bf16 *w = reinterpret_cast<const bf16 *>(&w4);
 #pragma unroll
         for (int r = 0; r < LQ_ROWS; r++) {
@@ -88,7 +103,12 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const LatentArgs a, c
 #pragma unroll
             for (int i = 0; i < 8; i++) acc[r][i] = fmaf(__bfloat162float(w[i]), x, acc[r][i]);
         }
-    }
+    };
+#pragma unroll
+    for (int i = 0; i < LQ_PRE; i++)
+        if (dg + 16 * i < a.dim) add(dg + 16 * i, pre[i]);
+    for (uint32_t d = dg + 16 * LQ_PRE; d < a.dim; d += 16)
+        add(d, on ? __ldg(reinterpret_cast<const uint4 *>(wk + (size_t)d * a.uk_pitch)) : make_uint4(0, 0, 0, 0));
 #pragma unroll
     for (int r = 0; r < LQ_ROWS; r++)
 #pragma unroll
@@ -272,39 +292,60 @@ __global__ void __launch_bounds__(128) latent_rows_mma_kernel(const LatentArgs a
 }
 
 // Merges a head's splits, applies W_uv and the gate.  Grid: (head, 32 value columns, row).
+constexpr int LO_PRE = 2;  // 256-column pieces of W_uv rows requested before the dependency wait
 template <typename TA>
 __global__ void __launch_bounds__(128) latent_out_kernel(const LatentArgs a, const LatentPart o, const RowMap rows, const TA *__restrict__ gate,
                                                          uint32_t gate_pitch, TA *__restrict__ out, uint32_t out_pitch) {
-    extern __shared__ float los[];  // [uk_pitch] weighted latent, then [splits] weights
+    extern __shared__ float los[];  // [uk_pitch] weighted latent, then maxima and sums of the splits
     pdl_launch_dependents();
-    pdl_wait();
     const uint32_t h = blockIdx.x, v0 = blockIdx.y * 32, r = blockIdx.z, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const bf16 *wv = a.uv + ((size_t)h * a.vdim + v0 + warp) * a.uk_pitch + lane * 8;  // this warp: value columns v0 + warp + 4 i
+    uint4 pre[8][LO_PRE];
+#pragma unroll
+    for (int i = 0; i < 8; i++)
+#pragma unroll
+        for (int k = 0; k < LO_PRE; k++) {
+            pre[i][k] = make_uint4(0, 0, 0, 0);
+            if (v0 + warp + 4 * i < a.vdim && lane * 8 + 256 * k < a.uk_pitch)
+                pre[i][k] = __ldg(reinterpret_cast<const uint4 *>(wv + (size_t)4 * i * a.uk_pitch + 256 * k));
+        }
+    pdl_wait();
     const int32_t pos = rows.pos_of(r);
     const uint32_t n = (uint32_t)(pos + 1 - first_key(a, pos) + LR_KT - 1) / LR_KT;
     const float *ml = o.ml + ((size_t)r * a.heads + h) * o.splits * 2, *part = o.part + ((size_t)r * a.heads + h) * o.splits * a.uk_pitch;
-    float *ol = los, *ws = los + a.uk_pitch;
-    float m = -INFINITY, l = 0.0f;
-    for (uint32_t s = 0; s < n; s++) m = fmaxf(m, ml[2 * s]);
-    for (uint32_t s = 0; s < n; s++) l += ml[2 * s + 1] * expf(ml[2 * s] - m);
-    const float inv = 1.0f / l;
-    for (uint32_t s = threadIdx.x; s < n; s += blockDim.x) ws[s] = expf(ml[2 * s] - m) * inv;
+    float *ol = los, *mls = los + a.uk_pitch;
+    for (uint32_t i = threadIdx.x; i < 2 * n; i += blockDim.x) mls[i] = ml[i];
     __syncthreads();
+    float m = -INFINITY, l = 0.0f;
+    for (uint32_t s = 0; s < n; s++) m = fmaxf(m, mls[2 * s]);
+    for (uint32_t s = 0; s < n; s++) l = fmaf(mls[2 * s + 1], expf(mls[2 * s] - m), l);
+    const float inv = 1.0f / l;
     for (uint32_t j = threadIdx.x; j < a.uk_pitch; j += blockDim.x) {
         float x = 0.0f;
-        if (j < a.kv_rank)
-            for (uint32_t s = 0; s < n; s++) x = fmaf(ws[s], part[(size_t)s * a.uk_pitch + j], x);
+        if (j < a.kv_rank) {
+#pragma unroll 4
+            for (uint32_t s = 0; s < n; s++) x = fmaf(expf(mls[2 * s] - m) * inv, part[(size_t)s * a.uk_pitch + j], x);
+        }
         ol[j] = x;
     }
     __syncthreads();
-    for (uint32_t v = v0 + warp; v < min(a.vdim, v0 + 32); v += 4) {
-        const bf16 *w = a.uv + ((size_t)h * a.vdim + v) * a.uk_pitch;
+    auto dot = [&](const uint4 &w4, uint32_t j) {
+        const bf16 *e = reinterpret_cast<const bf16 *>(&w4);
         float s = 0.0f;
-        for (uint32_t j = lane * 8; j < a.uk_pitch; j += 256) {
-            const uint4 w4 = __ldg(reinterpret_cast<const uint4 *>(w + j));
-            const bf16 *e = reinterpret_cast<const bf16 *>(&w4);
 #pragma unroll
-            for (int i = 0; i < 8; i++) s = fmaf(__bfloat162float(e[i]), ol[j + i], s);
-        }
+        for (int i = 0; i < 8; i++) s = fmaf(__bfloat162float(e[i]), ol[j + i], s);
+        return s;
+    };
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+        const uint32_t v = v0 + warp + 4 * i;
+        if (v >= a.vdim) break;
+        float s = 0.0f;
+#pragma unroll
+        for (int k = 0; k < LO_PRE; k++)
+            if (lane * 8 + 256 * k < a.uk_pitch) s += dot(pre[i][k], lane * 8 + 256 * k);
+        for (uint32_t j = lane * 8 + 256 * LO_PRE; j < a.uk_pitch; j += 256)
+            s += dot(__ldg(reinterpret_cast<const uint4 *>(a.uv + ((size_t)h * a.vdim + v) * a.uk_pitch + j)), j);
         s = warp_sum_f(s);
         if (lane == 0) {
             const uint32_t c = h * a.vdim + v;
@@ -325,21 +366,21 @@ size_t latent_rows_scratch_floats(const LatentArgs &a, uint32_t splits, size_t *
 }
 constexpr size_t LR_SMEM_MAX = 200 * 1024;
 
-int launch_latent_rows(prism_cuda_ctx *ctx, const LatentArgs &a, const LatentRowsScratch &s, const void *q, uint32_t q_pitch, const void *gate,
-                       uint32_t gate_pitch, void *out, uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32) {
+int launch_latent_rows(prism_cuda_ctx *ctx, const LatentArgs &a, const LatentRowsScratch &s, const void *q, uint32_t q_pitch, const void *dkv,
+                       uint32_t dkv_pitch, const void *gate, uint32_t gate_pitch, void *out, uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32) {
     const LatentPart p{s.part, s.ml, s.splits};
-    const dim3 gq(a.heads, (a.uk_pitch + 127) / 128, (n_rows + LQ_ROWS - 1) / LQ_ROWS), gout(a.heads, (a.vdim + 31) / 32, n_rows);
-    const size_t osm = ((size_t)a.uk_pitch + s.splits) * 4;
+    const dim3 gq(a.heads + 1, (a.uk_pitch + 127) / 128, (n_rows + LQ_ROWS - 1) / LQ_ROWS), gout(a.heads, (a.vdim + 31) / 32, n_rows);
+    const size_t osm = ((size_t)a.uk_pitch + 2 * s.splits) * 4;
     if (osm > 48 * 1024 || n_rows > s.rows_cap) return fail(ctx, PRISM_E_ARG, "latent attention: sizes beyond the kernel's scratch");
     if (act32) {
-        launch_pdl(ctx, "latent_query_kernel", latent_query_kernel<float>, gq, 256, 0, a, (const float *)q, q_pitch, rows, n_rows, s.qa);
+        launch_pdl(ctx, "latent_query_kernel", latent_query_kernel<float>, gq, 256, 0, a, (const float *)q, q_pitch, (const float *)dkv, dkv_pitch, rows, n_rows, s.qa);
         PRISM_TRY(after_launch(ctx, "latent_query_kernel"));
         launch_pdl(ctx, "latent_rows_kernel", latent_rows_kernel<float>, dim3(s.splits, a.heads, n_rows), 128, 0, a, (const float *)s.qa, rows, p);
         PRISM_TRY(after_launch(ctx, "latent_rows_kernel"));
         launch_pdl(ctx, "latent_out_kernel", latent_out_kernel<float>, gout, 128, osm, a, p, rows, (const float *)gate, gate_pitch, (float *)out, out_pitch);
         return after_launch(ctx, "latent_out_kernel");
     }
-    launch_pdl(ctx, "latent_query_kernel", latent_query_kernel<bf16>, gq, 256, 0, a, (const bf16 *)q, q_pitch, rows, n_rows, s.qa);
+    launch_pdl(ctx, "latent_query_kernel", latent_query_kernel<bf16>, gq, 256, 0, a, (const bf16 *)q, q_pitch, (const bf16 *)dkv, dkv_pitch, rows, n_rows, s.qa);
     PRISM_TRY(after_launch(ctx, "latent_query_kernel"));
     const size_t msm = (size_t)(LR_KT + 32) * (a.cache.pitch + 8) * 2;
     if (msm <= LR_SMEM_MAX) {

@@ -267,13 +267,18 @@ static int linear(prism_cuda_engine *e, const DenseLinear &l, const DenseIn &in,
                   uint32_t normed_pitch) {
     prism_cuda_ctx *ctx = e->ctx;
     LayeredModel *m = e->lm;
-    if (!m->act32 && ctx->fuse && dense_gemv_ok(l, in, rows)) return launch_dense_gemv(ctx, l, in, outs, rows);
+    if (!m->act32 && ctx->fuse && dense_gemv_ok(in, rows)) return launch_dense_gemv(ctx, l, in, outs, rows);
     const void *x = in.x;
     uint32_t pitch = in.pitch;
     if (in.norm_w) {
         PRISM_TRY(launch_dense_norm(ctx, in, normed, normed_pitch, rows, m->act32));
         x = normed;
         pitch = normed_pitch;
+        if (!m->act32 && ctx->fuse && rows <= DENSE_GEMV_ROWS) {
+            DenseIn plain{};
+            plain.x = x; plain.pitch = pitch;
+            return launch_dense_gemv(ctx, l, plain, outs, rows);
+        }
     }
     if (m->act32) return launch_dense_f32(ctx, l, (const float *)x, pitch, outs, rows);
     return launch_dense_gemm_tc5(ctx, l, (const bf16 *)x, pitch, outs, rows);
@@ -318,10 +323,10 @@ static int mix_latent(prism_cuda_engine *e, LayeredLayer &ly, const RowMap &rows
     qi.x = dq; qi.pitch = m->proj_pitch; qi.norm_w = ly.dq_norm; qi.n_norm = ly.c.q_rank; qi.eps = m->c.norm_eps;
     const DenseOut qo{m->q, m->q_pitch, ST_ACT};
     PRISM_TRY(linear(e, ly.uq, qi, &qo, n, m->cq, m->cq_pitch));
-    PRISM_TRY(launch_latent_append(ctx, la, dkv, m->proj_pitch, rows, n, m->act32));
     if (seq && n > DENSE_GEMV_ROWS && ly.ukv.w) {
         const uint32_t pos0 = (uint32_t)rows.pos0, lo = la.window && pos0 + 1 > la.window ? pos0 + 1 - la.window : 0, nk = pos0 + n - lo;
         const uint32_t kv_pitch = ly.ukv.n_tiles * 128, v0 = ly.ukv.seg[1].row0;
+        PRISM_TRY(launch_latent_append(ctx, la, dkv, m->proj_pitch, rows, n, false));
         PRISM_TRY(grow_bf16(e, m->ex_lat, m->ex_lat_n, (size_t)nk * ly.ukv.k_pad));
         PRISM_TRY(grow_bf16(e, m->ex_krot, m->ex_krot_n, (size_t)nk * la.rot_dim + 8));
         PRISM_TRY(grow_bf16(e, m->ex_kv, m->ex_kv_n, (size_t)nk * kv_pitch));
@@ -342,7 +347,8 @@ static int mix_latent(prism_cuda_engine *e, LayeredLayer &ly, const RowMap &rows
         } else {
             sub.pos0 += (int32_t)r;
         }
-        PRISM_TRY(launch_latent_rows(ctx, la, s, at(m, m->q, (size_t)r * m->q_pitch), m->q_pitch, at(m, gate, (size_t)r * m->proj_pitch), m->proj_pitch,
+        PRISM_TRY(launch_latent_rows(ctx, la, s, at(m, m->q, (size_t)r * m->q_pitch), m->q_pitch, at(m, dkv, (size_t)r * m->proj_pitch),
+                                     m->proj_pitch, at(m, gate, (size_t)r * m->proj_pitch), m->proj_pitch,
                                      at(m, m->cat, (size_t)r * m->cat_pitch), m->cat_pitch, sub, k, m->act32));
     }
     return PRISM_OK;
@@ -394,7 +400,7 @@ int layered_enqueue_step(prism_cuda_engine *e) {
     PRISM_TRY(launch_dense_embed(ctx, m->embed, m->c.width, m->c.vocab, e->tok, B, m->x));
     PRISM_TRY(forward_layers(e, rows, B, false));
     PRISM_TRY(head_rows(e, m->x, B));
-    PRISM_TRY(launch_argmax_f32(ctx, m->logits, m->c.vocab, m->vocab_pad, B, e->next));
+    PRISM_TRY(launch_argmax(ctx, m->logits, m->c.vocab, m->vocab_pad, B, e->next));
     return enqueue_advance(e, m->row_pos);
 }
 
@@ -503,7 +509,7 @@ static int logits_of(prism_cuda_engine *e, const uint32_t *idx, uint32_t n, floa
             PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(host + (size_t)i * m->c.vocab, (size_t)m->c.vocab * 4, m->logits, (size_t)m->vocab_pad * 4,
                                                   (size_t)m->c.vocab * 4, k, cudaMemcpyDeviceToHost, ctx->stream));
         if (next_host) {  // one row
-            PRISM_TRY(launch_argmax_f32(ctx, m->logits, m->c.vocab, m->vocab_pad, 1, e->next));
+            PRISM_TRY(launch_argmax(ctx, m->logits, m->c.vocab, m->vocab_pad, 1, e->next));
             PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(next_host, e->next, 4, cudaMemcpyDeviceToHost, ctx->stream));
         }
         PRISM_CUDA_TRY(ctx, cudaStreamSynchronize(ctx->stream));  // idx and the buffers are used again
@@ -531,7 +537,7 @@ int prism_cuda_engine_create_layered(prism_cuda_ctx *ctx, const prism_layered_co
     e->lm = new LayeredModel();
     e->lm->c = c;
     e->lm->act32 = c.dtype == PRISM_DTYPE_F32;
-    e->lm->chunk = std::min(c.max_seq, (uint32_t)std::max(1, ctx->prefill_chunk));
+    e->lm->chunk = std::min(c.max_seq, (uint32_t)std::max(1, ctx->layered_chunk));
     // what the shared loop reads of the palettized configuration
     e->cfg.num_layers = c.num_layers; e->cfg.hidden_size = c.width; e->cfg.vocab_size = c.vocab; e->cfg.norm_eps = c.norm_eps;
     e->cfg.max_seq = c.max_seq; e->cfg.max_batch = c.max_batch;

@@ -98,11 +98,11 @@ __global__ void __launch_bounds__(LT_THREADS) lightning_chunk_kernel(const Light
     pdl_wait();
     const uint32_t PD = dpad + 8, h = blockIdx.y, v0 = blockIdx.x * LT_VS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t g8 = lane >> 2, t4 = lane & 3;
-    bf16 *Qs = reinterpret_cast<bf16 *>(lcs), *Ks = Qs + LC_C * PD, *Vs = Ks + LC_C * PD, *Vh = Vs + LC_C * LC_PV, *Vl = Vh + LC_C * LC_PV,
+    const uint32_t TILE = 2 * LC_C * PD + LC_C * LC_PV;  // q, k and v of a chunk; two of them, the next chunk loads under this one
+    bf16 *tiles = reinterpret_cast<bf16 *>(lcs), *Vh = tiles + 2 * TILE, *Vl = Vh + LC_C * LC_PV,
          *Ah = Vl + LC_C * LC_PV, *Al = Ah + LC_C * LC_PA, *Sh = Al + LC_C * LC_PA, *Sl = Sh + dpad * LC_PV;
     float *pw = reinterpret_cast<float *>(Sl + dpad * LC_PV);  // d^0 .. d^64
-    const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(Qs), sK = (uint32_t)__cvta_generic_to_shared(Ks), sV = (uint32_t)__cvta_generic_to_shared(Vs),
-                   sVh = (uint32_t)__cvta_generic_to_shared(Vh), sVl = (uint32_t)__cvta_generic_to_shared(Vl), sAh = (uint32_t)__cvta_generic_to_shared(Ah),
+    const uint32_t sT = (uint32_t)__cvta_generic_to_shared(tiles), sVh = (uint32_t)__cvta_generic_to_shared(Vh), sVl = (uint32_t)__cvta_generic_to_shared(Vl), sAh = (uint32_t)__cvta_generic_to_shared(Ah),
                    sAl = (uint32_t)__cvta_generic_to_shared(Al), sSh = (uint32_t)__cvta_generic_to_shared(Sh), sSl = (uint32_t)__cvta_generic_to_shared(Sl);
     const bf16 zero = __float2bfloat16_rn(0.0f);
     const bf16 *q = reinterpret_cast<const bf16 *>(a.q) + h * a.dim, *k = reinterpret_cast<const bf16 *>(a.k) + h * a.dim,
@@ -126,38 +126,56 @@ __global__ void __launch_bounds__(LT_THREADS) lightning_chunk_kernel(const Light
                 st[m][n][i] = d < a.dim && c < a.vdim ? S[(size_t)d * a.vdim + c] : 0.0f;
             }
     const uint32_t n_mt = dpad / 16;
-    for (uint32_t r0 = 0; r0 < a.rows; r0 += LC_C) {
-        const uint32_t nt = min((uint32_t)LC_C, a.rows - r0);
-        __syncthreads();  // the previous chunk is done with the tiles
+    auto load_chunk = [&](uint32_t r0, uint32_t buf) {
+        const uint32_t nt = min((uint32_t)LC_C, a.rows - r0), sq = sT + buf * TILE * 2, sk = sq + LC_C * PD * 2, sv = sk + LC_C * PD * 2;
+        bf16 *Q = tiles + buf * TILE, *K = Q + LC_C * PD, *V = K + LC_C * PD;
         if (vec) {
+            const uint4 z = make_uint4(0, 0, 0, 0);
             const uint32_t d8 = dpad / 8, n8 = a.dim / 8;
             for (uint32_t i = tid; i < LC_C * d8; i += LT_THREADS) {
-                const uint32_t r = i / d8, c = i % d8;
-                uint4 x = make_uint4(0, 0, 0, 0), y = x;
+                const uint32_t r = i / d8, c = i % d8, at = r * PD + c * 8;
                 if (r < nt && c < n8) {
-                    x = *reinterpret_cast<const uint4 *>(q + (size_t)(r0 + r) * a.pitch + c * 8);
-                    y = *reinterpret_cast<const uint4 *>(k + (size_t)(r0 + r) * a.pitch + c * 8);
+                    cp_async16(sq + at * 2, q + (size_t)(r0 + r) * a.pitch + c * 8);
+                    cp_async16(sk + at * 2, k + (size_t)(r0 + r) * a.pitch + c * 8);
+                } else {
+                    *reinterpret_cast<uint4 *>(Q + at) = z;
+                    *reinterpret_cast<uint4 *>(K + at) = z;
                 }
-                *reinterpret_cast<uint4 *>(Qs + r * PD + c * 8) = x;
-                *reinterpret_cast<uint4 *>(Ks + r * PD + c * 8) = y;
+            }
+            {
+                const uint32_t r = tid / (LT_VS / 8), c = (tid % (LT_VS / 8)) * 8, at = r * LC_PV + c;  // 64 x 4 pieces: one per thread
+                if (r < nt && v0 + c < a.vdim) cp_async16(sv + at * 2, v + (size_t)(r0 + r) * a.pitch + v0 + c);
+                else *reinterpret_cast<uint4 *>(V + at) = z;
             }
         } else {
             for (uint32_t i = tid; i < LC_C * dpad; i += LT_THREADS) {
                 const uint32_t r = i / dpad, c = i % dpad;
                 const bool on = r < nt && c < a.dim;
-                Qs[r * PD + c] = on ? q[(size_t)(r0 + r) * a.pitch + c] : zero;
-                Ks[r * PD + c] = on ? k[(size_t)(r0 + r) * a.pitch + c] : zero;
+                Q[r * PD + c] = on ? q[(size_t)(r0 + r) * a.pitch + c] : zero;
+                K[r * PD + c] = on ? k[(size_t)(r0 + r) * a.pitch + c] : zero;
+            }
+            for (uint32_t i = tid; i < LC_C * LT_VS; i += LT_THREADS) {
+                const uint32_t r = i / LT_VS, c = i % LT_VS;
+                V[r * LC_PV + c] = r < nt && v0 + c < a.vdim ? v[(size_t)(r0 + r) * a.pitch + v0 + c] : zero;
             }
         }
+        cp_async_commit();
+    };
+    static_assert(LC_C * LT_VS / 8 == LT_THREADS, "one piece of v per thread");
+    load_chunk(0, 0);
+    uint32_t buf = 0;
+    for (uint32_t r0 = 0; r0 < a.rows; r0 += LC_C, buf ^= 1) {
+        const uint32_t nt = min((uint32_t)LC_C, a.rows - r0);
+        const uint32_t sQ = sT + buf * TILE * 2, sK = sQ + LC_C * PD * 2, sV = sK + LC_C * PD * 2;
+        const bf16 *Vs = tiles + buf * TILE + 2 * LC_C * PD;
+        cp_async_wait<0>();
+        __syncthreads();  // this chunk has arrived, and every warp is done with the previous one
+        if (r0 + LC_C < a.rows) load_chunk(r0 + LC_C, buf ^ 1);
         for (uint32_t i = tid; i < LC_C * LT_VS / 2; i += LT_THREADS) {
             const uint32_t r = i / (LT_VS / 2), c = (i % (LT_VS / 2)) * 2;
-            const bf16 *src = v + (size_t)(r0 + r) * a.pitch + v0 + c;
-            const bf16 x = r < nt && v0 + c < a.vdim ? src[0] : zero, y = r < nt && v0 + c + 1 < a.vdim ? src[1] : zero;
-            Vs[r * LC_PV + c] = x;
-            Vs[r * LC_PV + c + 1] = y;
             const float f = r < nt ? pw[nt - 1 - r] : 0.0f;
             uint32_t hi, lo;
-            split_bf16(__bfloat162float(x) * f, __bfloat162float(y) * f, hi, lo);
+            split_bf16(__bfloat162float(Vs[r * LC_PV + c]) * f, __bfloat162float(Vs[r * LC_PV + c + 1]) * f, hi, lo);
             *reinterpret_cast<uint32_t *>(Vh + r * LC_PV + c) = hi;
             *reinterpret_cast<uint32_t *>(Vl + r * LC_PV + c) = lo;
         }
@@ -176,7 +194,6 @@ __global__ void __launch_bounds__(LT_THREADS) lightning_chunk_kernel(const Light
                         *reinterpret_cast<uint32_t *>(Sl + at) = lo;
                     }
             }
-        __syncthreads();
         const uint32_t i0 = (warp & 3) * 16;
         // decayed scores: rows i0 .. +16, columns (warp / 4) * 32 .. +32
         {
@@ -277,7 +294,7 @@ __global__ void __launch_bounds__(LT_THREADS) lightning_chunk_kernel(const Light
 }
 
 // ---- host side ---------------------------------------------------------------------------------
-constexpr size_t LT_SMEM_MAX = 200 * 1024;
+constexpr size_t LT_SMEM_MAX = 224 * 1024;
 
 int launch_lightning_step(prism_cuda_ctx *ctx, const LightningArgs &a, const RowMap &rows, bool act32) {
     const dim3 grid((a.vdim + LT_VS - 1) / LT_VS, a.heads, a.rows);
@@ -298,9 +315,10 @@ int launch_lightning_seq(prism_cuda_ctx *ctx, const LightningArgs &a, const RowM
     }
     const dim3 grid((a.vdim + LT_VS - 1) / LT_VS, a.heads);
     const uint32_t dpad = round_up_u32(a.dim, 16);
-    const size_t csm = ((size_t)2 * LC_C * (dpad + 8) + 3 * LC_C * LC_PV + 2 * LC_C * LC_PA + 2 * (size_t)dpad * LC_PV) * 2 + (LC_C + 1) * 4;
+    const size_t csm = ((size_t)4 * LC_C * (dpad + 8) + 4 * LC_C * LC_PV + 2 * LC_C * LC_PA + 2 * (size_t)dpad * LC_PV) * 2 + (LC_C + 1) * 4;
     if (!act32 && dpad <= 256 && a.rows > DENSE_GEMV_ROWS && csm <= LT_SMEM_MAX) {
-        const uint32_t vec = a.dim % 8 == 0 && a.pitch % 8 == 0 && !((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k)) & 15);
+        const uint32_t vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.pitch % 8 == 0 &&
+                             !((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v)) & 15);
         launch_pdl(ctx, "lightning_chunk_kernel", lightning_chunk_kernel, grid, LT_THREADS, csm, a, rows.slot0, dpad, vec);
         return after_launch(ctx, "lightning_chunk_kernel");
     }
