@@ -404,7 +404,7 @@ int prism_cuda_engine_seq_close(prism_cuda_engine *eng, uint32_t seq);
 int prism_cuda_engine_seq_position(prism_cuda_engine *eng, uint32_t seq, uint32_t *pos);
 /* One step over `n` open sequences: entry i appends n_tokens[i] tokens (taken one entry after the other from
  * `tokens`) where its sequence stands.  Entries of one token run together as a decode step, longer ones as
- * prompt portions.  want lists, entry by entry, n_want[i] ascending places inside the entry's tokens whose
+ * prompt portions.  want lists, entry by entry, n_want[i] places inside the entry's tokens (any order) whose
  * fp32 logits go to `logits` ([sum n_want][vocab], host); next_tokens (optional) gets the greedy token
  * after each entry.  A sequence may appear once per call. */
 int prism_cuda_engine_extend(prism_cuda_engine *eng, uint32_t n, const uint32_t *seqs, const uint32_t *n_tokens,

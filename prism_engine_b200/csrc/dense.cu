@@ -99,45 +99,93 @@ struct GemvArgs {
     uint32_t pitch, f32;
     const float *norm_w;
     const bf16 *gate;
-    uint32_t gate_pitch, n_norm, norm_pad;  // norm_pad: n_norm rounded up to 64
+    uint32_t gate_pitch, n_norm, norm_pad, norm_vec;  // norm_pad: n_norm rounded up to 64; norm_vec: rows allow 4-value accesses
     float eps;
     DenseEpi epi;
 };
 constexpr int GV_THREADS = 256, GV_WARPS = 8, GV_U = 4, GV_KS_MAX = 4;
 
-// RMS norm (times weight, times gate) of the first n_norm entries of every row into shared memory as bf16.
-__device__ __forceinline__ void gemv_stage_norm(const GemvArgs &a, bf16 *xs, float *sh) {
-    const uint32_t R = a.rows;
-    const uint32_t tpr = R == 1 ? 256 : R == 2 ? 128 : R <= 4 ? 64 : 32;  // threads per row
-    const uint32_t r = threadIdx.x / tpr, i0 = threadIdx.x % tpr;
-    const bool on = r < R;
-    const float *xf = reinterpret_cast<const float *>(a.x) + (size_t)r * a.pitch;
-    const bf16 *xh = reinterpret_cast<const bf16 *>(a.x) + (size_t)r * a.pitch;
-    float ss = 0.0f;
-    if (on)
-        for (uint32_t i = i0; i < a.n_norm; i += tpr) {
-            const float v = a.f32 ? xf[i] : __bfloat162float(xh[i]);
-            ss += v * v;
-        }
-    ss = warp_sum_f(ss);
-    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = ss;
-    __syncthreads();
-    if (on) {
-        const uint32_t w0 = r * (tpr / 32);
-        float s = 0.0f;
-        for (uint32_t w = 0; w < tpr / 32; w++) s += sh[w0 + w];
-        const float inv = 1.0f / sqrtf(s / (float)a.n_norm + a.eps);
-        for (uint32_t i = i0; i < a.norm_pad; i += tpr) {
-            float v = 0.0f;
-            if (i < a.n_norm) {
-                v = (a.f32 ? xf[i] : __bfloat162float(xh[i])) * inv * __ldg(a.norm_w + i);
-                if (a.gate) v *= __bfloat162float(a.gate[(size_t)r * a.gate_pitch + i]);
+// Four consecutive values of a row.
+__device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 ld4(const bf16 *p) {
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void st4(bf16 *p, float4 v) { *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+
+// RMS norm (times weight, times gate) of the first n_norm entries of the one or two rows into shared memory as bf16.
+// A row's threads keep their values and weights in registers (the weights requested before the dependency wait).
+constexpr int GN_U = 8;
+struct GemvNorm {
+    float4 w[GN_U];
+    uint32_t tpr, r, i0;
+    bool vec;
+    __device__ __forceinline__ void prefetch(const GemvArgs &a) {
+        tpr = a.rows == 1 ? 256 : 128;  // threads per row
+        r = threadIdx.x / tpr;
+        i0 = threadIdx.x % tpr;
+        vec = a.norm_vec && a.n_norm <= tpr * 4 * GN_U;
+        if (vec) {
+#pragma unroll
+            for (int u = 0; u < GN_U; u++) {
+                const uint32_t i = (i0 + u * tpr) * 4;
+                w[u] = i < a.n_norm ? ld4(a.norm_w + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             }
-            xs[(size_t)r * a.norm_pad + i] = __float2bfloat16_rn(v);
         }
     }
-    __syncthreads();
-}
+    __device__ __forceinline__ float inverse(const GemvArgs &a, float ss, float *sh) const {
+        ss = warp_sum_f(ss);
+        if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = ss;
+        __syncthreads();
+        float s = 0.0f;
+        for (uint32_t k = 0; k < tpr / 32; k++) s += sh[r * (tpr / 32) + k];
+        return 1.0f / sqrtf(s / (float)a.n_norm + a.eps);
+    }
+    __device__ __forceinline__ void stage(const GemvArgs &a, bf16 *xs, float *sh) const {
+        const float *xf = reinterpret_cast<const float *>(a.x) + (size_t)r * a.pitch;
+        const bf16 *xh = reinterpret_cast<const bf16 *>(a.x) + (size_t)r * a.pitch, *gr = a.gate ? a.gate + (size_t)r * a.gate_pitch : nullptr;
+        bf16 *y = xs + (size_t)r * a.norm_pad;
+        float ss = 0.0f;
+        if (vec) {
+            float4 v[GN_U];
+#pragma unroll
+            for (int u = 0; u < GN_U; u++) {
+                const uint32_t i = (i0 + u * tpr) * 4;
+                v[u] = i < a.n_norm ? a.f32 ? ld4(xf + i) : ld4(xh + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+            }
+            const float inv = inverse(a, ss, sh);
+#pragma unroll
+            for (int u = 0; u < GN_U; u++) {
+                const uint32_t i = (i0 + u * tpr) * 4;
+                if (i >= a.norm_pad) break;
+                float4 o = make_float4(v[u].x * inv * w[u].x, v[u].y * inv * w[u].y, v[u].z * inv * w[u].z, v[u].w * inv * w[u].w);
+                if (gr && i < a.n_norm) {
+                    const float4 g = ld4(gr + i);
+                    o = make_float4(o.x * g.x, o.y * g.y, o.z * g.z, o.w * g.w);
+                }
+                st4(y + i, o);
+            }
+        } else {
+            for (uint32_t i = i0; i < a.n_norm; i += tpr) {
+                const float v = a.f32 ? xf[i] : __bfloat162float(xh[i]);
+                ss += v * v;
+            }
+            const float inv = inverse(a, ss, sh);
+            for (uint32_t i = i0; i < a.norm_pad; i += tpr) {
+                float v = 0.0f;
+                if (i < a.n_norm) {
+                    v = (a.f32 ? xf[i] : __bfloat162float(xh[i])) * inv * __ldg(a.norm_w + i);
+                    if (gr) v *= __bfloat162float(gr[i]);
+                }
+                y[i] = __float2bfloat16_rn(v);
+            }
+        }
+        __syncthreads();
+    }
+};
 
 template <bool NORM>
 __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArgs a) {
@@ -182,8 +230,10 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
     const uint32_t grp0 = blockIdx.x / a.ks;
     const uint4 *wt = locate(grp0, sg, rb);
     load(wt, first + warp);  // weights do not depend on the previous kernel; the input does
+    GemvNorm norm;
+    if (NORM) norm.prefetch(a);
     pdl_wait();
-    if (NORM) gemv_stage_norm(a, xs, sh);
+    if (NORM) norm.stage(a, xs, sh);
     bool loaded = true;
     for (uint32_t grp = grp0; grp < a.n_groups; grp += gridDim.x / a.ks) {
         if (!loaded) wt = locate(grp, sg, rb);
@@ -234,7 +284,7 @@ static size_t gemv_smem(const DenseIn &in, uint32_t rows) {
     return in.norm_w ? (size_t)rows * round_up_u32(in.n_norm, 64) * 2 : 0;
 }
 constexpr size_t GV_SMEM_MAX = 160 * 1024;
-constexpr uint32_t GV_FOLD_ROWS = 2;  // more rows: every CTA norming all of them costs more than a norm kernel does
+constexpr uint32_t GV_FOLD_ROWS = 2;  // as many as GemvNorm splits the block into; more rows: every CTA norming all of them costs more than a norm kernel does
 
 bool dense_gemv_ok(const DenseIn &in, uint32_t rows) {
     return rows <= DENSE_GEMV_ROWS && (in.norm_w ? rows <= GV_FOLD_ROWS && gemv_smem(in, rows) <= GV_SMEM_MAX : !in.f32) &&
@@ -249,6 +299,8 @@ int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &
     a.x = in.x; a.pitch = in.pitch; a.f32 = in.f32;
     a.norm_w = in.norm_w; a.n_norm = in.n_norm; a.norm_pad = round_up_u32(in.n_norm, 64); a.eps = in.eps;
     a.gate = reinterpret_cast<const bf16 *>(in.gate); a.gate_pitch = in.gate_pitch;
+    a.norm_vec = !((reinterpret_cast<uintptr_t>(in.x) | reinterpret_cast<uintptr_t>(in.gate) | reinterpret_cast<uintptr_t>(in.norm_w)) & 15) &&
+                 !((in.pitch | in.n_norm | (in.gate ? in.gate_pitch : 0)) & 3);
     a.epi = dense_epi(l, outs);
     for (uint32_t s = 0; s < l.n_segs; s++) a.n_groups += (l.seg[s].rows + 31) / 32;
     // few row blocks and a long k: share a block's k range inside a cluster, at least GV_WARPS * GV_U steps each
@@ -323,16 +375,6 @@ int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const float *x, 
 }
 
 // ---- element-wise ------------------------------------------------------------------------------------
-// Four consecutive values of a row.
-__device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
-__device__ __forceinline__ float4 ld4(const bf16 *p) {
-    const uint2 u = *reinterpret_cast<const uint2 *>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-__device__ __forceinline__ void st4(bf16 *p, float4 v) { *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
-
 constexpr int DN_THREADS = 256, DN_U = 8;  // a row of up to 8192 values is read once and kept in registers
 template <typename TX, typename TA>
 __global__ void __launch_bounds__(DN_THREADS) dense_norm_kernel(const TX *__restrict__ x, uint32_t pitch, const float *__restrict__ w,

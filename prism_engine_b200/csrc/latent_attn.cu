@@ -198,22 +198,27 @@ __global__ void __launch_bounds__(128) latent_rows_mma_kernel(const LatentArgs a
     const int32_t pos = rows.pos_of(r), slot = rows.slot_of(r), k0 = first_key(a, pos) + (int32_t)split * LR_KT, n = min(pos + 1 - k0, LR_KT);
     if (n <= 0) return;
     const uint32_t sC = (uint32_t)__cvta_generic_to_shared(Cs), sQh = (uint32_t)__cvta_generic_to_shared(Qh), sQl = (uint32_t)__cvta_generic_to_shared(Ql);
-    const uint32_t L8 = L / 8;
     const bf16 *c = reinterpret_cast<const bf16 *>(a.cache.rows);
-    for (uint32_t i = tid; i < LR_KT * L8; i += 128) {
-        const uint32_t k = i / L8, j = i % L8;
-        if ((int32_t)k < n) cp_async16(sC + (k * P + j * 8) * 2, c + cache_row(a.cache, slot, k0 + k) + j * 8);
-        else *reinterpret_cast<uint4 *>(Cs + k * P + j * 8) = make_uint4(0, 0, 0, 0);
+    for (uint32_t k = warp; k < LR_KT; k += 4) {  // a warp per cached row
+        const bf16 *src = c + cache_row(a.cache, slot, k0 + (int32_t)k);
+        for (uint32_t j = lane * 8; j < L; j += 256) {
+            if ((int32_t)k < n) cp_async16(sC + (k * P + j) * 2, src + j);
+            else *reinterpret_cast<uint4 *>(Cs + k * P + j) = make_uint4(0, 0, 0, 0);
+        }
     }
     cp_async_commit();
-    for (uint32_t i = tid; i < 16 * L / 2; i += 128) {
-        const uint32_t h = i / (L / 2), j = (i % (L / 2)) * 2;
-        float2 x = make_float2(0.0f, 0.0f);
-        if (h0 + h < a.heads) x = *reinterpret_cast<const float2 *>(qa + ((size_t)r * a.heads + h0 + h) * L + j);
-        uint32_t hi, lo;
-        split_bf16(x.x, x.y, hi, lo);
-        *reinterpret_cast<uint32_t *>(Qh + h * P + j) = hi;
-        *reinterpret_cast<uint32_t *>(Ql + h * P + j) = lo;
+    for (uint32_t h = warp; h < 16; h += 4) {
+        const float *src = qa + ((size_t)r * a.heads + h0 + h) * L;
+#pragma unroll 4
+        for (uint32_t j = lane * 4; j < L; j += 128) {
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (h0 + h < a.heads) x = *reinterpret_cast<const float4 *>(src + j);
+            uint2 hi, lo;
+            split_bf16(x.x, x.y, hi.x, lo.x);
+            split_bf16(x.z, x.w, hi.y, lo.y);
+            *reinterpret_cast<uint2 *>(Qh + h * P + j) = hi;
+            *reinterpret_cast<uint2 *>(Ql + h * P + j) = lo;
+        }
     }
     cp_async_wait<0>();
     __syncthreads();

@@ -496,8 +496,9 @@ uint64_t layered_step_bytes(const prism_cuda_engine *e) {
     return bytes;
 }
 
-// Greedy next token and wanted logits of rows `idx` (places in m->x) of a portion's chunk.
-static int logits_of(prism_cuda_engine *e, const uint32_t *idx, uint32_t n, float *host, uint32_t *next_host) {
+// Logits of rows `idx` (places in m->x) of a portion's chunk, row i to host row dst[i]; next_host: the greedy
+// token of a single row instead.
+static int logits_of(prism_cuda_engine *e, const uint32_t *idx, const uint32_t *dst, uint32_t n, float *host, uint32_t *next_host) {
     prism_cuda_ctx *ctx = e->ctx;
     LayeredModel *m = e->lm;
     for (uint32_t i = 0; i < n; i += m->lg_cap) {
@@ -505,9 +506,11 @@ static int logits_of(prism_cuda_engine *e, const uint32_t *idx, uint32_t n, floa
         PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(m->want_idx, idx + i, (size_t)k * 4, cudaMemcpyHostToDevice, ctx->stream));
         PRISM_TRY(launch_gather_rows_f32(ctx, m->x, m->want_idx, k, m->c.width, m->xw));
         PRISM_TRY(head_rows(e, m->xw, k));
-        if (host)
-            PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(host + (size_t)i * m->c.vocab, (size_t)m->c.vocab * 4, m->logits, (size_t)m->vocab_pad * 4,
-                                                  (size_t)m->c.vocab * 4, k, cudaMemcpyDeviceToHost, ctx->stream));
+        for (uint32_t j = 0, run; host && j < k; j += run) {  // runs of consecutive host rows
+            for (run = 1; j + run < k && dst[i + j + run] == dst[i + j] + run;) run++;
+            PRISM_CUDA_TRY(ctx, cudaMemcpy2DAsync(host + (size_t)dst[i + j] * m->c.vocab, (size_t)m->c.vocab * 4, m->logits + (size_t)j * m->vocab_pad,
+                                                  (size_t)m->vocab_pad * 4, (size_t)m->c.vocab * 4, run, cudaMemcpyDeviceToHost, ctx->stream));
+        }
         if (next_host) {  // one row
             PRISM_TRY(launch_argmax(ctx, m->logits, m->c.vocab, m->vocab_pad, 1, e->next));
             PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(next_host, e->next, 4, cudaMemcpyDeviceToHost, ctx->stream));
@@ -630,7 +633,7 @@ int prism_cuda_engine_extend(prism_cuda_engine *e, uint32_t n, const uint32_t *s
             if (tokens[nt + t] >= m->c.vocab) return fail(ctx, PRISM_E_ARG, "token id outside the vocabulary");
         const uint32_t w = n_want ? n_want[i] : 0;
         for (uint32_t k = 0; k < w; k++)
-            if (want[nw + k] >= n_tokens[i] || (k && want[nw + k] <= want[nw + k - 1])) return fail(ctx, PRISM_E_ARG, "wanted places must ascend inside the entry");
+            if (want[nw + k] >= n_tokens[i]) return fail(ctx, PRISM_E_ARG, "a wanted place lies outside the entry");
         nt += n_tokens[i];
         nw += w;
     }
@@ -655,8 +658,8 @@ int prism_cuda_engine_extend(prism_cuda_engine *e, uint32_t n, const uint32_t *s
         for (size_t r = 0; r < one.size(); r++) {
             const uint32_t i = one[r];
             m->slot_pos[seqs[i]] += 1;
-            if (n_want && n_want[i])
-                PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(logits + want0[i] * m->c.vocab, m->logits + r * m->vocab_pad, (size_t)m->c.vocab * 4,
+            for (uint32_t k = 0; n_want && k < n_want[i]; k++)
+                PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(logits + (want0[i] + k) * m->c.vocab, m->logits + r * m->vocab_pad, (size_t)m->c.vocab * 4,
                                                     cudaMemcpyDeviceToHost, ctx->stream));
         }
         PRISM_CUDA_TRY(ctx, cudaMemcpyAsync(nx.data(), e->next, nx.size() * 4, cudaMemcpyDeviceToHost, ctx->stream));
@@ -669,16 +672,16 @@ int prism_cuda_engine_extend(prism_cuda_engine *e, uint32_t n, const uint32_t *s
         const uint32_t nwi = n_want ? n_want[i] : 0;
         const uint32_t *w = want + want0[i];
         PRISM_TRY(run_portion(e, seqs[i], tokens + tok0[i], n_tokens[i], [&](uint32_t t0, uint32_t k) -> int {
-            std::vector<uint32_t> idx;
-            uint32_t first = 0;
-            for (uint32_t j = 0; j < nwi; j++) {
-                if (w[j] < t0) first = j + 1;
-                else if (w[j] < t0 + k) idx.push_back(w[j] - t0);
-            }
-            if (!idx.empty()) PRISM_TRY(logits_of(e, idx.data(), (uint32_t)idx.size(), logits + (want0[i] + first) * m->c.vocab, nullptr));
+            std::vector<uint32_t> idx, dst;
+            for (uint32_t j = 0; j < nwi; j++)
+                if (w[j] >= t0 && w[j] < t0 + k) {
+                    idx.push_back(w[j] - t0);
+                    dst.push_back((uint32_t)want0[i] + j);
+                }
+            if (!idx.empty()) PRISM_TRY(logits_of(e, idx.data(), dst.data(), (uint32_t)idx.size(), logits, nullptr));
             if (next_tokens && t0 + k == n_tokens[i]) {
                 const uint32_t last = k - 1;
-                PRISM_TRY(logits_of(e, &last, 1, nullptr, next_tokens + i));
+                PRISM_TRY(logits_of(e, &last, nullptr, 1, nullptr, next_tokens + i));
             }
             return PRISM_OK;
         }));

@@ -169,6 +169,20 @@ def test_decode_batch_beyond_the_small_kernel(backend):
         eng.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_odd_sizes_and_wanted_places_in_any_order(backend, dtype):
+    cfg = U.model([U.latent(3, 10, 6, 14, 23, 19, window=11, ff=37), U.lightning(3, 9, 5, ff=61), U.lightning(1, 5, 3)], width=45, vocab=101)
+    check(backend, cfg, n=90, sizes=(33, 2, 1), dtype=dtype, seed=17)
+    w, toks = U.weights(cfg, 18), tokens(40, 101, 18)
+    want = orc.forward(cfg, w, toks)
+    eng = U.engine(backend, cfg, w, dtype, max_seq=64, chunk=16)  # the places fall into several chunks
+    s = eng.open_sequence()
+    places = [38, 3, 3, 17, 16, 0, 30]
+    assert U.error(eng.extend([(s, toks[:39], places)]), want[places]) < U.TOL[dtype]
+    assert U.error(eng.extend([(s, toks[39:], [0, 0])]), want[[39, 39]]) < U.TOL[dtype]
+    eng.close()
+
+
 def test_unfused_path_agrees(backend):
     """Option fuse = 0: separate norms and the tensor-core GEMM at every size, one row included."""
     backend.set_option("fuse", 0)
@@ -344,7 +358,7 @@ def test_errors_are_reported(backend):
     s = eng.open_sequence()
     with pytest.raises(p.PrismCudaError, match="in use"):
         eng.open_sequence()
-    for bad in ([(s, [], [])], [(s, [131], [])], [(s, [1, 2], [1, 0])], [(s, [1], [1])], [(3, [1], [])], [(s, [1], []), (s, [2], [])]):
+    for bad in ([(s, [], [])], [(s, [131], [])], [(s, [1, 2], [2])], [(s, [1], [1])], [(3, [1], [])], [(s, [1], []), (s, [2], [])]):
         with pytest.raises(p.PrismCudaError):
             eng.extend(bad)
     with pytest.raises(p.PrismCudaError, match="max_seq"):
