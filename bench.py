@@ -666,7 +666,7 @@ def layered_raw(name):
     lightning = {"type": "lightning", "mixer": dict(li, decay=decay)}
     latent = {"type": "latent_attention", "mixer": dict(
         {k: v for k, v in la.items() if k != "window"}, mask={"size": la["window"]}, scale=(la["dim"] + la["rot_dim"]) ** -0.5,
-        rot={"base": 1e6, "dims": la["rot_dim"], "scaling": {"factor": 4.0, "fast": 32.0, "original": 4096, "slow": 1.0}})}
+        rot={"base": 5e5, "dims": la["rot_dim"], "scaling": {"factor": 8.0, "fast": 16.0, "original": 4096, "slow": 2.0}})}
     layers = [dict(latent if i % 2 else lightning, mlp={"kind": "dense", "ff": arch["intermediate_size"]})
               for i in range(arch["num_layers"])]
     raw = {"architecture": "Mefipel", "layers": layers, "logit_scale": 1.0, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
@@ -698,7 +698,8 @@ def measure_layered(env, be, name, batches, steps, warmup, ctx_len, n_prompt):
         else:
             eng = p.PrismEngine(be, p.model_config(**arch, max_seq=max_seq, max_batch=max(batches), profile="baseline"))
         eng.synth_weights(seed=1)
-        prompt = synth.make_prompt(n_prompt, arch["vocab_size"], seed=3)
+        # the layered generate() leaves the last prompt token to the first decode step
+        prompt = synth.make_prompt(n_prompt + (kind == "layered"), arch["vocab_size"], seed=3)
         for _ in range(2):
             eng.generate(prompt, 0)
         reps = 5

@@ -67,6 +67,45 @@ __device__ __forceinline__ void dg_item(const DgArgs &a, uint32_t w, uint32_t &r
     tt = rem / gr;
 }
 
+// The epilogue of dense_store for one weight row (a lane) over the NT tokens of a tile, with what does not change
+// along the way decided once: sixteen accumulators are read, the residual's old values requested together, and
+// the activation of a bf16 result takes the fast exponential and reciprocal.
+template <uint32_t ACT>
+__device__ __forceinline__ float act_fast(float z) {
+    if (ACT == ACT_NONE) return z;
+    const float u = ACT == ACT_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;  // (1 + tanh(u / 2)) / 2 = sigmoid(u)
+    const float g = __fdividef(1.0f, 1.0f + __expf(-u));
+    return ACT == ACT_SIGMOID ? g : z * g;
+}
+template <int NT, uint32_t ACT, uint32_t STORE>
+__device__ __forceinline__ void epilogue_row(const DenseEpiSeg &seg, uint32_t row, bool row_ok, uint32_t taddr, uint32_t t0, uint32_t rows) {
+    const float bias = seg.bias && row_ok ? __ldg(seg.bias + row) : 0.0f, mul = seg.mul;
+    const uint32_t pitch = seg.pitch;
+    bf16 *yh = reinterpret_cast<bf16 *>(seg.p) + (size_t)t0 * pitch + row;
+    float *yf = reinterpret_cast<float *>(seg.p) + (size_t)t0 * pitch + row;
+    const uint32_t n = rows > t0 ? min(rows - t0, (uint32_t)NT) : 0;
+#pragma unroll 1
+    for (uint32_t g = 0; g < n; g += 16) {
+        uint32_t v[16];
+        float old[16];
+        t5::ld16(taddr + g, v);
+        if (STORE == ST_RESID) {
+#pragma unroll
+            for (uint32_t i = 0; i < 16; i++) old[i] = row_ok && g + i < n ? yf[(size_t)(g + i) * pitch] : 0.0f;
+        }
+        t5::wait_ld();
+#pragma unroll
+        for (uint32_t i = 0; i < 16; i++) {
+            const float y = act_fast<ACT>(__uint_as_float(v[i]) + bias) * mul;
+            if (row_ok && g + i < n) {
+                if (STORE == ST_ACT) yh[(size_t)(g + i) * pitch] = __float2bfloat16_rn(y);
+                else yf[(size_t)(g + i) * pitch] = STORE == ST_RESID ? old[i] + y : y;
+            }
+        }
+        __syncwarp();  // the next TMEM read takes the whole warp
+    }
+}
+
 template <int NT, int RT>
 __global__ void __launch_bounds__(DgCfg<NT, RT>::THREADS, 1) dense_gemm_tc5_kernel(const DgArgs a, const __grid_constant__ CUtensorMap xmap) {
     using C = DgCfg<NT, RT>;
@@ -164,17 +203,14 @@ __global__ void __launch_bounds__(DgCfg<NT, RT>::THREADS, 1) dense_gemm_tc5_kern
             const bool row_ok = row < seg.rows;
             t5::mbar_wait_warp(b_dfull + 8 * b, ph, err_flag);
             t5::fence_after();
-#pragma unroll 1
-            for (int g = 0; g < NT / 16; g++) {
-                uint32_t v[16];
-                t5::ld16(tmem + ((q * 32) << 16) + b * NT + g * 16, v);
-                t5::wait_ld();
-                const uint32_t t0 = tt * NT + g * 16;
-                if (row_ok && t0 < a.rows) {
-#pragma unroll
-                    for (int i = 0; i < 16; i++)
-                        if (t0 + i < a.rows) dense_store<bf16>(seg, row, t0 + i, __uint_as_float(v[i]));
-                }
+            const uint32_t taddr = tmem + ((q * 32) << 16) + b * NT, t0 = tt * NT;
+            switch (seg.store * 4 + seg.act) {
+            case ST_ACT * 4 + ACT_NONE: epilogue_row<NT, ACT_NONE, ST_ACT>(seg, row, row_ok, taddr, t0, a.rows); break;
+            case ST_ACT * 4 + ACT_SILU: epilogue_row<NT, ACT_SILU, ST_ACT>(seg, row, row_ok, taddr, t0, a.rows); break;
+            case ST_ACT * 4 + ACT_SIGMOID: epilogue_row<NT, ACT_SIGMOID, ST_ACT>(seg, row, row_ok, taddr, t0, a.rows); break;
+            case ST_ACT * 4 + ACT_GELU_TANH: epilogue_row<NT, ACT_GELU_TANH, ST_ACT>(seg, row, row_ok, taddr, t0, a.rows); break;
+            case ST_F32 * 4 + ACT_NONE: epilogue_row<NT, ACT_NONE, ST_F32>(seg, row, row_ok, taddr, t0, a.rows); break;
+            default: epilogue_row<NT, ACT_NONE, ST_RESID>(seg, row, row_ok, taddr, t0, a.rows); break;  // the launcher rejects the rest
             }
             t5::fence_before();
             __syncwarp();
@@ -232,6 +268,8 @@ static int launch_dg(prism_cuda_ctx *ctx, const DenseLinear &l, DgArgs &a, const
 int launch_dense_gemm_tc5(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 *x, uint32_t pitch, const DenseOut *outs, uint32_t rows) {
     if ((reinterpret_cast<uintptr_t>(x) & 15) || pitch % 8 || pitch < l.k_pad || l.k_pad % 64)
         return fail(ctx, PRISM_E_ARG, "dense gemm: input rows must be 16-byte aligned and hold the padded k range");
+    for (uint32_t i = 0; i < l.n_segs; i++)
+        if (outs[i].store != ST_ACT && l.seg[i].act != ACT_NONE) return fail(ctx, PRISM_E_ARG, "dense gemm: fp32 outputs take no activation");
     DgArgs a{};
     a.w = reinterpret_cast<const uint8_t *>(l.w);
     a.kb = l.k_pad / 64;

@@ -36,7 +36,7 @@ def check(be, cfg, n=70, sizes=(10 ** 9,), dtype="float32", seed=0, **kw):
 
 LIGHTNING = [
     dict(heads=2, dim=16, vdim=32), dict(heads=1, dim=8, vdim=8, decay=[1.0]), dict(heads=3, dim=20, vdim=36, decay=[0.2, 0.97, 1.0]),
-    dict(heads=2, dim=7, vdim=13), dict(heads=1, dim=136, vdim=40), dict(heads=1, dim=256, vdim=64, decay=[0.999]),
+    dict(heads=2, dim=7, vdim=13), dict(heads=1, dim=136, vdim=40), dict(heads=1, dim=256, vdim=64, decay=[0.9985]),
     dict(heads=1, dim=272, vdim=24, decay=[0.9]), dict(heads=2, dim=24, vdim=16, decay=[0.0, 0.5])]
 LATENT = [
     dict(heads=2, dim=16, rot_dim=8, vdim=24, q_rank=40, kv_rank=32, window=20),

@@ -47,7 +47,7 @@ def test_unknown_parts_are_refused():
 
 
 @pytest.mark.parametrize("base,dims,scaling", [
-    (1e4, 16, None), (1e6, 64, {"factor": 8.0, "fast": 32.0, "original": 4096, "slow": 1.0}),
+    (1e4, 16, None), (2e5, 64, {"factor": 8.0, "fast": 24.0, "original": 4096, "slow": 1.5}),
     (5e5, 2, {"factor": 2.0, "fast": 4.0, "original": 128, "slow": 1.0}),
     (1e4, 10, {"factor": 1.0, "fast": 1.0, "original": 64, "slow": 1.0}),       # lo == hi or close
     (1e4, 24, {"factor": 40.0, "fast": 1e-3, "original": 64, "slow": 1e-4})])   # hi clamped to dims - 1
