@@ -1,6 +1,6 @@
 """Plain, slow restatement of the layer-list models (Mefipel), one numpy function per mechanism.
 
-It is the checker of the product's layered engine and shares nothing with it: it reads the same
+The tests compare the layered engine with it; it shares nothing with the product: it reads the same
 config.json keys and tensor names, works in numpy at the precision of ``dt`` (float64 by default) and
 handles one sequence, token positions 0 .. n-1, with no cache, no chunks and no batching.
 """
