@@ -362,8 +362,18 @@ uint32_t prism_cuda_engine_kernels_per_step(prism_cuda_engine *eng);
  * over a list of layers instead of the Llama/Qwen2 node order: every layer names its mixer and its sizes.
  * Residual, norms, attention scores and weights, positions and recurrent state are fp32; linears and
  * activations are bf16 with fp32 accumulation, or everything is fp32 (dtype). */
-enum { PRISM_MIXER_LIGHTNING = 0, PRISM_MIXER_LATENT_ATTENTION = 1 };
+enum {
+    PRISM_MIXER_LIGHTNING = 0,         /* linear attention with one decay per head */
+    PRISM_MIXER_LATENT_ATTENTION = 1,  /* keys and values expanded from one cached latent per token */
+    PRISM_MIXER_ATTENTION = 2,         /* softmax attention, query heads share key/value heads, no rotation */
+    PRISM_MIXER_GATED_DELTA = 3,       /* gated delta rule with short convolutions */
+    PRISM_MIXER_PAIR = 4               /* two mixers of one input, each result normed over the width, their mean */
+};
 enum { PRISM_DTYPE_BF16 = 0, PRISM_DTYPE_F32 = 1 };
+enum {
+    PRISM_ARRANGE_PARALLEL = 0,        /* mixer and feed-forward read one norm, both are added to the residual */
+    PRISM_ARRANGE_SEQUENTIAL = 1       /* x + mixer(norm1 x), then x + feed-forward(norm2 x) */
+};
 
 typedef struct prism_layer_config {
     uint32_t mixer;            /* PRISM_MIXER_* */
@@ -374,9 +384,15 @@ typedef struct prism_layer_config {
     uint32_t rot_pairs;        /* latent: pairs (i, i + rot_pairs) of it that turn; the rest passes */
     const float *rot_freq;     /* latent: [rot_pairs] angle per position */
     float rot_mul;             /* latent: factor of cos and sin */
-    float scale;               /* latent: factor of the scores */
-    uint32_t window;           /* latent: positions i - window + 1 .. i are visible; 0: all up to i */
-    uint32_t ff;               /* dense feed-forward size; 0: none */
+    float scale;               /* latent, attention: factor of the scores */
+    uint32_t window;           /* latent, attention: positions i - window + 1 .. i are visible; 0: all up to i */
+    uint32_t kv_heads;         /* attention: key/value heads; gated delta: query/key heads */
+    uint32_t conv;             /* gated delta: taps of the short convolutions */
+    const struct prism_layer_config *left, *right;  /* pair: its mixers (only the mixer fields are read) */
+    uint32_t ff;               /* feed-forward size (of one expert); 0: none */
+    uint32_t experts;          /* 0: a dense feed-forward with biases and GELU; else experts without, squared ReLU */
+    uint32_t top;              /* experts a token goes through: largest sigmoid score plus correction, weighted by the score */
+    uint32_t expert_groups, groups_keep;  /* groups of neighbouring experts, ranked by their two best; 0 or equal: no choice of groups */
 } prism_layer_config;
 
 typedef struct prism_layered_config {
@@ -384,14 +400,20 @@ typedef struct prism_layered_config {
     float norm_eps, residual_mult, logit_scale;
     uint32_t dtype;            /* PRISM_DTYPE_* */
     uint32_t max_seq, max_batch;
+    uint32_t arrangement;      /* PRISM_ARRANGE_*; the options below belong to the sequential one */
+    float norm_offset;         /* norm weights are stored minus this (the layers' norms and the final one) */
+    uint32_t canon_taps;       /* causal convolution added to the input of each sublayer; 0: none */
+    uint32_t gated_residual;   /* results are multiplied by sigmoid(W h + b) */
+    uint32_t depth_average;    /* what a layer hands on is a weighted sum of the embedding and all layers' results */
+    uint32_t max_positions;    /* rows of the learned position table; 0: none (max_seq may not exceed it) */
 } prism_layered_config;
 
 /* The arrays inside the layer configs are copied.  Prompt portions go through the layers in chunks of the
  * context's "layered_chunk" option at the time of this call (windowed caches are sized by it). */
 int prism_cuda_engine_create_layered(prism_cuda_ctx *ctx, const prism_layered_config *cfg, const prism_layer_config *layers,
                                      prism_cuda_engine **out);
-/* Sets one tensor by its checkpoint name ("embed", "l0.norm1", "l0.mix.q", "l0.mlp.up.b", "final.norm", "head",
- * ...) from bf16 bit patterns, row-major; a vector is rows x 1 (or 1 x n).  PRISM_E_NOTFOUND for a name the
+/* Sets one tensor by its checkpoint name ("embed", "pos", "l0.norm1", "l0.mix.q", "l0.mix.right.q.conv", "l0.mlp.up.b",
+ * "l0.mlp.e3.down", "final.norm", "head", ...) from bf16 bit patterns, row-major; a vector is rows x 1 (or 1 x n).  PRISM_E_NOTFOUND for a name the
  * configuration has no place for. */
 int prism_cuda_engine_set_tensor(prism_cuda_engine *eng, const char *name, const uint16_t *bf16, uint64_t rows, uint64_t cols);
 /* Every tensor of a .safetensors file (bf16) into the engine; fails when a tensor has no place, a wrong shape

@@ -1,4 +1,4 @@
-"""Plain, slow restatement of the layer-list models (Mefipel), one numpy function per mechanism.
+"""Plain, slow restatement of the layer-list models (Mefipel, Tozarax), one numpy function per mechanism.
 
 The tests compare the layered engine with it; it shares nothing with the product: it reads the same
 config.json keys and tensor names, works in numpy at the precision of ``dt`` (float64 by default) and
@@ -112,11 +112,128 @@ def latent_attention(h, w, mx, eps):
     return o @ w["o"].T
 
 
-MIXERS = {"lightning": lightning, "latent_attention": latent_attention}
+def attention(h, w, mx, eps):
+    """Grouped softmax attention without rotation; a window counts the token itself."""
+    T, H, G, D, V = h.shape[0], mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
+    q = (h @ w["q"].T).reshape(T, H, D)
+    k = (h @ w["k"].T).reshape(T, G, D)
+    v = (h @ w["v"].T).reshape(T, G, V)
+    size = (mx.get("mask") or {}).get("size")
+    out = np.zeros((T, H, V), h.dtype)
+    for n in range(H):
+        g = n // (H // G)
+        for i in range(T):
+            lo = min(j for j in range(i + 1) if window_visible(i, j, size))
+            s = k[lo:i + 1, g] @ q[i, n] * mx["scale"]
+            p = np.exp(s - s.max())
+            out[i, n] = (p / p.sum()) @ v[lo:i + 1, g]
+    return out.reshape(T, H * V) @ w["o"].T
+
+
+def causal_conv(x, w):
+    """Per channel: w's last column meets the current token, zeros before the first."""
+    T, taps = x.shape[0], w.shape[1]
+    y = np.zeros_like(x)
+    for j in range(taps):
+        back = taps - 1 - j
+        if back < T:
+            y[back:] += w[:, j] * x[:T - back]
+    return y
+
+
+def softplus(z):
+    return np.logaddexp(0.0, z)
+
+
+def unit(x):
+    return x / np.sqrt(np.sum(x * x, axis=-1, keepdims=True) + 1e-6)
+
+
+def gated_delta(h, w, mx, eps):
+    """Delta rule with one decay and one step size per head and token, token by token."""
+    T, H, G, D, V = h.shape[0], mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
+    short = lambda n: silu(causal_conv(h @ w[n].T, w[n + ".conv"]))  # noqa: E731
+    q = unit(short("q").reshape(T, G, D)) * D ** -0.5
+    k = unit(short("k").reshape(T, G, D))
+    v = short("v").reshape(T, H, V)
+    beta = sigmoid(h @ w["b"].T)
+    decay = np.exp(-np.exp(w["A_log"]) * softplus(h @ w["a"].T + w["dt_bias"]))
+    o = np.empty((T, H, V), h.dtype)
+    for n in range(H):
+        g, S = n // (H // G), np.zeros((D, V), h.dtype)
+        for t in range(T):
+            S = S * decay[t, n]
+            u = beta[t, n] * (v[t, n] - k[t, g] @ S)
+            S = S + np.outer(k[t, g], u)
+            o[t, n] = q[t, g] @ S
+    o = rms_norm(o, w["norm"], eps) * silu(h @ w["g"].T).reshape(T, H, V)
+    return o.reshape(T, H * V) @ w["o"].T
+
+
+def parallel(h, w, mx, eps):
+    """Two mixers on the same input; each result normed over the width, then their mean."""
+    left = attention(h, _sub(w, "left."), mx["left"], eps)
+    right = gated_delta(h, _sub(w, "right."), mx["right"], eps)
+    return 0.5 * (rms_norm(left, w["left.out"], eps) + rms_norm(right, w["right.out"], eps))
+
+
+MIXERS = {"lightning": lightning, "latent_attention": latent_attention, "attention": attention, "gated_delta": gated_delta,
+          "parallel": parallel}
 
 
 def dense_ff(h, w):
     return gelu_tanh(h @ w["up"].T + w["up.b"]) @ w["down"].T + w["down.b"]
+
+
+def route(z, correction, top, groups):
+    """Chosen experts of one token (best first) and their weights."""
+    s = sigmoid(z)
+    choice = s + correction
+    if groups:
+        per = len(z) // groups["count"]
+        score = [sum(sorted(choice[g * per:(g + 1) * per])[-2:]) for g in range(groups["count"])]
+        keep = sorted(range(groups["count"]), key=lambda g: (-score[g], g))[:groups["keep"]]
+        choice = np.array([c if e // per in keep else -np.inf for e, c in enumerate(choice)])
+    best = sorted(range(len(z)), key=lambda e: (-choice[e], e))[:top]
+    return best, s[best]
+
+
+def moe_ff(h, w, mlp):
+    """Sigmoid router with a correction that takes part in the choice only; experts with a squared relu."""
+    r, y = mlp["router"], np.zeros_like(h)
+    z = h @ w["router"].T
+    for t in range(h.shape[0]):
+        for e, weight in zip(*route(z[t], w["correction"], r["top"], r.get("groups"))):
+            y[t] += weight * (w[f"e{e}.down"] @ np.maximum(w[f"e{e}.up"] @ h[t], 0.0) ** 2)
+    return y
+
+
+# ---- a layer with sublayers one after the other -------------------------------------------------------
+def sublayer(x, w, p, n, eps, f):
+    """x plus the gated result of f on the convolved norm; n is "1" (mixer) or "2" (feed-forward)."""
+    h = rms_norm(x, 1.0 + w[p + "norm" + n], eps)
+    gate = sigmoid(h @ w[p + "rg" + n].T + w[p + "rg" + n + ".b"])
+    return x + gate * f(h + causal_conv(h, w[p + "canon" + n]))
+
+
+def depth_average(w, history):
+    return sum(a * x for a, x in zip(w, history))
+
+
+def forward_sequential(cfg, weights, tokens, layers_out=None):
+    eps, n = cfg["norm"]["eps"], len(tokens)
+    x = weights["embed"][np.asarray(tokens)] + weights["pos"][:n]
+    history = [x]
+    for i, ly in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        x = sublayer(x, weights, p, "1", eps, lambda h: MIXERS[ly["type"]](h, _sub(weights, p + "mix."), ly["mixer"], eps))
+        if ly.get("mlp"):
+            x = sublayer(x, weights, p, "2", eps, lambda h: moe_ff(h, _sub(weights, p + "mlp."), ly["mlp"]))
+        history.append(x)
+        x = depth_average(weights[p + "dwa"], history)
+        if layers_out is not None:
+            layers_out.append(x)
+    return rms_norm(x, 1.0 + weights["final.norm"], eps) @ weights["head"].T
 
 
 # ---- the model -------------------------------------------------------------------------------------
@@ -128,6 +245,8 @@ def _sub(weights, prefix):
 def forward(cfg, weights, tokens, dt=np.float64, layers_out=None):
     """Logits [tokens, vocab] of one sequence; ``layers_out`` (a list) receives the residual after every layer."""
     weights = {k: np.asarray(v, dt) for k, v in weights.items()}
+    if cfg["architecture"] == "Tozarax":
+        return forward_sequential(cfg, weights, tokens, layers_out)
     eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
     x = weights["embed"][np.asarray(tokens)]
     for i, ly in enumerate(cfg["layers"]):

@@ -43,7 +43,8 @@ class LayerConfig(C.Structure):
         ("mixer", C.c_uint32), ("heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32),
         ("decay", C.POINTER(C.c_float)), ("q_rank", C.c_uint32), ("kv_rank", C.c_uint32), ("rot_dim", C.c_uint32),
         ("rot_pairs", C.c_uint32), ("rot_freq", C.POINTER(C.c_float)), ("rot_mul", C.c_float), ("scale", C.c_float),
-        ("window", C.c_uint32), ("ff", C.c_uint32),
+        ("window", C.c_uint32), ("kv_heads", C.c_uint32), ("conv", C.c_uint32), ("left", C.c_void_p), ("right", C.c_void_p),
+        ("ff", C.c_uint32), ("experts", C.c_uint32), ("top", C.c_uint32), ("expert_groups", C.c_uint32), ("groups_keep", C.c_uint32),
     ]
 
 
@@ -53,7 +54,8 @@ class LayeredModelConfig(C.Structure):
     _fields_ = [
         ("vocab", C.c_uint32), ("width", C.c_uint32), ("num_layers", C.c_uint32), ("norm_eps", C.c_float),
         ("residual_mult", C.c_float), ("logit_scale", C.c_float), ("dtype", C.c_uint32), ("max_seq", C.c_uint32),
-        ("max_batch", C.c_uint32),
+        ("max_batch", C.c_uint32), ("arrangement", C.c_uint32), ("norm_offset", C.c_float), ("canon_taps", C.c_uint32),
+        ("gated_residual", C.c_uint32), ("depth_average", C.c_uint32), ("max_positions", C.c_uint32),
     ]
 
 

@@ -35,12 +35,12 @@ int launch_dense_pack(prism_cuda_ctx *ctx, const DenseLinear &l, const bf16 *src
     return after_launch(ctx, "dense_pack_kernel");
 }
 
-__global__ void bf16_to_f32_kernel(const bf16 *__restrict__ src, float *__restrict__ dst, size_t n) {
+__global__ void bf16_to_f32_kernel(const bf16 *__restrict__ src, float *__restrict__ dst, size_t n, float add, uint32_t cols, uint32_t pitch) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) dst[i] = __bfloat162float(src[i]);
+    if (i < n) dst[i % cols * pitch + i / cols] = __bfloat162float(src[i]) + add;
 }
-int launch_bf16_to_f32(prism_cuda_ctx *ctx, const bf16 *src, float *dst, size_t n) {
-    bf16_to_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(src, dst, n);
+int launch_bf16_to_f32(prism_cuda_ctx *ctx, const bf16 *src, float *dst, size_t n, float add, uint32_t cols, uint32_t pitch) {
+    bf16_to_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(src, dst, n, add, cols, pitch);
     return after_launch(ctx, "bf16_to_f32_kernel");
 }
 
@@ -80,7 +80,8 @@ DenseEpi dense_epi(const DenseLinear &l, const DenseOut *outs) {
     DenseEpi e{};
     e.n = l.n_segs;
     for (uint32_t i = 0; i < l.n_segs; i++)
-        e.s[i] = DenseEpiSeg{l.seg[i].row0, l.seg[i].rows, l.seg[i].act, outs[i].store, outs[i].pitch, l.seg[i].mul, l.seg[i].bias, outs[i].p};
+        e.s[i] = DenseEpiSeg{l.seg[i].row0, l.seg[i].rows, l.seg[i].act, outs[i].store, outs[i].pitch, l.seg[i].in,
+                             l.seg[i].k ? l.seg[i].k : l.k_pad, l.seg[i].mul, l.seg[i].bias, outs[i].p};
     return e;
 }
 
@@ -97,11 +98,17 @@ struct GemvArgs {
     uint32_t k8, n_groups, rows, ks;
     const void *x;
     uint32_t pitch, f32;
+    const bf16 *x2;
+    uint32_t pitch2;
     const float *norm_w;
     const bf16 *gate;
     uint32_t gate_pitch, n_norm, norm_pad, norm_vec;  // norm_pad: n_norm rounded up to 64; norm_vec: rows allow 4-value accesses
     float eps;
     DenseEpi epi;
+    // experts: the stack's row tiles per expert, the plan, whether input rows are pairs
+    uint32_t n_tiles, by_pair;
+    const uint32_t *n_active, *active;
+    const int32_t *pair_of;
 };
 constexpr int GV_THREADS = 256, GV_WARPS = 8, GV_U = 4, GV_KS_MAX = 4;
 
@@ -187,8 +194,11 @@ struct GemvNorm {
     }
 };
 
-template <bool NORM>
+// MOE: items are blocks of 32 rows of the experts in use; every token column is multiplied, the pairs are stored.
+enum GemvKind { GV_PLAIN = 0, GV_NORM = 1, GV_MOE = 2 };
+template <int KIND>
 __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArgs a) {
+    constexpr bool NORM = KIND == GV_NORM, MOE = KIND == GV_MOE;
     extern __shared__ __align__(16) uint8_t dsm[];
     __shared__ float red[GV_WARPS][8][33];
     __shared__ float peer[GV_KS_MAX][8][32];  // rank 0: sums of the other ranks
@@ -199,21 +209,27 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
     const uint32_t rank = a.ks > 1 ? cluster.block_rank() : 0;
     if (a.ks > 1) asm volatile("barrier.cluster.arrive.release.aligned;\n" ::: "memory");  // met before the first remote store
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g8 = lane >> 2, t4 = lane & 3;
-    const uint32_t all_steps = a.k8 / 4, norm8 = NORM ? a.norm_pad / 8 : 0;
-    const uint32_t first = all_steps * rank / a.ks, steps = all_steps * (rank + 1) / a.ks;  // this rank's k range
-    const bool tok_on = g8 < a.rows;
-    const uint4 *xg = reinterpret_cast<const uint4 *>(reinterpret_cast<const bf16 *>(a.x) + (size_t)g8 * a.pitch);
+    const uint32_t norm8 = NORM ? a.norm_pad / 8 : 0;
     const uint4 *xl = reinterpret_cast<const uint4 *>(xs + (size_t)g8 * a.norm_pad);
     uint4 w[GV_U][4];
-    auto locate = [&](uint32_t grp, uint32_t &sg, uint32_t &rb) -> const uint4 * {  // segment, block of 32 rows inside it, first unit
+    uint32_t sg = 0, rb = 0, act = 0, first = 0, steps = 0;  // segment, block of 32 rows inside it, expert in use, this rank's k range
+    auto locate = [&](uint32_t grp) -> const uint4 * {       // first unit
+        uint32_t tile0 = 0;
         sg = 0;
         rb = grp;
+        if (MOE) {
+            act = grp / a.n_groups;
+            rb = grp % a.n_groups;
+            tile0 = a.active[act] * a.n_tiles;
+        }
         while (sg + 1 < a.epi.n && rb >= (a.epi.s[sg].rows + 31) / 32) {
             rb -= (a.epi.s[sg].rows + 31) / 32;
             sg++;
         }
-        const uint32_t row = a.epi.s[sg].row0 + rb * 32;
-        return a.w + (size_t)(row >> 7) * a.k8 * 128 + (row & 127) + g8;
+        const uint32_t row = a.epi.s[sg].row0 + rb * 32, all = a.epi.s[sg].k / 32;
+        first = all * rank / a.ks;
+        steps = all * (rank + 1) / a.ks;
+        return a.w + (size_t)(tile0 + (row >> 7)) * a.k8 * 128 + (row & 127) + g8;
     };
     auto load = [&](const uint4 *wt, uint32_t s0) {
 #pragma unroll
@@ -226,17 +242,27 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
             }
         }
     };
-    uint32_t sg, rb;
     const uint32_t grp0 = blockIdx.x / a.ks;
-    const uint4 *wt = locate(grp0, sg, rb);
-    load(wt, first + warp);  // weights do not depend on the previous kernel; the input does
+    uint32_t n_items = a.n_groups;
+    const uint4 *wt = nullptr;
+    bool loaded = !MOE;
+    if (!MOE) {
+        wt = locate(grp0);
+        load(wt, first + warp);  // weights do not depend on the previous kernel; the input does
+    }
     GemvNorm norm;
     if (NORM) norm.prefetch(a);
     pdl_wait();
     if (NORM) norm.stage(a, xs, sh);
-    bool loaded = true;
-    for (uint32_t grp = grp0; grp < a.n_groups; grp += gridDim.x / a.ks) {
-        if (!loaded) wt = locate(grp, sg, rb);
+    if (MOE) n_items *= *reinterpret_cast<const volatile uint32_t *>(a.n_active);
+    if (MOE && a.ks > 1 && grp0 >= n_items) asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");  // nothing to do for this cluster
+    for (uint32_t grp = grp0; grp < n_items; grp += gridDim.x / a.ks) {
+        if (!loaded) wt = locate(grp);
+        const int32_t pair = MOE ? a.pair_of[act * DENSE_GEMV_ROWS + g8] : 0;
+        const bool tok_on = MOE ? g8 < a.rows && pair >= 0 : g8 < a.rows;
+        const uint32_t x_row = MOE && a.by_pair ? (uint32_t)pair : g8;
+        const uint4 *xg = !MOE && a.epi.s[sg].in ? reinterpret_cast<const uint4 *>(a.x2 + (size_t)g8 * a.pitch2)
+                                                 : reinterpret_cast<const uint4 *>(reinterpret_cast<const bf16 *>(a.x) + (size_t)x_row * a.pitch);
         float acc[2][4] = {};
         for (uint32_t s0 = first + warp; s0 < steps; s0 += GV_WARPS * GV_U) {
             if (!loaded) load(wt, s0);
@@ -275,7 +301,8 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
             if (rank) return;
             for (uint32_t r = 1; r < a.ks; r++) v += peer[r][t][lane];
         }
-        if (t < a.rows && rl < a.epi.s[sg].rows) dense_store<bf16>(a.epi.s[sg], rl, t, v);
+        const int32_t out_row = MOE ? a.pair_of[act * DENSE_GEMV_ROWS + t] : (int32_t)t;
+        if (t < a.rows && out_row >= 0 && rl < a.epi.s[sg].rows) dense_store<bf16>(a.epi.s[sg], rl, (uint32_t)out_row, v);
         __syncthreads();
     }
 }
@@ -287,38 +314,60 @@ constexpr size_t GV_SMEM_MAX = 160 * 1024;
 constexpr uint32_t GV_FOLD_ROWS = 2;  // as many as GemvNorm splits the block into; more rows: every CTA norming all of them costs more than a norm kernel does
 
 bool dense_gemv_ok(const DenseIn &in, uint32_t rows) {
-    return rows <= DENSE_GEMV_ROWS && (in.norm_w ? rows <= GV_FOLD_ROWS && gemv_smem(in, rows) <= GV_SMEM_MAX : !in.f32) &&
+    return rows <= DENSE_GEMV_ROWS && !(in.x2 && in.pitch2 % 8) && (in.norm_w ? rows <= GV_FOLD_ROWS && gemv_smem(in, rows) <= GV_SMEM_MAX : !in.f32) &&
            (in.f32 || in.pitch % 8 == 0);
 }
 
-int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows) {
+// Few row blocks and a long k: a block's k range is shared inside a cluster, at least GV_WARPS * GV_U steps each.
+static uint32_t gemv_cluster(prism_cuda_ctx *ctx, uint32_t blocks, uint32_t k8) {
+    const uint32_t slots = 2u * (uint32_t)ctx->sm_count;
+    uint32_t ks = 1;
+    while (ks < GV_KS_MAX && blocks * ks * 2 <= slots + slots / 2 && k8 / 4 >= ks * 2 * GV_WARPS * GV_U) ks *= 2;
+    return ks;
+}
+static GemvArgs gemv_args(const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows) {
     GemvArgs a{};
     a.w = reinterpret_cast<const uint4 *>(l.w);
     a.k8 = l.k_pad / 8;
     a.rows = rows;
     a.x = in.x; a.pitch = in.pitch; a.f32 = in.f32;
+    a.x2 = reinterpret_cast<const bf16 *>(in.x2); a.pitch2 = in.pitch2;
+    a.epi = dense_epi(l, outs);
+    for (uint32_t s = 0; s < l.n_segs; s++) a.n_groups += (l.seg[s].rows + 31) / 32;
+    return a;
+}
+
+int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows) {
+    GemvArgs a = gemv_args(l, in, outs, rows);
     a.norm_w = in.norm_w; a.n_norm = in.n_norm; a.norm_pad = round_up_u32(in.n_norm, 64); a.eps = in.eps;
     a.gate = reinterpret_cast<const bf16 *>(in.gate); a.gate_pitch = in.gate_pitch;
     a.norm_vec = !((reinterpret_cast<uintptr_t>(in.x) | reinterpret_cast<uintptr_t>(in.gate) | reinterpret_cast<uintptr_t>(in.norm_w)) & 15) &&
                  !((in.pitch | in.n_norm | (in.gate ? in.gate_pitch : 0)) & 3);
-    a.epi = dense_epi(l, outs);
-    for (uint32_t s = 0; s < l.n_segs; s++) a.n_groups += (l.seg[s].rows + 31) / 32;
-    // few row blocks and a long k: share a block's k range inside a cluster, at least GV_WARPS * GV_U steps each
-    const uint32_t slots = 2u * (uint32_t)ctx->sm_count;
-    a.ks = 1;
-    while (a.ks < GV_KS_MAX && a.n_groups * a.ks * 2 <= slots + slots / 2 && a.k8 / 4 >= a.ks * 2 * GV_WARPS * GV_U) a.ks *= 2;
+    a.ks = gemv_cluster(ctx, a.n_groups, a.k8);
     const size_t smem = gemv_smem(in, rows);
-    const uint32_t grid = a.ks > 1 ? a.n_groups * a.ks : std::min(a.n_groups, slots);
+    const uint32_t grid = a.ks > 1 ? a.n_groups * a.ks : std::min(a.n_groups, 2u * (uint32_t)ctx->sm_count);
     if (in.norm_w) {
         static bool configured[PRISM_MAX_DEVICES] = {false};
         if (!configured[ctx->device]) {
-            PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemv_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GV_SMEM_MAX));
+            PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(dense_gemv_kernel<GV_NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GV_SMEM_MAX));
             configured[ctx->device] = true;
         }
-        launch_cluster_pdl(ctx, dense_gemv_kernel<true>, grid, GV_THREADS, smem, a.ks, a);
+        launch_cluster_pdl(ctx, dense_gemv_kernel<GV_NORM>, grid, GV_THREADS, smem, a.ks, a);
     } else {
-        launch_cluster_pdl(ctx, dense_gemv_kernel<false>, grid, GV_THREADS, 0, a.ks, a);
+        launch_cluster_pdl(ctx, dense_gemv_kernel<GV_PLAIN>, grid, GV_THREADS, 0, a.ks, a);
     }
+    return after_launch(ctx, "dense_gemv_kernel");
+}
+
+int launch_moe_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const MoePlan &plan, const DenseIn &in, bool by_pair, const DenseOut &out, uint32_t tokens) {
+    if (tokens > DENSE_GEMV_ROWS || l.n_segs != 1 || in.pitch % 8) return fail(ctx, PRISM_E_ARG, "experts: too many tokens for the small-batch kernel");
+    GemvArgs a = gemv_args(l, in, &out, tokens);
+    a.n_tiles = l.n_tiles; a.by_pair = by_pair;
+    a.n_active = plan.n_active; a.active = plan.active; a.pair_of = plan.pair_of;
+    const uint32_t items = a.n_groups * std::min(tokens * plan.top, plan.experts);  // at most
+    a.ks = gemv_cluster(ctx, items, a.k8);
+    const uint32_t grid = a.ks > 1 ? items * a.ks : std::min(items, 2u * (uint32_t)ctx->sm_count);
+    launch_cluster_pdl(ctx, dense_gemv_kernel<GV_MOE>, grid, GV_THREADS, 0, a.ks, a);
     return after_launch(ctx, "dense_gemv_kernel");
 }
 
@@ -327,27 +376,38 @@ int launch_dense_gemv(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &
 struct F32Args {
     const bf16 *w;
     uint32_t k_pad, rows;
-    const float *x;
-    uint32_t pitch;
+    const float *x, *x2;
+    uint32_t pitch, pitch2;
     DenseEpi epi;
+    uint32_t n_tiles, experts;  // experts: rows are sorted by expert
+    const uint32_t *count;
 };
 constexpr int F32_BK = 16;
+template <bool MOE>
 __global__ void __launch_bounds__(256) dense_f32_kernel(const F32Args a) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float ws[F32_BK][68], xs[F32_BK][68];
-    const uint32_t tid = threadIdx.x, row0 = blockIdx.x * 64, t0 = blockIdx.y * 64;
-    uint32_t sg = 0;
-    while (sg + 1 < a.epi.n && row0 >= a.epi.s[sg + 1].row0) sg++;
-    if (row0 >= a.epi.s[sg].row0 + a.epi.s[sg].rows) return;  // padding
+    const uint32_t tid = threadIdx.x, row0 = blockIdx.x * 64;
+    uint32_t t0 = blockIdx.y * 64, t_end = a.rows, tile0 = 0;
+    if (MOE) {
+        uint32_t expert, left;
+        if (!moe_find_tile(a.count, a.experts, 64, blockIdx.y, expert, t0, left)) return;  // the same in every warp
+        tile0 = expert * a.n_tiles;
+        t_end = t0 + left;
+    }
+    const DenseEpiSeg &seg = dense_seg(a.epi, row0);
+    if (row0 >= seg.row0 + seg.rows) return;                  // padding
+    const float *x = seg.in ? a.x2 : a.x;
+    const uint32_t pitch = seg.in ? a.pitch2 : a.pitch;
     const uint32_t tx = tid & 15, ty = tid >> 4;              // rows tx*4.., tokens ty*4..
     float acc[4][4] = {};
-    for (uint32_t k0 = 0; k0 < a.k_pad; k0 += F32_BK) {
+    for (uint32_t k0 = 0; k0 < seg.k; k0 += F32_BK) {
         for (uint32_t i = tid; i < 64 * F32_BK; i += 256) {
             const uint32_t r = i / F32_BK, k = i % F32_BK;
             const uint32_t row = row0 + r, kk = k0 + k;
-            ws[k][r] = __bfloat162float(a.w[(((size_t)(row >> 7) * (a.k_pad / 8) + (kk >> 3)) * 128 + (row & 127)) * 8 + (kk & 7)]);
-            xs[k][r] = t0 + r < a.rows && kk < a.pitch ? a.x[(size_t)(t0 + r) * a.pitch + kk] : 0.0f;
+            ws[k][r] = __bfloat162float(a.w[(((size_t)(tile0 + (row >> 7)) * (a.k_pad / 8) + (kk >> 3)) * 128 + (row & 127)) * 8 + (kk & 7)]);
+            xs[k][r] = t0 + r < t_end && kk < pitch ? x[(size_t)(t0 + r) * pitch + kk] : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -364,13 +424,19 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const F32Args a) {
     }
     for (int j = 0; j < 4; j++)
         for (int i = 0; i < 4; i++) {
-            const uint32_t rl = row0 + tx * 4 + i - a.epi.s[sg].row0, t = t0 + ty * 4 + j;
-            if (rl < a.epi.s[sg].rows && t < a.rows) dense_store<float>(a.epi.s[sg], rl, t, acc[i][j]);
+            const uint32_t rl = row0 + tx * 4 + i - seg.row0, t = t0 + ty * 4 + j;
+            if (rl < seg.rows && t < t_end) dense_store<float>(seg, rl, t, acc[i][j]);
         }
 }
-int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const float *x, uint32_t pitch, const DenseOut *outs, uint32_t rows) {
-    F32Args a{l.w, l.k_pad, rows, x, pitch, dense_epi(l, outs)};
-    launch_pdl(ctx, "dense_f32_kernel", dense_f32_kernel, dim3(l.n_tiles * 2, (rows + 63) / 64), 256, 0, a);
+int launch_dense_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const DenseIn &in, const DenseOut *outs, uint32_t rows) {
+    F32Args a{l.w, l.k_pad, rows, (const float *)in.x, (const float *)in.x2, in.pitch, in.pitch2, dense_epi(l, outs), l.n_tiles, 1, nullptr};
+    launch_pdl(ctx, "dense_f32_kernel", dense_f32_kernel<false>, dim3(l.n_tiles * 2, (rows + 63) / 64), 256, 0, a);
+    return after_launch(ctx, "dense_f32_kernel");
+}
+int launch_moe_f32(prism_cuda_ctx *ctx, const DenseLinear &l, const MoePlan &plan, const DenseIn &in, const DenseOut &out, uint32_t pairs) {
+    F32Args a{l.w, l.k_pad, pairs, (const float *)in.x, nullptr, in.pitch, 0, dense_epi(l, &out), l.n_tiles, plan.experts, plan.count};
+    const uint32_t tiles = pairs / 64 + std::min(pairs, plan.experts);  // at most
+    launch_pdl(ctx, "dense_f32_kernel", dense_f32_kernel<true>, dim3(l.n_tiles * 2, tiles), 256, 0, a);
     return after_launch(ctx, "dense_f32_kernel");
 }
 
@@ -439,15 +505,20 @@ int launch_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t 
 }
 
 __global__ void dense_embed_kernel(const bf16 *__restrict__ table, uint32_t width, uint32_t vocab, const uint32_t *__restrict__ tokens,
-                                   float *__restrict__ x) {
+                                   float *__restrict__ x, const bf16 *__restrict__ pos_table, uint32_t max_pos, const RowMap map, float *__restrict__ x2) {
     pdl_launch_dependents();
     pdl_wait();
-    const uint32_t tok = min(tokens[blockIdx.x], vocab - 1);  // the host rejects larger ids before the launch
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x)
-        x[(size_t)blockIdx.x * width + i] = __bfloat162float(table[(size_t)tok * width + i]);
+    const uint32_t r = blockIdx.x, tok = min(tokens[r], vocab - 1);  // the host rejects larger ids before the launch
+    const bf16 *pt = pos_table ? pos_table + (size_t)min((uint32_t)map.pos_of(r), max_pos - 1) * width : nullptr;  // and later positions
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = __bfloat162float(table[(size_t)tok * width + i]) + (pt ? __bfloat162float(pt[i]) : 0.0f);
+        x[(size_t)r * width + i] = v;
+        if (x2) x2[(size_t)r * width + i] = v;
+    }
 }
-int launch_dense_embed(prism_cuda_ctx *ctx, const bf16 *table, uint32_t width, uint32_t vocab, const uint32_t *tokens, uint32_t rows, float *x) {
-    launch_pdl(ctx, "dense_embed_kernel", dense_embed_kernel, rows, 256, 0, table, width, vocab, tokens, x);
+int launch_dense_embed(prism_cuda_ctx *ctx, const bf16 *table, uint32_t width, uint32_t vocab, const uint32_t *tokens, uint32_t rows, float *x,
+                       const bf16 *pos_table, uint32_t max_pos, const RowMap &map, float *x2) {
+    launch_pdl(ctx, "dense_embed_kernel", dense_embed_kernel, rows, 256, 0, table, width, vocab, tokens, x, pos_table, max_pos, map, x2);
     return after_launch(ctx, "dense_embed_kernel");
 }
 

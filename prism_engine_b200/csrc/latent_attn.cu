@@ -3,7 +3,8 @@
 //   rows     W_uk is folded into the query and W_uv applied to the weighted latent, so the cached latents
 //            themselves are scored and weighed (all heads share them): decode, short portions, and 32-bit;
 //   expanded a prompt portion expands keys and values of the positions it can see once (two stacked
-//            linears) and runs a tiled tensor-core attention over them.
+//            linears) and runs a tiled tensor-core attention over them (tiled_attn_kernel, which the
+//            grouped attention runs over its cache too).
 // The cache keeps [latent | rotated key] per position; a windowed layer's cache is a ring.
 #include <algorithm>
 #include <cmath>
@@ -15,15 +16,13 @@ namespace prism {
 __device__ __forceinline__ size_t cache_row(const LatentCache &c, int32_t slot, int32_t pos) {
     return ((size_t)slot * c.ring + (uint32_t)pos % c.ring) * c.pitch;
 }
-__device__ __forceinline__ int32_t first_key(const LatentArgs &a, int32_t pos) {
-    return a.window && pos + 1 > (int32_t)a.window ? pos + 1 - (int32_t)a.window : 0;
-}
+__device__ __forceinline__ int32_t first_key(const LatentArgs &a, int32_t pos) { return window_first(a.window, pos); }
 // Rotate-half of the pair (u, v) with index i at position pos.
-__device__ __forceinline__ void rotate_pair(const LatentArgs &a, int32_t pos, uint32_t i, float &u, float &v) {
+__device__ __forceinline__ void rotate_pair(const float *__restrict__ freq, float mul, int32_t pos, uint32_t i, float &u, float &v) {
     float s, c;
-    sincosf((float)pos * __ldg(a.rot_freq + i), &s, &c);
-    s *= a.rot_mul;
-    c *= a.rot_mul;
+    sincosf((float)pos * __ldg(freq + i), &s, &c);
+    s *= mul;
+    c *= mul;
     const float x = u * c - v * s, y = v * c + u * s;
     u = x;
     v = y;
@@ -48,7 +47,7 @@ __device__ __forceinline__ void append_row(const LatentArgs &a, const TA *__rest
     y += a.kv_rank;
     for (uint32_t i = threadIdx.x; i < a.rot_pairs; i += blockDim.x) {
         float u = ld_act(x + i), v = ld_act(x + a.rot_pairs + i);
-        rotate_pair(a, pos, i, u, v);
+        rotate_pair(a.rot_freq, a.rot_mul, pos, i, u, v);
         st_act(y + i, u);
         st_act(y + a.rot_pairs + i, v);
     }
@@ -131,7 +130,7 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const LatentArgs a, c
             if (c < 2 * a.rot_pairs) {
                 const uint32_t p = c < a.rot_pairs ? c : c - a.rot_pairs;
                 float u = ld_act(x + p), w = ld_act(x + a.rot_pairs + p);
-                rotate_pair(a, rows.pos_of(r0 + r), p, u, w);
+                rotate_pair(a.rot_freq, a.rot_mul, rows.pos_of(r0 + r), p, u, w);
                 v = c < a.rot_pairs ? u : w;
             } else if (c < a.rot_dim) {
                 v = ld_act(x + c);
@@ -420,52 +419,48 @@ int launch_latent_gather(prism_cuda_ctx *ctx, const LatentArgs &a, int32_t slot,
     return after_launch(ctx, "latent_gather_kernel");
 }
 
-struct LatentPrefill {
-    LatentArgs a;
-    const bf16 *q, *kx, *vx, *krot, *gate;
-    bf16 *out;
-    uint32_t q_pitch, kx_pitch, vx_pitch, gate_pitch, out_pitch;
-    uint32_t lo, pos0, n_rows;  // first expanded position, first query position, queries
-};
 constexpr int LP_Q = 128, LP_K = 64, LP_THREADS = 256;
-static size_t latent_prefill_smem(const LatentArgs &a, uint32_t vd) {
+static size_t tiled_attn_smem(const TiledAttn &a, uint32_t vd) {
     const uint32_t dq = round_up_u32(a.dim + a.rot_dim, 16);
     return ((size_t)(LP_Q + 2 * LP_K) * (dq + 8) + (size_t)2 * LP_K * (vd + 8)) * 2;
 }
 
 // 128 queries of one head per CTA (16 per warp), key tiles of 64 in two buffers, online softmax in fp32; the
-// weights enter the second product as two bf16 parts.
+// weights enter the second product as two bf16 parts.  Key and value heads start at multiples of 8 and may be
+// shared by a group of query heads; rows of a ring are taken by position.
 template <int VD>
-__global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const LatentPrefill p) {
+__global__ void __launch_bounds__(LP_THREADS) tiled_attn_kernel(const TiledAttn a) {
     extern __shared__ __align__(16) uint8_t lps[];
     pdl_launch_dependents();
     pdl_wait();
-    const LatentArgs &a = p.a;
-    const uint32_t h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+    const uint32_t h = blockIdx.y, kh = h / a.group, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
     const uint32_t dq = a.dim + a.rot_dim, dqp = round_up_u32(dq, 16), PQ = dqp + 8;
     constexpr uint32_t PV = VD + 8;
     bf16 *Qs = reinterpret_cast<bf16 *>(lps), *Ks = Qs + LP_Q * PQ, *Vs = Ks + 2 * LP_K * PQ;
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(Qs), sK = (uint32_t)__cvta_generic_to_shared(Ks), sV = (uint32_t)__cvta_generic_to_shared(Vs);
-    const uint32_t q0 = blockIdx.x * LP_Q, nq = min((uint32_t)LP_Q, p.n_rows - q0);
-    const int32_t first = max((int32_t)p.lo, first_key(a, (int32_t)(p.pos0 + q0)));
-    const int32_t end = (int32_t)(p.pos0 + q0 + nq);  // keys first .. end-1
+    const uint32_t q0 = blockIdx.x * LP_Q, nq = min((uint32_t)LP_Q, a.n_rows - q0);
+    const int32_t first = max((int32_t)a.lo, window_first(a.window, (int32_t)(a.pos0 + q0)));
+    const int32_t end = (int32_t)(a.pos0 + q0 + nq);  // keys first .. end-1
     const uint32_t n_kt = ((uint32_t)(end - first) + LP_K - 1) / LP_K;
     const uint4 z4 = make_uint4(0, 0, 0, 0);
-    const uint32_t d8 = a.dim / 8, r8 = a.rot_dim / 8, q8 = dqp / 8, v8 = a.vdim / 8;
+    const uint32_t d8 = (a.dim + 7) / 8, r8 = a.rot_dim / 8, q8 = dqp / 8, v8 = (a.vdim + 7) / 8;
+    const bool q_vec = !((a.dim | a.q_pitch) & 7) && !(reinterpret_cast<uintptr_t>(a.q) & 15);
 
     auto load_keys = [&](uint32_t kt, uint32_t buf) {
         const int32_t k0 = first + (int32_t)(kt * LP_K);
+        const uint32_t row0 = a.ring ? (uint32_t)k0 % a.ring : (uint32_t)k0 - a.lo;
+        auto row_of = [&](uint32_t r) { return a.ring && row0 + r >= a.ring ? row0 + r - a.ring : row0 + r; };  // the visible keys fit into the ring
         for (uint32_t i = tid; i < LP_K * q8; i += LP_THREADS) {
             const uint32_t r = i / q8, c = i % q8, at = (buf * LP_K + r) * PQ + c * 8;
             const int32_t key = k0 + (int32_t)r;
-            if (key < end && c < d8) cp_async16(sK + at * 2, p.kx + (size_t)(key - (int32_t)p.lo) * p.kx_pitch + h * a.dim + c * 8);
-            else if (key < end && c < d8 + r8) cp_async16(sK + at * 2, p.krot + (size_t)(key - (int32_t)p.lo) * a.rot_dim + (c - d8) * 8);
+            if (key < end && c < d8) cp_async16(sK + at * 2, a.kx + (size_t)row_of(r) * a.kx_pitch + kh * a.kx_head + c * 8);
+            else if (key < end && c < d8 + r8) cp_async16(sK + at * 2, a.krot + (size_t)row_of(r) * a.rot_dim + (c - d8) * 8);
             else *reinterpret_cast<uint4 *>(Ks + at) = z4;
         }
         for (uint32_t i = tid; i < LP_K * (VD / 8); i += LP_THREADS) {
             const uint32_t r = i / (VD / 8), c = i % (VD / 8), at = (buf * LP_K + r) * PV + c * 8;
             const int32_t key = k0 + (int32_t)r;
-            if (key < end && c < v8) cp_async16(sV + at * 2, p.vx + (size_t)(key - (int32_t)p.lo) * p.vx_pitch + h * a.vdim + c * 8);
+            if (key < end && c < v8) cp_async16(sV + at * 2, a.vx + (size_t)row_of(r) * a.vx_pitch + kh * a.vx_head + c * 8);
             else *reinterpret_cast<uint4 *>(Vs + at) = z4;
         }
         cp_async_commit();
@@ -473,8 +468,15 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const Latent
     load_keys(0, 0);
     for (uint32_t i = tid; i < LP_Q * q8; i += LP_THREADS) {
         const uint32_t r = i / q8, c = i % q8;
+        const bf16 *src = a.q + (size_t)(q0 + r) * a.q_pitch + h * dq + c * 8;
         uint4 x = z4;
-        if (r < nq && c < d8 + r8) x = *reinterpret_cast<const uint4 *>(p.q + (size_t)(q0 + r) * p.q_pitch + h * dq + c * 8);
+        if (r < nq && q_vec) {
+            if (c < d8 + r8) x = *reinterpret_cast<const uint4 *>(src);
+        } else if (r < nq) {
+#pragma unroll
+            for (uint32_t j = 0; j < 8; j++)
+                if (c * 8 + j < dq) reinterpret_cast<bf16 *>(&x)[j] = src[j];
+        }
         *reinterpret_cast<uint4 *>(Qs + r * PQ + c * 8) = x;
     }
     __syncthreads();
@@ -482,7 +484,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const Latent
         const uint32_t r = i / a.rot_pairs, j = i % a.rot_pairs;
         bf16 *u = Qs + r * PQ + a.dim + j, *v = u + a.rot_pairs;
         float x = __bfloat162float(*u), y = __bfloat162float(*v);
-        rotate_pair(a, (int32_t)(p.pos0 + q0 + r), j, x, y);
+        rotate_pair(a.rot_freq, a.rot_mul, (int32_t)(a.pos0 + q0 + r), j, x, y);
         *u = __float2bfloat16_rn(x);
         *v = __float2bfloat16_rn(y);
     }
@@ -493,7 +495,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const Latent
         for (int i = 0; i < 4; i++) acc[n][i] = 0.0f;
     float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.0f, 0.0f};
     const float sc2 = a.scale * 1.4426950408889634f;
-    const int32_t wq0 = (int32_t)(p.pos0 + q0 + warp * 16);  // positions of this warp's queries: wq0 .. wq0+15
+    const int32_t wq0 = (int32_t)(a.pos0 + q0 + warp * 16);  // positions of this warp's queries: wq0 .. wq0+15
     for (uint32_t kt = 0; kt < n_kt; kt++) {
         const uint32_t buf = kt & 1;
         if (kt + 1 < n_kt) {
@@ -504,7 +506,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const Latent
         }
         __syncthreads();
         const int32_t k0 = first + (int32_t)(kt * LP_K);
-        const bool none = k0 > wq0 + 15 || k0 + LP_K - 1 < first_key(a, wq0) || warp * 16 >= nq;
+        const bool none = k0 > wq0 + 15 || k0 + LP_K - 1 < window_first(a.window, wq0) || warp * 16 >= nq;
         if (!none) {
             float s[LP_K / 8][4];
 #pragma unroll
@@ -522,7 +524,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const Latent
                     mma_bf16(s[2 * n + 1], aq, b[2], b[3]);
                 }
             }
-            const bool edge = k0 + LP_K - 1 > wq0 || (a.window && k0 < first_key(a, wq0 + 15));
+            const bool edge = k0 + LP_K - 1 > wq0 || (a.window && k0 < window_first(a.window, wq0 + 15));
             float mx[2] = {mrow[0], mrow[1]};
 #pragma unroll
             for (int n = 0; n < LP_K / 8; n++)
@@ -588,40 +590,59 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const Latent
 #pragma unroll
         for (int n = 0; n < VD / 8; n++) {
             const uint32_t c = n * 8 + 2 * t4;
-            if (c < a.vdim) {  // vdim is a multiple of 8
-                const uint32_t at = h * a.vdim + c;
-                const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(p.gate + row * p.gate_pitch + at));
-                *reinterpret_cast<uint32_t *>(p.out + row * p.out_pitch + at) = pack_bf16(acc[n][2 * i] * inv * g.x, acc[n][2 * i + 1] * inv * g.y);
+            const uint32_t at = h * a.vdim + c;
+            float o0 = acc[n][2 * i] * inv, o1 = acc[n][2 * i + 1] * inv;
+            if (a.vdim & 1) {  // no gate
+                if (c < a.vdim) st_act(a.out + row * a.out_pitch + at, o0);
+                if (c + 1 < a.vdim) st_act(a.out + row * a.out_pitch + at + 1, o1);
+            } else if (c < a.vdim) {
+                if (a.gate) {
+                    const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(a.gate + row * a.gate_pitch + at));
+                    o0 *= g.x;
+                    o1 *= g.y;
+                }
+                *reinterpret_cast<uint32_t *>(a.out + row * a.out_pitch + at) = pack_bf16(o0, o1);
             }
         }
     }
 }
 
-bool latent_expand_ok(const LatentArgs &a) {
-    return a.dim % 8 == 0 && a.rot_dim % 8 == 0 && a.vdim % 8 == 0 && a.dim + a.rot_dim <= 256 && a.vdim <= 256;
-}
-
 template <int VD>
-static int launch_lp(prism_cuda_ctx *ctx, const LatentPrefill &p) {
+static int launch_ta(prism_cuda_ctx *ctx, const TiledAttn &p) {
     static bool configured[PRISM_MAX_DEVICES] = {false};
     if (!configured[ctx->device]) {
-        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(latent_prefill_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024));
+        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(tiled_attn_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024));
         configured[ctx->device] = true;
     }
-    launch_pdl(ctx, "latent_prefill_kernel", latent_prefill_kernel<VD>, dim3((p.n_rows + LP_Q - 1) / LP_Q, p.a.heads), LP_THREADS,
-               latent_prefill_smem(p.a, VD), p);
-    return after_launch(ctx, "latent_prefill_kernel");
+    launch_pdl(ctx, "tiled_attn_kernel", tiled_attn_kernel<VD>, dim3((p.n_rows + LP_Q - 1) / LP_Q, p.heads), LP_THREADS, tiled_attn_smem(p, VD), p);
+    return after_launch(ctx, "tiled_attn_kernel");
+}
+bool tiled_attn_ok(uint32_t dim, uint32_t vdim) { return dim <= 256 && vdim <= 256; }
+int launch_tiled_attn(prism_cuda_ctx *ctx, const TiledAttn &p) {
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(p.kx) | reinterpret_cast<uintptr_t>(p.vx) | reinterpret_cast<uintptr_t>(p.krot);
+    if (!tiled_attn_ok(p.dim + p.rot_dim, p.vdim) || (ptrs & 15) || p.kx_pitch % 8 || p.vx_pitch % 8 || p.kx_head % 8 || p.vx_head % 8 || p.rot_dim % 8 ||
+        (p.rot_dim && p.dim % 8) || p.out_pitch % 2 || (p.gate && (p.gate_pitch % 2 || p.vdim % 2)))
+        return fail(ctx, PRISM_E_ARG, "tiled attention: keys and values need 16-byte rows and heads of at most 256");
+    if (p.vdim <= 64) return launch_ta<64>(ctx, p);
+    if (p.vdim <= 128) return launch_ta<128>(ctx, p);
+    return launch_ta<256>(ctx, p);
+}
+
+bool latent_expand_ok(const LatentArgs &a) {
+    return a.dim % 8 == 0 && a.rot_dim % 8 == 0 && a.vdim % 8 == 0 && tiled_attn_ok(a.dim + a.rot_dim, a.vdim);
 }
 
 int launch_latent_prefill(prism_cuda_ctx *ctx, const LatentArgs &a, const bf16 *q, uint32_t q_pitch, const bf16 *kx, uint32_t kx_pitch,
                           const bf16 *vx, uint32_t vx_pitch, const bf16 *krot, uint32_t lo, const bf16 *gate, uint32_t gate_pitch, bf16 *out,
                           uint32_t out_pitch, uint32_t pos0, uint32_t n_rows) {
-    if (!latent_expand_ok(a) || q_pitch % 8 || kx_pitch % 8 || vx_pitch % 8 || gate_pitch % 2 || out_pitch % 2)
-        return fail(ctx, PRISM_E_ARG, "latent prefill: head sizes and row pitches must be multiples of 8");
-    const LatentPrefill p{a, q, kx, vx, krot, gate, out, q_pitch, kx_pitch, vx_pitch, gate_pitch, out_pitch, lo, pos0, n_rows};
-    if (a.vdim <= 64) return launch_lp<64>(ctx, p);
-    if (a.vdim <= 128) return launch_lp<128>(ctx, p);
-    return launch_lp<256>(ctx, p);
+    TiledAttn p{};
+    p.heads = a.heads; p.group = 1; p.dim = a.dim; p.rot_dim = a.rot_dim; p.rot_pairs = a.rot_pairs; p.vdim = a.vdim; p.window = a.window;
+    p.scale = a.scale; p.rot_mul = a.rot_mul; p.rot_freq = a.rot_freq;
+    p.q = q; p.kx = kx; p.vx = vx; p.krot = krot; p.gate = gate; p.out = out;
+    p.q_pitch = q_pitch; p.kx_pitch = kx_pitch; p.vx_pitch = vx_pitch; p.gate_pitch = gate_pitch; p.out_pitch = out_pitch;
+    p.kx_head = a.dim; p.vx_head = a.vdim;
+    p.lo = lo; p.pos0 = pos0; p.n_rows = n_rows;
+    return launch_tiled_attn(ctx, p);
 }
 
 }  // namespace prism

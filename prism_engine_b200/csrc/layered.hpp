@@ -10,18 +10,39 @@
 
 namespace prism {
 
-struct LayeredLayer {
+// One mixer of a layer.
+struct LayeredMixer {
     prism_layer_config c{};
-    DenseLinear in;      // everything that reads the layer's normed input: the mixer's projections, gate, feed-forward up
-    DenseLinear out;     // [W_o | W_down] along k: both sublayers' outputs, added into the residual
-    DenseLinear uq;      // latent: queries from the query latent
-    DenseLinear ukv;     // latent: keys | values from latents (prompt portions)
-    uint32_t seg_up = 0; // index of the feed-forward segment of `in`
-    uint32_t k_mix = 0;  // columns of the out input before the feed-forward part (mixer width rounded up to 64)
-    float *norm1 = nullptr, *mix_norm = nullptr, *dq_norm = nullptr, *up_b = nullptr, *down_b = nullptr, *decay = nullptr;
+    std::string name;         // prefix of its tensors
+    uint32_t seg0 = 0;        // its first segment of the layer's `in`
+    uint32_t col = 0;         // its first column in the rows of `cat`
+    DenseLinear uq;           // latent: queries from the query latent
+    DenseLinear ukv;          // latent: keys | values from latents (prompt portions)
+    float *mix_norm = nullptr, *dq_norm = nullptr, *decay = nullptr;
     float *state = nullptr;   // lightning: [slot][heads][dim][vdim]
     LatentArgs la{};          // latent: sizes, cache, row-major W_uk / W_uv
     uint32_t splits = 0;
+    GroupedArgs ga{};         // attention: sizes, cache
+    DeltaArgs da{};           // gated delta: sizes, small weights, state, ring
+    uint32_t conv_col[3] = {0, 0, 0};  // gated delta: columns of q, k, v in the convolved rows
+    float *out_norm = nullptr;         // pair: norm of its result
+    uint32_t width() const { return c.heads * c.vdim; }
+};
+
+struct LayeredLayer {
+    prism_layer_config c{};
+    std::vector<LayeredMixer> mix;  // two in a pair
+    DenseLinear in;      // everything that reads the first norm (sequential: convolved or not)
+    DenseLinear out;     // parallel: [W_o | W_down] along k, added into the residual; sequential: the mixers' W_o, each from its own columns
+    uint32_t seg_up = 0; // index of the feed-forward segment of `in` (sequential: of `in2`)
+    uint32_t k_mix = 0;  // columns of the out input before the feed-forward part (mixer width rounded up to 64)
+    float *norm1 = nullptr, *up_b = nullptr, *down_b = nullptr;
+    // sequential
+    DenseLinear in2;     // what reads the second norm: router or feed-forward up, gate
+    DenseLinear up, down;  // experts; dense: down alone
+    uint32_t seg_gate1 = 0, seg_gate2 = 0;
+    float *norm2 = nullptr, *canon1 = nullptr, *canon2 = nullptr, *gate1_b = nullptr, *gate2_b = nullptr, *correction = nullptr, *avg = nullptr;
+    void *ring1 = nullptr, *ring2 = nullptr;  // inputs of the two input convolutions, [slot][taps][width]
 };
 
 // Where a checkpoint tensor goes.
@@ -31,8 +52,11 @@ struct LayeredDst {
     uint32_t row0 = 0, k0 = 0;
     bf16 *rowmajor = nullptr;                      // also (or only) kept row-major, rows `pitch` apart
     uint32_t pitch = 0;
-    float *vec = nullptr;                          // fp32 copy of a vector
-    bool is_norm = false, bound = false;
+    float *vec = nullptr;                          // fp32 copy of a vector, or of a matrix transposed
+    uint32_t vec_pitch = 0;                        // between the rows of the transposed copy
+    float add = 0.0f;                              // added to the copy
+    float mean = 0.0f;                             // of synthetic values
+    bool bound = false;
 };
 
 struct LayeredModel {
@@ -40,7 +64,7 @@ struct LayeredModel {
     std::vector<LayeredLayer> layers;
     bool act32 = false;
     uint32_t width_pad = 0, vocab_pad = 0;
-    bf16 *embed = nullptr;
+    bf16 *embed = nullptr, *pos = nullptr;
     DenseLinear head;
     float *final_norm = nullptr;
     std::unordered_map<std::string, LayeredDst> names;
@@ -52,6 +76,12 @@ struct LayeredModel {
     uint32_t proj_pitch = 0, cat_pitch = 0, q_pitch = 0, cq_pitch = 0;
     uint32_t *want_idx = nullptr, *pf_tok = nullptr;
     LatentRowsScratch rows_scratch{};
+    // sequential arrangement
+    void *xc = nullptr, *y = nullptr, *moe_x = nullptr, *act = nullptr, *conv = nullptr, *delta = nullptr;  // convolved norm, results, experts' rows
+    float *aux = nullptr, *history = nullptr, *o32 = nullptr;  // fp32 projections, residual stream after every layer, outputs before their norm
+    uint32_t aux_pitch = 0, y_pitch = 0, act_pitch = 0, conv_pitch = 0, o32_width = 0;
+    size_t pairs_cap = 0;                          // rows of the experts' buffers
+    MoePlan plan{};                                // buffers; experts and top are the layer's
     // expanded keys and values of a prompt portion, grown on demand
     bf16 *ex_lat = nullptr, *ex_krot = nullptr, *ex_kv = nullptr;
     size_t ex_lat_n = 0, ex_krot_n = 0, ex_kv_n = 0;
