@@ -11,6 +11,14 @@ import math
 import numpy as np
 
 
+# What a 16-bit run keeps of an activation; `forward(rounding=...)` sets it to see how far rounding alone goes.
+def _exact(x):
+    return x
+
+
+_keep = _exact
+
+
 # ---- elementwise pieces ----------------------------------------------------------------------------
 def sigmoid(z):
     return 1.0 / (1.0 + np.exp(-z))
@@ -115,9 +123,9 @@ def latent_attention(h, w, mx, eps):
 def attention(h, w, mx, eps):
     """Grouped softmax attention without rotation; a window counts the token itself."""
     T, H, G, D, V = h.shape[0], mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
-    q = (h @ w["q"].T).reshape(T, H, D)
-    k = (h @ w["k"].T).reshape(T, G, D)
-    v = (h @ w["v"].T).reshape(T, G, V)
+    q = _keep(h @ w["q"].T).reshape(T, H, D)
+    k = _keep(h @ w["k"].T).reshape(T, G, D)
+    v = _keep(h @ w["v"].T).reshape(T, G, V)
     size = (mx.get("mask") or {}).get("size")
     out = np.zeros((T, H, V), h.dtype)
     for n in range(H):
@@ -127,7 +135,7 @@ def attention(h, w, mx, eps):
             s = k[lo:i + 1, g] @ q[i, n] * mx["scale"]
             p = np.exp(s - s.max())
             out[i, n] = (p / p.sum()) @ v[lo:i + 1, g]
-    return out.reshape(T, H * V) @ w["o"].T
+    return _keep(_keep(out.reshape(T, H * V)) @ w["o"].T)
 
 
 def causal_conv(x, w):
@@ -152,7 +160,7 @@ def unit(x):
 def gated_delta(h, w, mx, eps):
     """Delta rule with one decay and one step size per head and token, token by token."""
     T, H, G, D, V = h.shape[0], mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
-    short = lambda n: silu(causal_conv(h @ w[n].T, w[n + ".conv"]))  # noqa: E731
+    short = lambda n: _keep(silu(causal_conv(_keep(h @ w[n].T), w[n + ".conv"])))  # noqa: E731
     q = unit(short("q").reshape(T, G, D)) * D ** -0.5
     k = unit(short("k").reshape(T, G, D))
     v = short("v").reshape(T, H, V)
@@ -166,8 +174,8 @@ def gated_delta(h, w, mx, eps):
             u = beta[t, n] * (v[t, n] - k[t, g] @ S)
             S = S + np.outer(k[t, g], u)
             o[t, n] = q[t, g] @ S
-    o = rms_norm(o, w["norm"], eps) * silu(h @ w["g"].T).reshape(T, H, V)
-    return o.reshape(T, H * V) @ w["o"].T
+    o = rms_norm(o, w["norm"], eps) * _keep(silu(h @ w["g"].T)).reshape(T, H, V)
+    return _keep(_keep(o.reshape(T, H * V)) @ w["o"].T)
 
 
 def parallel(h, w, mx, eps):
@@ -204,16 +212,19 @@ def moe_ff(h, w, mlp):
     z = h @ w["router"].T
     for t in range(h.shape[0]):
         for e, weight in zip(*route(z[t], w["correction"], r["top"], r.get("groups"))):
-            y[t] += weight * (w[f"e{e}.down"] @ np.maximum(w[f"e{e}.up"] @ h[t], 0.0) ** 2)
+            y[t] += weight * _keep(w[f"e{e}.down"] @ _keep(np.maximum(w[f"e{e}.up"] @ h[t], 0.0) ** 2))
     return y
 
 
 # ---- a layer with sublayers one after the other -------------------------------------------------------
-def sublayer(x, w, p, n, eps, f):
-    """x plus the gated result of f on the convolved norm; n is "1" (mixer) or "2" (feed-forward)."""
-    h = rms_norm(x, 1.0 + w[p + "norm" + n], eps)
-    gate = sigmoid(h @ w[p + "rg" + n].T + w[p + "rg" + n + ".b"])
-    return x + gate * f(h + causal_conv(h, w[p + "canon" + n]))
+def sublayer(x, w, p, n, eps, offset, f):
+    """x plus the result of f on the norm; n is "1" (mixer) or "2" (feed-forward).  With a convolution f reads the
+    norm plus its convolution, with a gate the result is multiplied by it."""
+    h = _keep(rms_norm(x, offset + w[p + "norm" + n], eps))
+    y = f(_keep(h + causal_conv(h, w[p + "canon" + n])) if p + "canon" + n in w else h)
+    if p + "rg" + n in w:
+        y = y * _keep(sigmoid(h @ w[p + "rg" + n].T + w[p + "rg" + n + ".b"]))
+    return x + y
 
 
 def depth_average(w, history):
@@ -221,19 +232,23 @@ def depth_average(w, history):
 
 
 def forward_sequential(cfg, weights, tokens, layers_out=None):
-    eps, n = cfg["norm"]["eps"], len(tokens)
-    x = weights["embed"][np.asarray(tokens)] + weights["pos"][:n]
+    eps, offset = cfg["norm"]["eps"], cfg.get("norm_offset", 1.0)
+    x = weights["embed"][np.asarray(tokens)]
+    if "pos" in weights:
+        x = x + weights["pos"][:len(tokens)]
     history = [x]
     for i, ly in enumerate(cfg["layers"]):
-        p = f"l{i}."
-        x = sublayer(x, weights, p, "1", eps, lambda h: MIXERS[ly["type"]](h, _sub(weights, p + "mix."), ly["mixer"], eps))
-        if ly.get("mlp"):
-            x = sublayer(x, weights, p, "2", eps, lambda h: moe_ff(h, _sub(weights, p + "mlp."), ly["mlp"]))
+        p, mlp = f"l{i}.", ly.get("mlp")
+        x = sublayer(x, weights, p, "1", eps, offset, lambda h: MIXERS[ly["type"]](h, _sub(weights, p + "mix."), ly["mixer"], eps))
+        if mlp:
+            ff = (lambda h: dense_ff(h, _sub(weights, p + "mlp."))) if mlp["kind"] == "dense" else (lambda h: moe_ff(h, _sub(weights, p + "mlp."), mlp))
+            x = sublayer(x, weights, p, "2", eps, offset, ff)
         history.append(x)
-        x = depth_average(weights[p + "dwa"], history)
+        if p + "dwa" in weights:
+            x = depth_average(weights[p + "dwa"], history)
         if layers_out is not None:
             layers_out.append(x)
-    return rms_norm(x, 1.0 + weights["final.norm"], eps) @ weights["head"].T
+    return _keep(rms_norm(x, offset + weights["final.norm"], eps)) @ weights["head"].T
 
 
 # ---- the model -------------------------------------------------------------------------------------
@@ -242,10 +257,13 @@ def _sub(weights, prefix):
     return {k[n:]: v for k, v in weights.items() if k.startswith(prefix)}
 
 
-def forward(cfg, weights, tokens, dt=np.float64, layers_out=None):
-    """Logits [tokens, vocab] of one sequence; ``layers_out`` (a list) receives the residual after every layer."""
+def forward(cfg, weights, tokens, dt=np.float64, layers_out=None, rounding=_exact):
+    """Logits [tokens, vocab] of one sequence; ``layers_out`` (a list) receives the residual after every layer.
+    ``rounding`` is applied to the activations between linears (sequential layers only)."""
+    global _keep
+    _keep = rounding
     weights = {k: np.asarray(v, dt) for k, v in weights.items()}
-    if cfg["architecture"] == "Tozarax":
+    if cfg["architecture"] != "Mefipel":
         return forward_sequential(cfg, weights, tokens, layers_out)
     eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
     x = weights["embed"][np.asarray(tokens)]

@@ -25,14 +25,16 @@ __device__ __forceinline__ float log_decay(const DeltaArgs &a, const float *ba, 
 }
 
 // ---- decode ----------------------------------------------------------------------------------------------
-// silu(conv) of channel c at position pos; cur: its projection at pos.
+// silu(conv) of channel c at position pos as the activation type holds it; cur: its projection at pos.
 template <typename TA>
 __device__ __forceinline__ float short_conv(const DeltaArgs &a, const TA *ring, uint32_t c, int32_t pos, float cur) {
     const uint32_t C = a.channels;
     const int32_t T = (int32_t)a.taps - 1;
     float s = a.conv_w[(size_t)T * C + c] * cur;
     for (int32_t j = max(0, T - pos); j < T; j++) s = fmaf(a.conv_w[(size_t)j * C + c], ld_act(ring + (size_t)((uint32_t)(pos - T + j) % a.taps) * C + c), s);
-    return s * sigmoid_f(s);
+    TA y;
+    st_act(&y, s * sigmoid_f(s));
+    return ld_act(&y);
 }
 
 // Grid: (CTAs of a cluster, head, row).  A CTA takes every cs-th slice of 32 value columns; thread (d group, column)

@@ -29,6 +29,103 @@ def model(layers, width=48, vocab=131, eps=1e-5, residual_mult=0.7, logit_scale=
             "vocab": vocab, "width": width}
 
 
+# ---- sequential arrangement --------------------------------------------------------------------------
+def attention(heads, kv_heads, dim, vdim, window=None, scale=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": 1.3 * dim ** -0.5 if scale is None else scale}
+    if window:
+        m["mask"] = {"size": window}
+    return m
+
+
+def delta(heads, kv_heads, dim, vdim, conv=3):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}
+
+
+def moe(experts, top, ff, groups=None):
+    r = {"experts": experts, "top": top}
+    if groups:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "expert": {"ff": ff}, "router": r}
+
+
+def pair(left, right, mlp=None):
+    return {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": mlp}
+
+
+def tozarax(layers, width=48, vocab=131, eps=1e-5, taps=3, max_positions=600):
+    return {"architecture": "Tozarax", "canon": {"taps": taps}, "layers": layers, "max_positions": max_positions, "norm": {"eps": eps},
+            "vocab": vocab, "width": width}
+
+
+def sequential(layers, width=48, vocab=131, eps=1e-5, norm_offset=0.0, **options):
+    """A design of its own from the same parts: any mixer or feed-forward, any of the options left out."""
+    return {"architecture": "SequentialTest", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "norm_offset": norm_offset,
+            "options": options}
+
+
+def _register():
+    from prism_engine_b200 import models as m
+
+    m.REGISTRY["SequentialTest"] = lambda raw: m.LayeredConfig(
+        vocab=raw["vocab"], width=raw["width"], norm_eps=raw["norm"]["eps"], layers=m.LayeredConfig.read_layers(raw),
+        arrangement=m.ARRANGE_SEQUENTIAL, norm_offset=raw["norm_offset"], **raw["options"])
+
+
+_register()
+
+
+def sequential_weights(cfg, seed=0, apart=0.12):
+    """As weights(); `apart`: how far the experts of a layer (and their corrections) differ.  A little makes a routing
+    decided by rounding harmless, 1 makes them independent."""
+    import prism_engine_b200 as p
+
+    rng = np.random.default_rng([8, seed])
+    c = p.LayeredConfig.from_dict(cfg)
+    out, base = {}, {}
+    for name, shape in c.tensor_shapes().items():
+        leaf = name.split(".")[-1]
+        if leaf.startswith("norm") and name.count(".") == 1 or name == "final.norm":
+            v = rng.normal(0.0, 0.3, shape) + 1.0 - c.norm_offset
+        elif leaf in ("norm", "out"):
+            v = rng.normal(1.0, 0.3, shape)
+        elif leaf == "dwa":
+            v = rng.normal(0.0, 0.2, shape)
+            v[-1] += 1.0
+        elif leaf == "correction":
+            v = rng.normal(0.0, 0.3 * apart, shape)
+        elif leaf in ("A_log", "dt_bias"):
+            v = rng.normal(-1.0, 0.8, shape)
+        elif leaf.startswith("canon") or leaf == "conv":
+            v = rng.normal(0.0, 0.5, shape)
+        elif leaf == "pos":
+            v = rng.normal(0.0, 0.4, shape)
+        elif leaf == "b" and len(shape) == 1:
+            v = rng.normal(0.0, 0.5, shape)
+        elif len(shape) == 1:
+            v = rng.normal(0.0, 0.3, shape)
+        else:
+            v = rng.normal(0.0, 1.0 if name == "embed" else 1.2 / np.sqrt(shape[1]), shape)
+        head, _, part = name.partition(".mlp.e")
+        if part:
+            key = head, leaf
+            base.setdefault(key, rng.normal(0.0, 1.2 / np.sqrt(shape[1]), shape))
+            v = (1.0 - apart) * base[key] + apart * v
+        out[name] = round_bf16(v)[1]
+    return out
+
+
+def keep_bf16(x):
+    return round_bf16(x)[1].astype(np.float64).reshape(np.shape(x))
+
+
+def expected(cfg, w, toks, dtype):
+    """The restatement's logits of a sequential model; for bf16 with the activations between linears rounded as a
+    16-bit run rounds them, so that norms of small values and choices of experts see the same rounding."""
+    from oracle import layered as orc
+
+    return orc.forward(cfg, w, toks, **({"rounding": keep_bf16} if dtype == "bfloat16" else {}))
+
+
 def round_bf16(x):
     """Nearest bf16 (ties to even) of a float array: (bit patterns, float32 values)."""
     u = np.ascontiguousarray(x, np.float32).view(np.uint32)
