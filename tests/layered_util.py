@@ -74,7 +74,7 @@ def _register():
 _register()
 
 
-def sequential_weights(cfg, seed=0, apart=0.12):
+def sequential_weights(cfg, seed=0, apart=1.0):
     """As weights(); `apart`: how far the experts of a layer (and their corrections) differ.  A little makes a routing
     decided by rounding harmless, 1 makes them independent."""
     import prism_engine_b200 as p

@@ -96,14 +96,6 @@ def test_experts_alone(backend, dtype, i):
     check(backend, cfg, 120, WHOLE_AND_STEPS + [(4, 8, 7)], dtype, seed=20 + i, without=["left.out", "right.out"])
 
 
-@pytest.mark.parametrize("rows", [9, 17, 40, 100, 129, 200, 300, 520])
-@pytest.mark.parametrize("ff", [72, 512])
-def test_row_tiles_of_the_expert_gemm(backend, rows, ff):
-    """One and several row tiles per expert, few and many rows each; some experts without any."""
-    cfg = U.tozarax([U.pair(TINY_A, TINY_D, U.moe(9, 3, ff, (3, 2)))], width=256)
-    check(backend, cfg, rows, [(10 ** 9,)], "bfloat16", seed=rows, without=["left.out", "right.out"])
-
-
 def _clear_choices(cfg, w, n, margin, seed):
     """Token ids whose choices (groups and experts) stand out by `margin` at every place; layer 0, mixers silent."""
     mlp, eps, taps = cfg["layers"][0]["mlp"], cfg["norm"]["eps"], cfg["canon"]["taps"]
@@ -147,6 +139,18 @@ def test_choice_of_experts(backend, dtype, i, correction):
         plain = dict(w, **{"l0.mlp.correction": 0 * w["l0.mlp.correction"]})
         assert U.error(orc.forward(cfg, plain, toks), want) > 5 * U.TOL[dtype]
     compare(backend, cfg, w, toks, WHOLE_AND_STEPS + [(8, 3, 1)], dtype)
+
+
+@pytest.mark.parametrize("rows", [9, 17, 40, 100, 129, 200, 300, 520])
+@pytest.mark.parametrize("ff", [72, 512])
+def test_row_tiles_of_the_expert_gemm(backend, rows, ff):
+    """One and several row tiles per expert, few and many rows each, independent experts, some of them without a row."""
+    cfg = U.tozarax([U.pair(TINY_A, TINY_D, U.moe(12, 3, ff, (4, 2)))], width=256)
+    w = U.sequential_weights(cfg, rows, apart=1.0)
+    for name in ("left", "right"):
+        w[f"l0.mix.{name}.out"] *= 0.0
+    w["l0.mlp.correction"] = U.round_bf16(np.linspace(-0.4, 0.4, 12))[1]
+    compare(backend, cfg, w, _clear_choices(cfg, w, rows, 0.02, rows), [(10 ** 9,)], "bfloat16")
 
 
 # ---- around the sublayers ----------------------------------------------------------------------------------

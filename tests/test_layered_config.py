@@ -111,3 +111,72 @@ def test_rotation_is_relative_and_window_counts_itself():
     assert s[0] == pytest.approx(s[1], rel=1e-9)
     assert np.array_equal(orc.rotate(a, [7], rot)[0, 6:], a[0, 6:])
     assert [orc.window_visible(10, j, 3) for j in (7, 8, 9, 10, 11)] == [False, True, True, True, False]
+
+
+# ---- sequential layers -----------------------------------------------------------------------------------------
+
+def _tozarax():
+    return U.tozarax([U.pair(U.attention(4, 2, 8, 12, window=9), U.delta(3, 1, 16, 20, conv=4), U.moe(8, 3, 24, (4, 2))),
+                      U.pair(U.attention(2, 1, 8, 8), U.delta(1, 1, 8, 8))], taps=2, max_positions=70)
+
+
+def test_sequential_configuration(tmp_path):
+    cfg = p.read_config(_write(tmp_path, _tozarax()))
+    a, b = cfg.layers
+    assert (cfg.arrangement, cfg.norm_offset, cfg.canon_taps, cfg.max_positions) == (models.ARRANGE_SEQUENTIAL, 1.0, 2, 70)
+    assert cfg.gated_residual and cfg.depth_average
+    assert a.mixer == models.MIXER_PAIR and a.left.window == 9 and b.left.window == 0 and a.right.conv == 4
+    assert (a.ff, a.experts, a.top, a.expert_groups, a.groups_keep, b.ff) == (24, 8, 3, 4, 2, 0)
+    sh = cfg.tensor_shapes()
+    assert sh["l0.mix.left.v"] == (24, 48) and sh["l0.mix.right.v"] == (60, 48) and sh["l0.mix.right.k.conv"] == (16, 4)
+    assert sh["l0.dwa"] == (2,) and sh["l1.dwa"] == (3,) and sh["pos"] == (70, 48) and sh["l0.rg2"] == (48, 48) and sh["l0.canon1"] == (48, 2)
+    assert "l1.norm2" not in sh and "l1.rg2" not in sh and "l1.canon2" not in sh and "l0.mlp.e8.up" not in sh
+    mc, arr, keep = cfg.to_c("bfloat16", 64, 2)
+    assert (mc.arrangement, mc.canon_taps, mc.depth_average, mc.max_positions) == (1, 2, 1, 70)
+    from prism_engine_b200._lib import LayerConfig
+    right = LayerConfig.from_address(arr[0].right)
+    assert (right.heads, right.kv_heads, right.dim, right.vdim, right.conv) == (3, 1, 16, 20, 4) and keep
+    bad = _tozarax()
+    bad["layers"][0]["mlp"]["router"]["groups"]["keep"] = 1
+    with pytest.raises(ValueError, match="choose 3"):
+        p.LayeredConfig.from_dict(bad)
+    bad = _tozarax()
+    bad["layers"][0]["mixer"]["left"]["kv_heads"] = 3
+    with pytest.raises(ValueError, match="share"):
+        p.LayeredConfig.from_dict(bad)
+
+
+def test_oracle_gated_delta_against_its_triangular_form():
+    """The recurrence against the solved system of all updates (one chunk, state from zero)."""
+    rng = np.random.default_rng(3)
+    T, D, V = 11, 4, 5
+    mx = {"heads": 1, "kv_heads": 1, "dim": D, "vdim": V, "conv": 2}
+    w = {n: rng.normal(size=s) for n, s in {"q": (D, 6), "k": (D, 6), "v": (V, 6), "b": (1, 6), "a": (1, 6), "g": (V, 6), "o": (6, V), "q.conv": (D, 2),
+                                            "k.conv": (D, 2), "v.conv": (V, 2), "A_log": 1, "dt_bias": 1, "norm": V}.items()}
+    h = rng.normal(size=(T, 6))
+    act = lambda n: orc.silu(orc.causal_conv(h @ w[n].T, w[n + ".conv"]))  # noqa: E731
+    q, k, v = orc.unit(act("q")) * D ** -0.5, orc.unit(act("k")), act("v")
+    L = np.cumsum(-np.exp(w["A_log"]) * np.log1p(np.exp(h @ w["a"].T + w["dt_bias"])))
+    beta = orc.sigmoid(h @ w["b"].T)[:, 0]
+    dec = np.exp(L[:, None] - L[None, :])
+    u = np.linalg.solve(np.eye(T) + np.tril(beta[:, None] * dec * (k @ k.T), -1), beta[:, None] * v)
+    o = np.tril(dec * (q @ k.T)) @ u
+    want = orc.rms_norm(o, w["norm"], 1e-3) * orc.silu(h @ w["g"].T) @ w["o"].T
+    np.testing.assert_allclose(orc.gated_delta(h, w, mx, 1e-3), want, rtol=1e-8, atol=1e-10)
+
+
+def test_oracle_routing():
+    z = np.log(np.array([0.9, 0.12, 0.6, 0.55, 0.5, 0.45, 0.8, 0.2]) / (1 - np.array([0.9, 0.12, 0.6, 0.55, 0.5, 0.45, 0.8, 0.2])))
+    best, weight = orc.route(z, np.zeros(8), 3, None)
+    assert best == [0, 6, 2] and weight == pytest.approx([0.9, 0.8, 0.6])
+    # groups (0 1)(2 3)(4 5)(6 7) score 1.02, 1.15, 0.95, 1.0: the first two are kept
+    assert orc.route(z, np.zeros(8), 3, {"count": 4, "keep": 2})[0] == [0, 2, 3]
+    best, weight = orc.route(z, np.array([-2.0, 0, 0, 0, 0, 0, -2.0, -2.0]), 2, {"count": 4, "keep": 3})
+    assert best == [2, 3] and weight == pytest.approx([0.6, 0.55])  # the weight is the score without the correction
+    assert orc.route(z, np.full(8, -5.0), 2, {"count": 2, "keep": 1})[0] == [0, 2]
+
+
+def test_oracle_convolution_and_average():
+    x, w = np.arange(1.0, 6.0)[:, None], np.array([[100.0, 10.0, 1.0]])
+    assert orc.causal_conv(x, w)[:, 0].tolist() == [1.0, 12.0, 123.0, 234.0, 345.0]
+    assert orc.depth_average([0.5, 2.0], [np.ones(2), np.full(2, 3.0)]).tolist() == [6.5, 6.5]
