@@ -68,7 +68,15 @@ LAYERED_WORKLOADS = {
                                         latent=dict(heads=28, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=2048))),
     "mefipel-72b-8-layers": ("QWEN25_72B", 8, dict(lightning=dict(heads=64, dim=128, vdim=128),
                                                    latent=dict(heads=64, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, window=2048))),
+    # a token's experts together are as wide as the dense feed-forward of the model of equal size
+    "tozarax-0.5b": ("QWEN25_0P5B", 0, dict(left=dict(heads=14, kv_heads=2, dim=64, vdim=64, window=1024),
+                                            right=dict(heads=14, kv_heads=14, dim=64, vdim=64, conv=4), experts=16, top=4)),
+    "tozarax-7b": ("QWEN25_7B", 0, dict(left=dict(heads=28, kv_heads=4, dim=128, vdim=128, window=2048),
+                                        right=dict(heads=28, kv_heads=14, dim=128, vdim=128, conv=4), experts=16, top=4)),
+    "tozarax-72b-4-layers": ("QWEN25_72B", 4, dict(left=dict(heads=64, kv_heads=8, dim=128, vdim=128, window=2048),
+                                                   right=dict(heads=64, kv_heads=32, dim=128, vdim=128, conv=4), experts=16, top=4)),
 }
+LAYERED_WORKLOADS["mefipel-72b-4-layers"] = ("QWEN25_72B", 4, LAYERED_WORKLOADS["mefipel-72b-8-layers"][2])
 METRIC = "decode_tokens_per_s"
 UNIT = "tok/s"
 FALLBACK_HBM_GBS = 6650.0
@@ -653,14 +661,23 @@ def run_gemm(args):
     return 0
 
 
-def layered_raw(name):
-    """config.json of a layered workload: lightning and latent attention layers in turn."""
+def layered_raw(name, n_layers=0):
+    """config.json of a layered workload: lightning and latent attention layers in turn (Mefipel), or layers of
+    windowed attention beside a gated delta rule with experts (Tozarax)."""
     import prism_engine_b200 as p
 
-    arch_name, n_layers, mix = LAYERED_WORKLOADS[name]
+    arch_name, own_layers, mix = LAYERED_WORKLOADS[name]
     arch = dict(getattr(p, arch_name))
-    if n_layers:
-        arch["num_layers"] = n_layers
+    arch["num_layers"] = n_layers or own_layers or arch["num_layers"]
+    raw = {"norm": {"eps": 1e-6}, "vocab": arch["vocab_size"], "width": arch["hidden_size"]}
+    if name.startswith("tozarax"):
+        left = {k: v for k, v in mix["left"].items() if k != "window"}
+        left.update(mask={"size": mix["left"]["window"]}, scale=left["dim"] ** -0.5)
+        mlp = {"kind": "moe", "expert": {"ff": arch["intermediate_size"] // mix["top"]},
+               "router": {"experts": mix["experts"], "top": mix["top"], "groups": {"count": 4, "keep": 2}}}
+        raw.update(architecture="Tozarax", canon={"taps": 4}, max_positions=8192,
+                   layers=[{"type": "parallel", "mixer": {"left": left, "right": dict(mix["right"])}, "mlp": mlp}] * arch["num_layers"])
+        return raw, arch
     li, la = mix["lightning"], mix["latent"]
     decay = [1.0 - 2.0 ** (-4.0 - 6.0 * h / li["heads"]) for h in range(li["heads"])]
     lightning = {"type": "lightning", "mixer": dict(li, decay=decay)}
@@ -669,37 +686,52 @@ def layered_raw(name):
         rot={"base": 5e5, "dims": la["rot_dim"], "scaling": {"factor": 8.0, "fast": 16.0, "original": 4096, "slow": 2.0}})}
     layers = [dict(latent if i % 2 else lightning, mlp={"kind": "dense", "ff": arch["intermediate_size"]})
               for i in range(arch["num_layers"])]
-    raw = {"architecture": "Mefipel", "layers": layers, "logit_scale": 1.0, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
-           "vocab": arch["vocab_size"], "width": arch["hidden_size"]}
+    raw.update(architecture="Mefipel", layers=layers, logit_scale=1.0, residual_mult=0.5)
     return raw, arch
 
 
 def linear_flops_per_token(cfg):
-    """2 x weights of every linear a prompt token goes through (no head; keys and values expanded once per token)."""
-    return 2.0 * sum(float(np.prod(s)) for n, s in cfg.tensor_shapes().items() if len(s) == 2 and n not in ("embed", "head"))
+    """2 x weights of every linear a prompt token goes through (no head; keys and values expanded once per token;
+    of the experts, as many as a token is sent through)."""
+    flops = 0.0
+    for n, s in cfg.tensor_shapes().items():
+        if len(s) != 2 or n in ("embed", "head", "pos") or n.endswith("conv") or "canon" in n:
+            continue
+        share = 1.0
+        if ".mlp.e" in n:
+            spec = cfg.layers[int(n[1:n.index(".")])]
+            share = spec.top / spec.experts
+        flops += 2.0 * share * float(np.prod(s))
+    return flops
 
 
-def measure_layered(env, be, name, batches, steps, warmup, ctx_len, n_prompt):
+def measure_layered(env, be, name, batches, steps, warmup, ctx_len, n_prompt, n_layers=0):
+    """The layered model and the closest model of equal size: the palettized one beside a Mefipel, a Mefipel beside
+    a Tozarax."""
     import prism_engine_b200 as p
     from prism_engine_b200 import synth
 
-    raw, arch = layered_raw(name)
-    cfg = p.LayeredConfig.from_dict(raw)
-    peak, _ = measured_peaks()
+    raw, arch = layered_raw(name, n_layers)
     sustained, _, _ = measured_tensor_peak()
     H, I, L = arch["hidden_size"], arch["intermediate_size"], arch["num_layers"]
     qkv = (arch["num_heads"] + 2 * arch["num_kv_heads"]) * arch["head_dim"]
     pal_flops = 2.0 * L * (qkv * H + H * arch["num_heads"] * arch["head_dim"] + 3 * H * I)
     max_seq = max(ctx_len + 40 + 2 * (warmup + steps), n_prompt) + 16
+    kinds = [("layered", raw)]
+    if name.startswith("tozarax"):
+        kinds.append(("mefipel", layered_raw(name.replace("tozarax", "mefipel"), n_layers)[0]))
+    else:
+        kinds.append(("palettized", None))
     out = {}
-    for kind in ("layered", "palettized"):
-        if kind == "layered":
+    for kind, doc in kinds:
+        if doc:
+            cfg = p.LayeredConfig.from_dict(doc)
             eng = p.PrismEngine(be, cfg, max_seq=max_seq, max_batch=max(batches))
         else:
             eng = p.PrismEngine(be, p.model_config(**arch, max_seq=max_seq, max_batch=max(batches), profile="baseline"))
         eng.synth_weights(seed=1)
         # the layered generate() leaves the last prompt token to the first decode step
-        prompt = synth.make_prompt(n_prompt + (kind == "layered"), arch["vocab_size"], seed=3)
+        prompt = synth.make_prompt(n_prompt + (doc is not None), arch["vocab_size"], seed=3)
         for _ in range(2):
             eng.generate(prompt, 0)
         reps = 5
@@ -708,20 +740,20 @@ def measure_layered(env, be, name, batches, steps, warmup, ctx_len, n_prompt):
             eng.generate(prompt, 0)
             ms += eng.last_ms()
         ms /= reps
-        flops = (linear_flops_per_token(cfg) if kind == "layered" else pal_flops) * n_prompt
+        flops = (linear_flops_per_token(cfg) if doc else pal_flops) * n_prompt
         res = {"prefill": {"tokens": n_prompt, "ms": ms, "tok_s": n_prompt / ms * 1e3, "linear_tflops": flops / ms / 1e9,
                            "frac_of_sustained": flops / ms / 1e9 / sustained}}
         for b in batches:
             m, _ = measure_decode(env, be, eng, arch, b, ctx_len, steps, warmup)
             res[f"decode_batch{b}"] = m
-        res["weights"] = "bf16" if kind == "layered" else "4-bit palettized"
+        res["weights"] = "bf16" if doc else "4-bit palettized"
         out[kind] = res
         eng.close()
     return out
 
 
 def run_layered(args):
-    """Prefill and decode of a model described layer by layer beside the palettized model of equal size."""
+    """Prefill and decode of a model described layer by layer beside the closest model of equal size."""
     import prism_engine_b200 as p
 
     env = Env(args)
@@ -732,7 +764,7 @@ def run_layered(args):
         key, val = kv.split("=")
         be.set_option(key, int(val))
     ctx_len = 512 if args.ctx < 0 else args.ctx
-    res = measure_layered(env, be, args.workload, sorted({1, 8, args.batch}), args.steps, args.warmup, ctx_len, 2048)
+    res = measure_layered(env, be, args.workload, sorted({1, 8, args.batch}), args.steps, args.warmup, ctx_len, 2048, args.layers)
     main = res["layered"][f"decode_batch{args.batch}"]
     emit({"metric": METRIC, "value": main["value"], "unit": UNIT, "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
           "ms_per_step": main["ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,

@@ -44,7 +44,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const DeltaArgs 
     extern __shared__ float dsm[];
     __shared__ float red[2][8][DL_VS + 1], sh[32], part;
     pdl_launch_dependents();
-    pdl_wait();
+    if (!a.beside) pdl_wait();
     const uint32_t rank = blockIdx.x, h = blockIdx.y, r = blockIdx.z, tid = threadIdx.x, vl = tid & 31, dg = tid >> 5;
     const uint32_t group = a.heads / a.kv_heads, kh = h / group, C = a.channels, qk = a.kv_heads * a.dim;
     const int32_t pos = rows.pos_of(r), slot = rows.slot_of(r);
@@ -77,7 +77,20 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const DeltaArgs 
             now[qk + c] = kc;
         }
     }
-    const float rq = 1.0f / (sqrtf(block_sum_f(sq, sh) + DL_UNIT_EPS) * sqrtf((float)a.dim)), rk = 1.0f / sqrtf(block_sum_f(sk, sh) + DL_UNIT_EPS);
+    sq = warp_sum_f(sq);
+    sk = warp_sum_f(sk);
+    if (vl == 0) {
+        sh[dg] = sq;
+        sh[8 + dg] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.0f;
+#pragma unroll
+    for (int e = 0; e < 8; e++) {
+        sq += sh[e];
+        sk += sh[8 + e];
+    }
+    const float rq = 1.0f / (sqrtf(sq + DL_UNIT_EPS) * sqrtf((float)a.dim)), rk = 1.0f / sqrtf(sk + DL_UNIT_EPS);
     float ss = 0.0f;
     for (uint32_t sl = rank, i = 0; sl < n_slices; sl += cs, i++) {
         const uint32_t v = sl * DL_VS + vl, c = 2 * qk + h * a.vdim + v;
@@ -147,6 +160,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const DeltaArgs 
                    os[i * DL_VS + vl] * inv * a.norm[v] * ld_act(reinterpret_cast<const TA *>(a.gate) + (size_t)r * a.gate_pitch + h * a.vdim + v));
     }
     if (cs > 1) cg::this_cluster().sync();  // the peers read this CTA's sum
+    if (a.beside) pdl_wait();  // the kernel after this one relies on the one before it too
 }
 
 template <typename TA>
@@ -244,7 +258,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_gate_kernel(const DeltaArgs 
 //   S   = e^(L_last) S0 + sum_j e^(L_last-L_j) k_j u_j^T,
 // with T = (I + A)^-1 diag(beta).  The unit factors are scalars per row, so q and k themselves stay the bf16 values
 // they are; everything else enters the tensor cores as two bf16 parts.
-constexpr int DC_C = 64, DC_PV = DL_VS + 8, DC_PT = DC_C + 8;
+constexpr int DC_C = 64, DC_PV = DL_VS + 8, DC_PT = DC_C + 8, DC_PA = DC_C + 4, DC_PY = 36;
 constexpr uint32_t DC_SCALARS = 256;                              // floats: e[64] f[64] w[64], last: e^(L_last)
 constexpr size_t DC_ITEM = 4 * DC_C * DC_C * 2 + DC_SCALARS * 4;  // T hi, T lo, P hi, P lo, scalars
 
@@ -274,8 +288,8 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs 
     pdl_wait();
     const uint32_t PD = dpad + 8, ch = blockIdx.x, h = blockIdx.y, kh = h / (a.heads / a.kv_heads), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t g8 = lane >> 2, t4 = lane & 3, r0 = ch * DC_C, nt = min((uint32_t)DC_C, a.rows - r0);
-    constexpr uint32_t PA = DC_C + 4;
-    float *A = reinterpret_cast<float *>(dps), *X = A + DC_C * PA;  // X shares its place with Q and K
+    constexpr uint32_t PA = DC_PA, PY = DC_PY;
+    float *A = reinterpret_cast<float *>(dps), *X = A + DC_C * PA, *Y = X + DC_C * PA;  // X and Y share their place with Q and K
     bf16 *Q = reinterpret_cast<bf16 *>(X), *K = Q + DC_C * PD;
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(Q), sK = (uint32_t)__cvta_generic_to_shared(K);
     load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec);
@@ -367,39 +381,70 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs 
         if (tid == 0) sc[3 * DC_C] = expf(L[DC_C - 1]);
     }
     __syncthreads();
-    {   // column c of (I + A)^-1 by four threads: the one with s = i / 16 keeps entry i
-        const uint32_t c = tid >> 2, s = tid & 3;
+    // X = (I + A)^-1: the diagonal blocks of 16 by substitution, then X21 = -X22 A21 X11 for blocks of 16 and of 32
+    for (uint32_t i = tid; i < DC_C * DC_C; i += DL_THREADS) X[(i / DC_C) * PA + i % DC_C] = 0.0f;
+    __syncthreads();
+    if (tid < DC_C) {
+        const uint32_t d = tid & ~15u, c = tid & 15;
         float x[16];
 #pragma unroll
-        for (int j = 0; j < 16; j++) x[j] = 0.0f;
-        const float b = bt[c];
+        for (int i = 0; i < 16; i++) {
+            float p0 = i == (int)c ? 1.0f : 0.0f, p1 = 0.0f;
 #pragma unroll
-        for (int i = 0; i < DC_C; i++) {
-            const float4 *ar = reinterpret_cast<const float4 *>(A + i * PA + s * 16);
-            float p0 = 0.0f, p1 = 0.0f;
-#pragma unroll
-            for (int q = 0; q < 4; q++) {
-                const float4 v = ar[q];
-                p0 = fmaf(v.x, x[4 * q], p0);
-                p1 = fmaf(v.y, x[4 * q + 1], p1);
-                p0 = fmaf(v.z, x[4 * q + 2], p0);
-                p1 = fmaf(v.w, x[4 * q + 3], p1);
+            for (int j = 0; j < i; j++) {
+                const float t = A[(d + i) * PA + d + j] * x[j];
+                if (j & 1) p1 -= t;
+                else p0 -= t;
             }
-            p0 += p1;
-            p0 += __shfl_xor_sync(0xFFFFFFFFu, p0, 1);
-            p0 += __shfl_xor_sync(0xFFFFFFFFu, p0, 2);
-            const float xi = (i == (int)c ? 1.0f : 0.0f) - p0;
-            if ((int)s == i / 16) {
-                x[i % 16] = xi;
-                X[i * (DC_C + 1) + c] = xi * b;
-            }
+            x[i] = p0 + p1;
+            X[(d + i) * PA + d + c] = x[i];
         }
+    }
+    __syncthreads();
+    {
+        const uint32_t d = (tid >> 7) * 32, r = (tid & 127) >> 3, c = (tid & 7) * 2;
+        float2 y = make_float2(0.0f, 0.0f);
+#pragma unroll
+        for (uint32_t k = 0; k < 16; k++) {
+            const float t = A[(d + 16 + r) * PA + d + k];
+            const float2 x = *reinterpret_cast<const float2 *>(X + (d + k) * PA + d + c);
+            y = make_float2(fmaf(t, x.x, y.x), fmaf(t, x.y, y.y));
+        }
+        *reinterpret_cast<float2 *>(Y + (d / 2 + r) * PY + c) = y;
+        __syncthreads();
+        float2 z = make_float2(0.0f, 0.0f);
+#pragma unroll
+        for (uint32_t k = 0; k < 16; k++) {
+            const float t = -X[(d + 16 + r) * PA + d + 16 + k];
+            const float2 x = *reinterpret_cast<const float2 *>(Y + (d / 2 + k) * PY + c);
+            z = make_float2(fmaf(t, x.x, z.x), fmaf(t, x.y, z.y));
+        }
+        *reinterpret_cast<float2 *>(X + (d + 16 + r) * PA + d + c) = z;
+    }
+    __syncthreads();
+    {
+        const uint32_t r = tid >> 3, c = (tid & 7) * 4;
+        auto mul = [&](const float *m, const float *q, uint32_t pitch) {
+            float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+            for (uint32_t k = 0; k < 32; k++) {
+                const float t = m[k];
+                const float4 x = *reinterpret_cast<const float4 *>(q + k * pitch + c);
+                y = make_float4(fmaf(t, x.x, y.x), fmaf(t, x.y, y.y), fmaf(t, x.z, y.z), fmaf(t, x.w, y.w));
+            }
+            return y;
+        };
+        const float4 y = mul(A + (32 + r) * PA, X, PA);
+        *reinterpret_cast<float4 *>(Y + r * PY + c) = y;
+        __syncthreads();
+        const float4 z = mul(X + (32 + r) * PA + 32, Y, PY);
+        *reinterpret_cast<float4 *>(X + (32 + r) * PA + c) = make_float4(-z.x, -z.y, -z.z, -z.w);
     }
     __syncthreads();
     for (uint32_t i = tid; i < DC_C * DC_C / 2; i += DL_THREADS) {
         const uint32_t r = i / (DC_C / 2), c = (i % (DC_C / 2)) * 2;
         uint32_t hi, lo;
-        split_bf16(X[r * (DC_C + 1) + c], X[r * (DC_C + 1) + c + 1], hi, lo);
+        split_bf16(X[r * PA + c] * bt[c], X[r * PA + c + 1] * bt[c + 1], hi, lo);
         *reinterpret_cast<uint32_t *>(Th + r * DC_C + c) = hi;
         *reinterpret_cast<uint32_t *>(Tl + r * DC_C + c) = lo;
     }
@@ -602,7 +647,7 @@ int launch_delta_seq(prism_cuda_ctx *ctx, const DeltaArgs &a, const RowMap &rows
         const uint32_t vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.pitch % 8 == 0 &&
                              !((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v)) & 15);
         const size_t qk = (size_t)2 * DC_C * (dpad + 8) * 2;
-        const size_t prep = (size_t)DC_C * (DC_C + 4) * 4 + std::max(qk, (size_t)DC_C * (DC_C + 1) * 4);
+        const size_t prep = (size_t)DC_C * DC_PA * 4 + std::max(qk, (size_t)(DC_C * DC_PA + 32 * DC_PY) * 4);
         launch_pdl(ctx, "delta_prep_kernel", delta_prep_kernel, dim3((a.rows + DC_C - 1) / DC_C, a.heads), DL_THREADS, prep, a, dpad, vec);
         PRISM_TRY(after_launch(ctx, "delta_prep_kernel"));
         const size_t tile = qk + (size_t)(DC_C * DC_PV + 4 * DC_C * DC_PT) * 2 + DC_SCALARS * 4, rest = (size_t)(2 * dpad + 6 * DC_C) * DC_PV * 2;

@@ -504,13 +504,15 @@ int launch_dense_norm(prism_cuda_ctx *ctx, const DenseIn &in, void *y, uint32_t 
     return after_launch(ctx, "dense_norm_kernel");
 }
 
+constexpr uint32_t DE_COLS = 1024;  // columns of a CTA
 __global__ void dense_embed_kernel(const bf16 *__restrict__ table, uint32_t width, uint32_t vocab, const uint32_t *__restrict__ tokens,
                                    float *__restrict__ x, const bf16 *__restrict__ pos_table, uint32_t max_pos, const RowMap map, float *__restrict__ x2) {
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t r = blockIdx.x, tok = min(tokens[r], vocab - 1);  // the host rejects larger ids before the launch
+    const uint32_t c1 = min(width, (blockIdx.y + 1) * DE_COLS);
     const bf16 *pt = pos_table ? pos_table + (size_t)min((uint32_t)map.pos_of(r), max_pos - 1) * width : nullptr;  // and later positions
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
+    for (uint32_t i = blockIdx.y * DE_COLS + threadIdx.x; i < c1; i += blockDim.x) {
         const float v = __bfloat162float(table[(size_t)tok * width + i]) + (pt ? __bfloat162float(pt[i]) : 0.0f);
         x[(size_t)r * width + i] = v;
         if (x2) x2[(size_t)r * width + i] = v;
@@ -518,7 +520,7 @@ __global__ void dense_embed_kernel(const bf16 *__restrict__ table, uint32_t widt
 }
 int launch_dense_embed(prism_cuda_ctx *ctx, const bf16 *table, uint32_t width, uint32_t vocab, const uint32_t *tokens, uint32_t rows, float *x,
                        const bf16 *pos_table, uint32_t max_pos, const RowMap &map, float *x2) {
-    launch_pdl(ctx, "dense_embed_kernel", dense_embed_kernel, rows, 256, 0, table, width, vocab, tokens, x, pos_table, max_pos, map, x2);
+    launch_pdl(ctx, "dense_embed_kernel", dense_embed_kernel, dim3(rows, (width + DE_COLS - 1) / DE_COLS), 256, 0, table, width, vocab, tokens, x, pos_table, max_pos, map, x2);
     return after_launch(ctx, "dense_embed_kernel");
 }
 

@@ -340,9 +340,10 @@ struct GroupedArgs {
 uint32_t grouped_splits(const GroupedArgs &a, uint32_t max_seq);
 int launch_grouped_append(prism_cuda_ctx *ctx, const GroupedArgs &a, const void *k, const void *v, uint32_t pitch, const RowMap &rows, uint32_t n_rows,
                           bool act32);
-// k, v: null when the rows' keys are in the cache already, else they are appended (rows of different sequences)
+// k, v: null when the rows' keys are in the cache already, else they are appended (rows of different sequences).
+// late: the next kernel of the stream is released only once what this one waits for is complete (DeltaArgs::beside).
 int launch_grouped_rows(prism_cuda_ctx *ctx, const GroupedArgs &a, const void *q, const void *k, const void *v, uint32_t pitch, void *out,
-                        uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32);
+                        uint32_t out_pitch, const RowMap &rows, uint32_t n_rows, bool act32, bool late = false);
 int launch_grouped_prefill(prism_cuda_ctx *ctx, const GroupedArgs &a, const bf16 *q, uint32_t pitch, bf16 *out, uint32_t out_pitch, const RowMap &rows,
                            uint32_t n_rows);
 
@@ -421,6 +422,9 @@ struct DeltaArgs {
     float *o32;                       // sequence: outputs before their norm, [rows][heads * vdim]
     void *chunk_scratch;              // sequence: delta_scratch_bytes
     uint32_t channels;                // 2 * kv_heads * dim + heads * vdim
+    // step: runs beside the kernel launched before it, which has released its dependents only after its own
+    // dependency wait: what this one reads is there when it starts, and it waits for that kernel at its end
+    uint32_t beside;
 };
 size_t delta_scratch_bytes(const DeltaArgs &a, uint32_t rows);
 int launch_delta_step(prism_cuda_ctx *ctx, const DeltaArgs &a, const RowMap &rows, bool act32);

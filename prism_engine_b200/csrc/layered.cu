@@ -521,20 +521,20 @@ static int mix_lightning(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &m
     return seq ? launch_lightning_seq(e->ctx, a, rows, m->act32) : launch_lightning_step(e->ctx, a, rows, m->act32);
 }
 
-static int mix_attention(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, const RowMap &rows, uint32_t n, bool seq) {
+static int mix_attention(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, const RowMap &rows, uint32_t n, bool seq, bool late) {
     prism_cuda_ctx *ctx = e->ctx;
     LayeredModel *m = e->lm;
     const DenseSeg *seg = ly.in.seg + mx.seg0;
     const void *q = at(m, m->proj, seg[0].row0), *k = at(m, m->proj, seg[1].row0), *v = at(m, m->proj, seg[2].row0);
     void *out = at(m, m->cat, mx.col);
-    if (!seq) return launch_grouped_rows(ctx, mx.ga, q, k, v, m->proj_pitch, out, m->cat_pitch, rows, n, m->act32);
+    if (!seq) return launch_grouped_rows(ctx, mx.ga, q, k, v, m->proj_pitch, out, m->cat_pitch, rows, n, m->act32, late);
     PRISM_TRY(launch_grouped_append(ctx, mx.ga, k, v, m->proj_pitch, rows, n, m->act32));
     if (!m->act32 && n > DENSE_GEMV_ROWS && tiled_attn_ok(mx.ga.dp, mx.ga.vp))
         return launch_grouped_prefill(ctx, mx.ga, (const bf16 *)q, m->proj_pitch, (bf16 *)out, m->cat_pitch, rows, n);
     return launch_grouped_rows(ctx, mx.ga, q, nullptr, nullptr, m->proj_pitch, out, m->cat_pitch, rows, n, m->act32);
 }
 
-static int mix_delta(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, const RowMap &rows, uint32_t n, bool seq) {
+static int mix_delta(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, const RowMap &rows, uint32_t n, bool seq, bool beside) {
     prism_cuda_ctx *ctx = e->ctx;
     LayeredModel *m = e->lm;
     const DenseSeg *seg = ly.in.seg + mx.seg0;
@@ -544,6 +544,7 @@ static int mix_delta(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, c
     a.ba = m->aux; a.ba_pitch = m->aux_pitch;
     a.gate = at(m, m->proj, seg[4].row0); a.gate_pitch = m->proj_pitch;
     a.o = at(m, m->cat, mx.col); a.o_pitch = m->cat_pitch;
+    a.beside = beside;
     if (!seq) return launch_delta_step(ctx, a, rows, m->act32);
     const uint32_t hk = a.kv_heads * a.dim;
     ConvArgs c{};
@@ -600,12 +601,14 @@ static int mix_latent(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, 
     return PRISM_OK;
 }
 
+// In a decode step the two kernels of an attention and a gated delta rule run side by side: neither needs the other.
 static int run_mixer(prism_cuda_engine *e, LayeredLayer &ly, LayeredMixer &mx, const RowMap &rows, uint32_t n, bool seq) {
+    const bool side = !seq && ly.mix.size() == 2 && ly.mix[0].c.mixer == PRISM_MIXER_ATTENTION && ly.mix[1].c.mixer == PRISM_MIXER_GATED_DELTA;
     switch (mx.c.mixer) {
     case PRISM_MIXER_LIGHTNING: return mix_lightning(e, ly, mx, rows, n, seq);
     case PRISM_MIXER_LATENT_ATTENTION: return mix_latent(e, ly, mx, rows, n, seq);
-    case PRISM_MIXER_ATTENTION: return mix_attention(e, ly, mx, rows, n, seq);
-    default: return mix_delta(e, ly, mx, rows, n, seq);
+    case PRISM_MIXER_ATTENTION: return mix_attention(e, ly, mx, rows, n, seq, side);
+    default: return mix_delta(e, ly, mx, rows, n, seq, side);
     }
 }
 // Lightning: all heads normed together, then gated, as the input of the output linear takes it.

@@ -51,13 +51,13 @@ __device__ __forceinline__ float as_act(float v, const float *) { return v; }
 __device__ __forceinline__ float as_act(float v, const bf16 *) { return __bfloat162float(__float2bfloat16_rn(v)); }
 
 // ---- convolution along a portion ---------------------------------------------------------------------------
-// Thread: V channels of a strip of tokens.  Only the first strip reaches back before the portion, and the same
-// threads leave the portion's last inputs in the ring after they have read what was there.
-constexpr int CV_THREADS = 128, CV_STRIP = 16;
-template <typename TA, int V>
+// Thread: V channels of a strip of tokens; with TAPS the last inputs stay in registers.  Only the first strip reaches
+// back before the portion, and the same threads leave the portion's last inputs in the ring after they have read what
+// was there.
+constexpr int CV_THREADS = 128, CV_STRIP = 16, CV_U = 8;
+template <typename TA, int V, int TAPS>
 __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, const RowMap rows, uint32_t n, uint32_t strip) {
     pdl_launch_dependents();
-    pdl_wait();
     uint32_t b = blockIdx.x, pc = 0;
     while (pc + 1 < a.pieces && b >= (a.piece[pc].channels + CV_THREADS * V - 1) / (CV_THREADS * V)) {
         b -= (a.piece[pc].channels + CV_THREADS * V - 1) / (CV_THREADS * V);
@@ -70,21 +70,54 @@ __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, 
     TA *y = reinterpret_cast<TA *>(p.y) + c, *ring = reinterpret_cast<TA *>(a.ring) + (size_t)rows.slot0 * a.taps * a.channels + p.c0 + c;
     const float *w = a.w + p.c0 + c;
     const int32_t T = (int32_t)a.taps - 1, t0 = (int32_t)(blockIdx.y * strip), t1 = min((int32_t)n, t0 + (int32_t)strip);
-    for (int32_t t = t0; t < t1; t++) {
-        Vals<V> s, cur = ldv<V>(x + (size_t)t * a.x_pitch);
+    auto earlier = [&](int32_t u) {  // the input of the portion's token u, u < t0
+        const int32_t pos = rows.pos0 + u;
+        if (pos < 0) return Vals<V>{};
+        return u >= 0 ? ldv<V>(x + (size_t)u * a.x_pitch) : ldv<V>(ring + (size_t)((uint32_t)pos % a.taps) * a.channels);
+    };
+    auto finish = [&](int32_t t, const Vals<V> &s, const Vals<V> &cur) {
+        Vals<V> o;
 #pragma unroll
-        for (int i = 0; i < V; i++) s.v[i] = 0.0f;
-        for (int32_t j = 0; j <= T; j++) {
-            const int32_t u = t - T + j, pos = rows.pos0 + u;
-            if (pos < 0) continue;
-            const Vals<V> h = u >= 0 ? ldv<V>(x + (size_t)u * a.x_pitch) : ldv<V>(ring + (size_t)((uint32_t)pos % a.taps) * a.channels);
-            const Vals<V> wj = ldv<V>(w + (size_t)j * a.channels);
+        for (int i = 0; i < V; i++) o.v[i] = a.silu ? s.v[i] * sigmoid_f(s.v[i]) : cur.v[i] + s.v[i];
+        stv<V>(y + (size_t)t * a.y_pitch, o);
+    };
+    if constexpr (TAPS > 0) {
+        Vals<V> wr[TAPS], h[TAPS];  // h[j]: the input TAPS - 1 - j tokens ago
 #pragma unroll
-            for (int i = 0; i < V; i++) s.v[i] = fmaf(wj.v[i], h.v[i], s.v[i]);
+        for (int j = 0; j < TAPS; j++) wr[j] = ldv<V>(w + (size_t)j * a.channels);
+        pdl_wait();
+#pragma unroll
+        for (int j = 1; j < TAPS; j++) h[j] = earlier(t0 - TAPS + j);
+        for (int32_t t = t0; t < t1; t += CV_U) {
+            Vals<V> in[CV_U];
+#pragma unroll
+            for (int k = 0; k < CV_U; k++)
+                if (t + k < t1) in[k] = ldv<V>(x + (size_t)(t + k) * a.x_pitch);
+#pragma unroll
+            for (int k = 0; k < CV_U; k++) {
+                if (t + k >= t1) break;
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; j++) h[j] = h[j + 1];
+                h[TAPS - 1] = in[k];
+                Vals<V> s{};
+#pragma unroll
+                for (int j = 0; j < TAPS; j++)
+#pragma unroll
+                    for (int i = 0; i < V; i++) s.v[i] = fmaf(wr[j].v[i], h[j].v[i], s.v[i]);
+                finish(t + k, s, in[k]);
+            }
         }
+    } else {
+        pdl_wait();
+        for (int32_t t = t0; t < t1; t++) {
+            Vals<V> s{};
+            for (int32_t j = 0; j <= T; j++) {
+                const Vals<V> h = earlier(t - T + j), wj = ldv<V>(w + (size_t)j * a.channels);
 #pragma unroll
-        for (int i = 0; i < V; i++) s.v[i] = a.silu ? s.v[i] * sigmoid_f(s.v[i]) : cur.v[i] + s.v[i];
-        stv<V>(y + (size_t)t * a.y_pitch, s);
+                for (int i = 0; i < V; i++) s.v[i] = fmaf(wj.v[i], h.v[i], s.v[i]);
+            }
+            finish(t, s, ldv<V>(x + (size_t)t * a.x_pitch));
+        }
     }
     if (blockIdx.y == 0)
         for (int32_t t = max(0, (int32_t)n - T); t < (int32_t)n; t++)
@@ -103,8 +136,11 @@ static int run_conv(prism_cuda_ctx *ctx, const ConvArgs &a, const RowMap &rows, 
     for (uint32_t i = 0; i < a.pieces; i++) blocks += (a.piece[i].channels + CV_THREADS * (vec ? 4 : 1) - 1) / (CV_THREADS * (vec ? 4 : 1));
     const uint32_t strip = std::max((uint32_t)CV_STRIP, a.taps);
     const dim3 grid(blocks, (n + strip - 1) / strip);
-    if (vec) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4>, grid, CV_THREADS, 0, a, rows, n, strip);
-    else launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 1>, grid, CV_THREADS, 0, a, rows, n, strip);
+    if (!vec) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 1, 0>, grid, CV_THREADS, 0, a, rows, n, strip);
+    else if (a.taps == 2) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 2>, grid, CV_THREADS, 0, a, rows, n, strip);
+    else if (a.taps == 3) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 3>, grid, CV_THREADS, 0, a, rows, n, strip);
+    else if (a.taps == 4) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 4>, grid, CV_THREADS, 0, a, rows, n, strip);
+    else launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 0>, grid, CV_THREADS, 0, a, rows, n, strip);
     return after_launch(ctx, "conv_seq_kernel");
 }
 int launch_conv_seq(prism_cuda_ctx *ctx, const ConvArgs &a, const RowMap &rows, uint32_t n_rows, bool act32) {
@@ -125,6 +161,37 @@ __device__ __forceinline__ float cluster_sum_f(float v, float *sh, float *slot, 
     float s = 0.0f;
     for (uint32_t r = 0; r < cs; r++) s += *cluster.map_shared_rank(slot, r);
     return s;
+}
+
+// Two sums at once (the block's part: sh holds 32 floats, slot two).
+__device__ __forceinline__ float2 cluster_sum2_f(float a, float b, float *sh, float *slot, uint32_t cs) {
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    a = warp_sum_f(a);
+    b = warp_sum_f(b);
+    if (lane == 0) {
+        sh[warp] = a;
+        sh[16 + warp] = b;
+    }
+    __syncthreads();
+    a = b = 0.0f;
+#pragma unroll
+    for (uint32_t i = 0; i < RU_THREADS / 32; i++) {
+        a += sh[i];
+        b += sh[16 + i];
+    }
+    if (cs == 1) return make_float2(a, b);
+    cg::cluster_group cluster = cg::this_cluster();
+    if (threadIdx.x == 0) {
+        slot[0] = a;
+        slot[1] = b;
+    }
+    cluster.sync();
+    a = b = 0.0f;
+    for (uint32_t r = 0; r < cs; r++) {
+        a += *cluster.map_shared_rank(slot, r);
+        b += *cluster.map_shared_rank(slot + 1, r);
+    }
+    return make_float2(a, b);
 }
 
 template <typename TA, int V>
@@ -148,8 +215,9 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(const RowUpdate 
                 s2 = fmaf(q.v[i], q.v[i], s2);
             }
         }
-        inv1 = 0.5f / sqrtf(cluster_sum_f(s1, sh, slot, cs) / (float)D + u.eps);
-        inv2 = 0.5f / sqrtf(cluster_sum_f(s2, sh, slot + 1, cs) / (float)D + u.eps);
+        const float2 q = cluster_sum2_f(s1, s2, sh, slot, cs);
+        inv1 = 0.5f / sqrtf(q.x / (float)D + u.eps);
+        inv2 = 0.5f / sqrtf(q.y / (float)D + u.eps);
     }
     float ss = 0.0f;
     for (uint32_t c = c_lo + threadIdx.x * V; c < c_hi; c += RU_THREADS * V) {
@@ -227,6 +295,121 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(const RowUpdate 
     if (cs > 1) cg::this_cluster().sync();  // the peers read this CTA's sums
 }
 
+// The same for rows whose run of columns is at most one vector per thread (narrow, or few rows with a cluster each):
+// everything is requested before the first sum, weights before the dependency wait.
+template <typename TA, int V>
+__global__ void __launch_bounds__(RU_THREADS) row_update_few_kernel(const RowUpdate u, const RowMap rows, uint32_t cs, uint32_t per) {
+    __shared__ float sh[32], slot[3];
+    pdl_launch_dependents();
+    const uint32_t r = blockIdx.y, D = u.width, c_lo = blockIdx.x * per, c = c_lo + threadIdx.x * V;
+    const bool on = c < min(c_lo + per, D);
+    constexpr int RU_TAPS = 4;  // weights of the convolution requested early
+    Vals<V> w1{}, w2{}, nw{}, cw[RU_TAPS] = {};
+    if (on) {
+        if (u.add == ROW_ADD_PAIR) {
+            w1 = ldv<V>(u.w + c);
+            w2 = ldv<V>(u.w2 + c);
+        }
+        if (u.norm) nw = ldv<V>(u.norm + c);
+#pragma unroll
+        for (int j = 0; j < RU_TAPS; j++)
+            if (u.conv_w && j < (int)u.taps) cw[j] = ldv<V>(u.conv_w + (size_t)j * D + c);
+    }
+    pdl_wait();
+    const int32_t pos = u.conv_w ? rows.pos_of(r) : 0, T = (int32_t)u.taps - 1;
+    TA *ring = u.conv_w ? reinterpret_cast<TA *>(u.ring) + (size_t)rows.slot_of(r) * u.taps * D + c : nullptr;
+    Vals<V> v{}, d{}, d2{}, g, old{}, past[RU_TAPS - 1] = {};
+#pragma unroll
+    for (int i = 0; i < V; i++) g.v[i] = 1.0f;
+    float own = 1.0f;
+    if (on) {
+        v = ldv<V>(u.x + (size_t)r * D + c);
+        if (u.add == ROW_ADD_ONE || u.add == ROW_ADD_PAIR) d = ldv<V>(reinterpret_cast<const TA *>(u.y) + (size_t)r * u.y_pitch + c);
+        if (u.add == ROW_ADD_PAIR) d2 = ldv<V>(reinterpret_cast<const TA *>(u.y2) + (size_t)r * u.y2_pitch + c);
+        if (u.gate) g = ldv<V>(reinterpret_cast<const TA *>(u.gate) + (size_t)r * u.gate_pitch + c);
+#pragma unroll
+        for (int j = 0; j < RU_TAPS - 1; j++)
+            if (u.conv_w && j < T && pos - T + j >= 0) past[j] = ldv<V>(ring + (size_t)((uint32_t)(pos - T + j) % u.taps) * D);
+        if (u.history) {
+            own = u.avg[u.n_history];
+            const float *h = u.history + (size_t)r * D + c;
+#pragma unroll 8
+            for (uint32_t j = 0; j < u.n_history; j++) {
+                const Vals<V> o = ldv<V>(h + j * u.history_stride);
+                const float aj = u.avg[j];
+#pragma unroll
+                for (int i = 0; i < V; i++) old.v[i] = fmaf(aj, o.v[i], old.v[i]);
+            }
+        }
+        if (u.add == ROW_ADD_EXPERTS) {
+#pragma unroll 8
+            for (uint32_t k = 0; k < u.top; k++) {
+                const uint32_t pair = r * u.top + k, row = u.inv ? u.inv[pair] : pair;
+                const Vals<V> e = ldv<V>(reinterpret_cast<const TA *>(u.y) + (size_t)row * u.y_pitch + c);
+                const float w = u.wgt[pair];
+#pragma unroll
+                for (int i = 0; i < V; i++) d.v[i] = fmaf(w, e.v[i], d.v[i]);
+            }
+        }
+    }
+    if (u.add == ROW_ADD_PAIR) {
+        float s1 = 0.0f, s2 = 0.0f;
+#pragma unroll
+        for (int i = 0; i < V; i++) {
+            s1 = fmaf(d.v[i], d.v[i], s1);
+            s2 = fmaf(d2.v[i], d2.v[i], s2);
+        }
+        const float2 q = cluster_sum2_f(s1, s2, sh, slot, cs);
+        const float inv1 = 0.5f / sqrtf(q.x / (float)D + u.eps), inv2 = 0.5f / sqrtf(q.y / (float)D + u.eps);
+#pragma unroll
+        for (int i = 0; i < V; i++) d.v[i] = d.v[i] * inv1 * w1.v[i] + d2.v[i] * inv2 * w2.v[i];
+    }
+    float ss = 0.0f;
+    if (on) {
+#pragma unroll
+        for (int i = 0; i < V; i++) v.v[i] = fmaf(u.mul, d.v[i] * g.v[i], v.v[i]);
+        if (u.history) {
+            stv<V>(u.history + u.n_history * u.history_stride + (size_t)r * D + c, v);
+#pragma unroll
+            for (int i = 0; i < V; i++) v.v[i] = fmaf(own, v.v[i], old.v[i]);
+        }
+        if (u.x_out) stv<V>(u.x_out + (size_t)r * D + c, v);
+#pragma unroll
+        for (int i = 0; i < V; i++) ss = fmaf(v.v[i], v.v[i], ss);
+    }
+    if (u.norm) {
+        const float inv = 1.0f / sqrtf(cluster_sum_f(ss, sh, slot + 2, cs) / (float)D + u.eps);
+        if (on) {
+            TA *h = reinterpret_cast<TA *>(u.h) + (size_t)r * u.h_pitch + c;
+#pragma unroll
+            for (int i = 0; i < V; i++) v.v[i] = as_act(v.v[i] * inv * nw.v[i], h);
+            stv<V>(h, v);
+            if (u.conv_w) {
+                Vals<V> s = v;
+                for (int32_t j = max(0, T - pos); j <= T; j++) {
+                    Vals<V> o = v, wj;
+                    if (T < RU_TAPS) {
+#pragma unroll
+                        for (int e = 0; e < RU_TAPS; e++)
+                            if (e == j) {
+                                wj = cw[e];
+                                if (e < RU_TAPS - 1 && e < T) o = past[e];
+                            }
+                    } else {
+                        wj = ldv<V>(u.conv_w + (size_t)j * D + c);
+                        if (j < T) o = ldv<V>(ring + (size_t)((uint32_t)(pos - T + j) % u.taps) * D);
+                    }
+#pragma unroll
+                    for (int i = 0; i < V; i++) s.v[i] = fmaf(wj.v[i], o.v[i], s.v[i]);
+                }
+                stv<V>(ring + (size_t)((uint32_t)pos % u.taps) * D, v);
+                stv<V>(reinterpret_cast<TA *>(u.hc) + (size_t)r * u.h_pitch + c, s);
+            }
+        }
+    }
+    if (cs > 1) cg::this_cluster().sync();  // the peers read this CTA's sums
+}
+
 template <typename TA>
 static int run_row_update(prism_cuda_ctx *ctx, const RowUpdate &u, const RowMap &rows, uint32_t n) {
     uintptr_t at = 0;
@@ -245,6 +428,11 @@ static int run_row_update(prism_cuda_ctx *ctx, const RowUpdate &u, const RowMap 
         PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(row_update_kernel<TA, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     }
     if (n > 65535) return fail(ctx, PRISM_E_ARG, "row update: too many rows");
+    if (per <= RU_THREADS * (vec ? 4u : 1u)) {
+        if (vec) launch_cluster_pdl(ctx, row_update_few_kernel<TA, 4>, dim3(cs, n), RU_THREADS, 0, cs, u, rows, cs, per);
+        else launch_cluster_pdl(ctx, row_update_few_kernel<TA, 1>, dim3(cs, n), RU_THREADS, 0, cs, u, rows, cs, per);
+        return after_launch(ctx, "row_update_few_kernel");
+    }
     if (vec) launch_cluster_pdl(ctx, row_update_kernel<TA, 4>, dim3(cs, n), RU_THREADS, (size_t)per * 4, cs, u, rows, cs, per);
     else launch_cluster_pdl(ctx, row_update_kernel<TA, 1>, dim3(cs, n), RU_THREADS, (size_t)per * 4, cs, u, rows, cs, per);
     return after_launch(ctx, "row_update_kernel");
