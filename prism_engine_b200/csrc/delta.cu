@@ -234,21 +234,42 @@ __global__ void __launch_bounds__(DL_THREADS) delta_seq_kernel(const DeltaArgs a
         if (on) S[(size_t)d * a.vdim + v] = ss[d * DL_VS + vl];
 }
 
-// One warp per row and head: the output's norm over its head, weight and gate.
+// One warp per row and head: the output's norm over its head, weight and gate.  vec: four values of a lane at a time,
+// kept in registers.
+constexpr int DG_U = 2;  // vectors of a lane: heads of up to 256 values
 template <typename TA>
-__global__ void __launch_bounds__(DL_THREADS) delta_gate_kernel(const DeltaArgs a) {
+__global__ void __launch_bounds__(DL_THREADS) delta_gate_kernel(const DeltaArgs a, uint32_t vec) {
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t lane = threadIdx.x & 31, i = blockIdx.x * (DL_THREADS / 32) + (threadIdx.x >> 5);
     if (i >= a.rows * a.heads) return;
     const uint32_t r = i / a.heads, h = i % a.heads;
     const float *o = a.o32 + (size_t)i * a.vdim;
+    const TA *gate = reinterpret_cast<const TA *>(a.gate) + (size_t)r * a.gate_pitch + h * a.vdim;
+    TA *to = reinterpret_cast<TA *>(a.o) + (size_t)r * a.o_pitch + h * a.vdim;
     float ss = 0.0f;
+    if (vec) {
+        float4 x[DG_U], g[DG_U];
+#pragma unroll
+        for (int u = 0; u < DG_U; u++) {
+            const uint32_t v = (lane + 32 * u) * 4;
+            x[u] = v < a.vdim ? ld4(o + v) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (v < a.vdim) g[u] = ld4(gate + v);
+            ss += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
+        }
+        const float inv = 1.0f / sqrtf(warp_sum_f(ss) / (float)a.vdim + a.eps);
+#pragma unroll
+        for (int u = 0; u < DG_U; u++) {
+            const uint32_t v = (lane + 32 * u) * 4;
+            if (v >= a.vdim) break;
+            const float4 w = ld4(a.norm + v);
+            st4(to + v, make_float4(x[u].x * inv * w.x * g[u].x, x[u].y * inv * w.y * g[u].y, x[u].z * inv * w.z * g[u].z, x[u].w * inv * w.w * g[u].w));
+        }
+        return;
+    }
     for (uint32_t v = lane; v < a.vdim; v += 32) ss = fmaf(o[v], o[v], ss);
     const float inv = 1.0f / sqrtf(warp_sum_f(ss) / (float)a.vdim + a.eps);
-    for (uint32_t v = lane; v < a.vdim; v += 32)
-        st_act(reinterpret_cast<TA *>(a.o) + (size_t)r * a.o_pitch + h * a.vdim + v,
-               o[v] * inv * a.norm[v] * ld_act(reinterpret_cast<const TA *>(a.gate) + (size_t)r * a.gate_pitch + h * a.vdim + v));
+    for (uint32_t v = lane; v < a.vdim; v += 32) st_act(to + v, o[v] * inv * a.norm[v] * ld_act(gate + v));
 }
 
 // ---- prompts in chunks -------------------------------------------------------------------------------------
@@ -262,17 +283,16 @@ constexpr int DC_C = 64, DC_PV = DL_VS + 8, DC_PT = DC_C + 8, DC_PA = DC_C + 4, 
 constexpr uint32_t DC_SCALARS = 256;                              // floats: e[64] f[64] w[64], last: e^(L_last)
 constexpr size_t DC_ITEM = 4 * DC_C * DC_C * 2 + DC_SCALARS * 4;  // T hi, T lo, P hi, P lo, scalars
 
-// Rows of a chunk into shared memory, zeros past row nt and column `valid`.
+// Rows of a chunk into shared memory, zeros past row nt and column `valid`; 2^sh threads take a row.
 __device__ __forceinline__ void load_rows(bf16 *dst, uint32_t pitch, uint32_t cols, const bf16 *src, uint32_t src_pitch, uint32_t nt, uint32_t valid,
-                                          bool vec) {
+                                          bool vec, uint32_t sh) {
     const uint32_t s = (uint32_t)__cvta_generic_to_shared(dst);
     if (vec) {
-        const uint32_t n8 = cols / 8;
-        for (uint32_t i = threadIdx.x; i < DC_C * n8; i += DL_THREADS) {
-            const uint32_t r = i / n8, c = (i % n8) * 8;
-            if (r < nt && c < valid) cp_async16(s + (r * pitch + c) * 2, src + (size_t)r * src_pitch + c);
-            else *reinterpret_cast<uint4 *>(dst + r * pitch + c) = make_uint4(0, 0, 0, 0);
-        }
+        for (uint32_t r = threadIdx.x >> sh; r < DC_C; r += DL_THREADS >> sh)
+            for (uint32_t c = (threadIdx.x & ((1u << sh) - 1)) * 8; c < cols; c += 8u << sh) {
+                if (r < nt && c < valid) cp_async16(s + (r * pitch + c) * 2, src + (size_t)r * src_pitch + c);
+                else *reinterpret_cast<uint4 *>(dst + r * pitch + c) = make_uint4(0, 0, 0, 0);
+            }
     } else {
         for (uint32_t i = threadIdx.x; i < DC_C * cols; i += DL_THREADS) {
             const uint32_t r = i / cols, c = i % cols;
@@ -281,7 +301,7 @@ __device__ __forceinline__ void load_rows(bf16 *dst, uint32_t pitch, uint32_t co
     }
 }
 
-__global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs a, uint32_t dpad, uint32_t vec) {
+__global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs a, uint32_t dpad, uint32_t vec, uint32_t sh) {
     extern __shared__ __align__(16) uint8_t dps[];
     __shared__ float L[DC_C], rq[DC_C], rk[DC_C], bt[DC_C];
     pdl_launch_dependents();
@@ -292,8 +312,8 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs 
     float *A = reinterpret_cast<float *>(dps), *X = A + DC_C * PA, *Y = X + DC_C * PA;  // X and Y share their place with Q and K
     bf16 *Q = reinterpret_cast<bf16 *>(X), *K = Q + DC_C * PD;
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(Q), sK = (uint32_t)__cvta_generic_to_shared(K);
-    load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec);
-    load_rows(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec);
+    load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+    load_rows(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
     cp_async_commit();
     if (warp == 0) {  // running sums of the logarithms
         float carry = 0.0f;
@@ -452,7 +472,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs 
 
 // Grid: (slice of 32 value columns, head).  The slice of the state lives in mma accumulators from the first chunk to
 // the last; nbuf 2: the next chunk loads under this one.
-__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs a, int32_t slot, uint32_t dpad, uint32_t vec, uint32_t nbuf) {
+__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs a, int32_t slot, uint32_t dpad, uint32_t vec, uint32_t nbuf, uint32_t sh) {
     extern __shared__ __align__(16) uint8_t dcs[];
     pdl_launch_dependents();
     pdl_wait();
@@ -478,9 +498,9 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
     auto load_chunk = [&](uint32_t r0, uint32_t buf) {
         const uint32_t nt = min((uint32_t)DC_C, a.rows - r0);
         bf16 *Q = tiles + buf * TILE, *K = Q + DC_C * PD, *V = K + DC_C * PD, *TP = V + DC_C * DC_PV, *sc = TP + 4 * DC_C * DC_PT;
-        load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec);
-        load_rows(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec);
-        load_rows(V, DC_PV, DL_VS, reinterpret_cast<const bf16 *>(a.v) + (size_t)r0 * a.pitch + h * a.vdim + v0, a.pitch, nt, a.vdim - v0, vec);
+        load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+        load_rows(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+        load_rows(V, DC_PV, DL_VS, reinterpret_cast<const bf16 *>(a.v) + (size_t)r0 * a.pitch + h * a.vdim + v0, a.pitch, nt, a.vdim - v0, vec, 2);
         const uint8_t *item = reinterpret_cast<const uint8_t *>(a.chunk_scratch) + ((size_t)(r0 / DC_C) * a.heads + h) * DC_ITEM;
         for (uint32_t i = tid; i < 4 * DC_C * 8; i += DL_THREADS)
             cp_async16(sm(TP) + ((i >> 3) * DC_PT + (i & 7) * 8) * 2, item + (size_t)i * 16);
@@ -517,20 +537,29 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
         __syncthreads();  // this chunk and the state are there; every warp is done with the previous chunk
         if (nbuf == 2 && r0 + DC_C < a.rows) load_chunk(r0 + DC_C, buf ^ 1);
         const uint32_t i0 = (warp & 3) * 16, c0 = (warp >> 2) * 16;  // rows and value columns of this warp
-        float ks[2][4] = {}, qs[2][4] = {};
+        float ks[2][4] = {}, qs[2][4] = {}, kl[2][4] = {}, ql[2][4] = {};  // products with the state's high and low parts
         for (uint32_t d = 0; d < dpad; d += 16) {
             uint32_t ak[4], aq[4], b[4];
             ldsm_x4(ak, sK + ((i0 + (lane & 15)) * PD + d + (lane >> 4) * 8) * 2);
             ldsm_x4(aq, sQ + ((i0 + (lane & 15)) * PD + d + (lane >> 4) * 8) * 2);
-#pragma unroll
-            for (int half = 0; half < 2; half++) {
-                ldsm_x4_t(b, (half ? sSl : sSh) + ((d + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2);
-                mma_bf16(ks[0], ak, b[0], b[1]);
-                mma_bf16(ks[1], ak, b[2], b[3]);
-                mma_bf16(qs[0], aq, b[0], b[1]);
-                mma_bf16(qs[1], aq, b[2], b[3]);
-            }
+            ldsm_x4_t(b, sSh + ((d + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2);
+            mma_bf16(ks[0], ak, b[0], b[1]);
+            mma_bf16(ks[1], ak, b[2], b[3]);
+            mma_bf16(qs[0], aq, b[0], b[1]);
+            mma_bf16(qs[1], aq, b[2], b[3]);
+            ldsm_x4_t(b, sSl + ((d + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2);
+            mma_bf16(kl[0], ak, b[0], b[1]);
+            mma_bf16(kl[1], ak, b[2], b[3]);
+            mma_bf16(ql[0], aq, b[0], b[1]);
+            mma_bf16(ql[1], aq, b[2], b[3]);
         }
+#pragma unroll
+        for (int n = 0; n < 2; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                ks[n][i] += kl[n][i];
+                qs[n][i] += ql[n][i];
+            }
 #pragma unroll
         for (int n = 0; n < 2; n++)
 #pragma unroll
@@ -546,6 +575,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
         __syncthreads();
         // a lower triangular matrix (high and low parts at m) times columns c0 .. +16 of a right-hand side
         auto tri = [&](float (&o)[2][4], uint32_t m, uint32_t bh, uint32_t bl) {
+            float p[2][4] = {}, q[2][4] = {};
             for (uint32_t j = 0; j <= i0; j += 16) {
                 uint32_t xh[4], xl[4], b[4];
                 const uint32_t at = ((i0 + (lane & 15)) * DC_PT + j + (lane >> 4) * 8) * 2, bt = ((j + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2;
@@ -554,12 +584,16 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
                 ldsm_x4_t(b, bh + bt);
                 mma_bf16(o[0], xh, b[0], b[1]);
                 mma_bf16(o[1], xh, b[2], b[3]);
-                mma_bf16(o[0], xl, b[0], b[1]);
-                mma_bf16(o[1], xl, b[2], b[3]);
+                mma_bf16(p[0], xl, b[0], b[1]);
+                mma_bf16(p[1], xl, b[2], b[3]);
                 ldsm_x4_t(b, bl + bt);
-                mma_bf16(o[0], xh, b[0], b[1]);
-                mma_bf16(o[1], xh, b[2], b[3]);
+                mma_bf16(q[0], xh, b[0], b[1]);
+                mma_bf16(q[1], xh, b[2], b[3]);
             }
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) o[n][i] += p[n][i] + q[n][i];
         };
         float u[2][4] = {};
         tri(u, sT, sWh, sWl);
@@ -646,13 +680,14 @@ int launch_delta_seq(prism_cuda_ctx *ctx, const DeltaArgs &a, const RowMap &rows
     if (!act32 && dpad <= 256 && a.rows > DENSE_GEMV_ROWS) {
         const uint32_t vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.pitch % 8 == 0 &&
                              !((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.k) | reinterpret_cast<uintptr_t>(a.v)) & 15);
+        const uint32_t sh = row_shift(dpad / 8);
         const size_t qk = (size_t)2 * DC_C * (dpad + 8) * 2;
         const size_t prep = (size_t)DC_C * DC_PA * 4 + std::max(qk, (size_t)(DC_C * DC_PA + 32 * DC_PY) * 4);
-        launch_pdl(ctx, "delta_prep_kernel", delta_prep_kernel, dim3((a.rows + DC_C - 1) / DC_C, a.heads), DL_THREADS, prep, a, dpad, vec);
+        launch_pdl(ctx, "delta_prep_kernel", delta_prep_kernel, dim3((a.rows + DC_C - 1) / DC_C, a.heads), DL_THREADS, prep, a, dpad, vec, sh);
         PRISM_TRY(after_launch(ctx, "delta_prep_kernel"));
         const size_t tile = qk + (size_t)(DC_C * DC_PV + 4 * DC_C * DC_PT) * 2 + DC_SCALARS * 4, rest = (size_t)(2 * dpad + 6 * DC_C) * DC_PV * 2;
         const uint32_t nbuf = 2 * tile + rest <= DL_SMEM_MAX ? 2 : 1;
-        launch_pdl(ctx, "delta_chunk_kernel", delta_chunk_kernel, grid, DL_THREADS, nbuf * tile + rest, a, rows.slot0, dpad, vec, nbuf);
+        launch_pdl(ctx, "delta_chunk_kernel", delta_chunk_kernel, grid, DL_THREADS, nbuf * tile + rest, a, rows.slot0, dpad, vec, nbuf, sh);
         PRISM_TRY(after_launch(ctx, "delta_chunk_kernel"));
     } else {
         const size_t smem = (size_t)a.dim * (2 + DL_VS) * 4;
@@ -662,8 +697,10 @@ int launch_delta_seq(prism_cuda_ctx *ctx, const DeltaArgs &a, const RowMap &rows
         PRISM_TRY(after_launch(ctx, "delta_seq_kernel"));
     }
     const uint32_t blocks = (uint32_t)(((uint64_t)a.rows * a.heads + DL_THREADS / 32 - 1) / (DL_THREADS / 32));
-    if (act32) launch_pdl(ctx, "delta_gate_kernel", delta_gate_kernel<float>, blocks, DL_THREADS, 0, a);
-    else launch_pdl(ctx, "delta_gate_kernel", delta_gate_kernel<bf16>, blocks, DL_THREADS, 0, a);
+    const uint32_t vec = a.vdim <= 128 * DG_U && !((a.vdim | a.gate_pitch | a.o_pitch) & 3) &&
+                         !((reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.o) | reinterpret_cast<uintptr_t>(a.norm)) & 15);
+    if (act32) launch_pdl(ctx, "delta_gate_kernel", delta_gate_kernel<float>, blocks, DL_THREADS, 0, a, vec);
+    else launch_pdl(ctx, "delta_gate_kernel", delta_gate_kernel<bf16>, blocks, DL_THREADS, 0, a, vec);
     return after_launch(ctx, "delta_gate_kernel");
 }
 

@@ -112,16 +112,6 @@ struct GemvArgs {
 };
 constexpr int GV_THREADS = 256, GV_WARPS = 8, GV_U = 4, GV_KS_MAX = 4;
 
-// Four consecutive values of a row.
-__device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
-__device__ __forceinline__ float4 ld4(const bf16 *p) {
-    const uint2 u = *reinterpret_cast<const uint2 *>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-__device__ __forceinline__ void st4(bf16 *p, float4 v) { *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
-
 // RMS norm (times weight, times gate) of the first n_norm entries of the one or two rows into shared memory as bf16.
 // A row's threads keep their values and weights in registers (the weights requested before the dependency wait).
 constexpr int GN_U = 8;

@@ -209,6 +209,15 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t &hi, uint3
     hi = pack_bf16(ah, bh);
     lo = pack_bf16(a - ah, b - bh);
 }
+// Four consecutive values of a row.
+__device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 ld4(const bf16 *p) {
+    const uint2 u = *reinterpret_cast<const uint2 *>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void st4(bf16 *p, float4 v) { *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src) : "memory");
 }
@@ -216,6 +225,12 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 #endif
+// Rows of `n8` 16-byte pieces copied by the threads of a block: 2^row_shift(n8) neighbours take a row.
+inline uint32_t row_shift(uint32_t n8) {
+    uint32_t s = 0;
+    while (s < 5 && (1u << s) < n8) s++;
+    return s;
+}
 
 // First position that position pos sees under a window (0: none).
 #ifdef __CUDACC__
@@ -325,6 +340,7 @@ struct TiledAttn {
     uint32_t kx_head, vx_head;        // elements between the key (value) heads of a position, multiples of 8
     uint32_t lo, ring;                // ring 0: position p is row p - lo; else row p % ring
     uint32_t pos0, n_rows;            // first query position, queries
+    uint32_t shift;                   // set by the launcher: row_shift of a key's pieces
 };
 bool tiled_attn_ok(uint32_t dim, uint32_t vdim);
 int launch_tiled_attn(prism_cuda_ctx *ctx, const TiledAttn &p);

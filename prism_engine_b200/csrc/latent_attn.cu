@@ -419,26 +419,26 @@ int launch_latent_gather(prism_cuda_ctx *ctx, const LatentArgs &a, int32_t slot,
     return after_launch(ctx, "latent_gather_kernel");
 }
 
-constexpr int LP_Q = 128, LP_K = 64, LP_THREADS = 256;
-static size_t tiled_attn_smem(const TiledAttn &a, uint32_t vd) {
+constexpr int LP_Q = 128, LP_THREADS = 256;
+static size_t tiled_attn_smem(const TiledAttn &a, uint32_t vd, uint32_t kt) {
     const uint32_t dq = round_up_u32(a.dim + a.rot_dim, 16);
-    return ((size_t)(LP_Q + 2 * LP_K) * (dq + 8) + (size_t)2 * LP_K * (vd + 8)) * 2;
+    return ((size_t)(LP_Q + 2 * kt) * (dq + 8) + (size_t)2 * kt * (vd + 8)) * 2;
 }
 
-// 128 queries of one head per CTA (16 per warp), key tiles of 64 in two buffers, online softmax in fp32; the
+// 128 queries of one head per CTA (16 per warp), key tiles of LP_K in two buffers, online softmax in fp32; the
 // weights enter the second product as two bf16 parts.  Key and value heads start at multiples of 8 and may be
-// shared by a group of query heads; rows of a ring are taken by position.
-template <int VD>
-__global__ void __launch_bounds__(LP_THREADS) tiled_attn_kernel(const TiledAttn a) {
+// shared by a group of query heads; rows of a ring are taken by position.  The last queries, which see most, go first.
+template <int VD, int LP_K, int MIN_CTAS>
+__global__ void __launch_bounds__(LP_THREADS, MIN_CTAS) tiled_attn_kernel(const TiledAttn a) {
     extern __shared__ __align__(16) uint8_t lps[];
     pdl_launch_dependents();
     pdl_wait();
-    const uint32_t h = blockIdx.y, kh = h / a.group, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
+    const uint32_t h = blockIdx.x, kh = h / a.group, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
     const uint32_t dq = a.dim + a.rot_dim, dqp = round_up_u32(dq, 16), PQ = dqp + 8;
     constexpr uint32_t PV = VD + 8;
     bf16 *Qs = reinterpret_cast<bf16 *>(lps), *Ks = Qs + LP_Q * PQ, *Vs = Ks + 2 * LP_K * PQ;
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(Qs), sK = (uint32_t)__cvta_generic_to_shared(Ks), sV = (uint32_t)__cvta_generic_to_shared(Vs);
-    const uint32_t q0 = blockIdx.x * LP_Q, nq = min((uint32_t)LP_Q, a.n_rows - q0);
+    const uint32_t q0 = (gridDim.y - 1 - blockIdx.y) * LP_Q, nq = min((uint32_t)LP_Q, a.n_rows - q0);
     const int32_t first = max((int32_t)a.lo, window_first(a.window, (int32_t)(a.pos0 + q0)));
     const int32_t end = (int32_t)(a.pos0 + q0 + nq);  // keys first .. end-1
     const uint32_t n_kt = ((uint32_t)(end - first) + LP_K - 1) / LP_K;
@@ -450,12 +450,15 @@ __global__ void __launch_bounds__(LP_THREADS) tiled_attn_kernel(const TiledAttn 
         const int32_t k0 = first + (int32_t)(kt * LP_K);
         const uint32_t row0 = a.ring ? (uint32_t)k0 % a.ring : (uint32_t)k0 - a.lo;
         auto row_of = [&](uint32_t r) { return a.ring && row0 + r >= a.ring ? row0 + r - a.ring : row0 + r; };  // the visible keys fit into the ring
-        for (uint32_t i = tid; i < LP_K * q8; i += LP_THREADS) {
-            const uint32_t r = i / q8, c = i % q8, at = (buf * LP_K + r) * PQ + c * 8;
-            const int32_t key = k0 + (int32_t)r;
-            if (key < end && c < d8) cp_async16(sK + at * 2, a.kx + (size_t)row_of(r) * a.kx_pitch + kh * a.kx_head + c * 8);
-            else if (key < end && c < d8 + r8) cp_async16(sK + at * 2, a.krot + (size_t)row_of(r) * a.rot_dim + (c - d8) * 8);
-            else *reinterpret_cast<uint4 *>(Ks + at) = z4;
+        for (uint32_t r = tid >> a.shift; r < LP_K; r += LP_THREADS >> a.shift) {
+            const bool on = k0 + (int32_t)r < end;
+            const size_t row = row_of(r);
+            for (uint32_t c = tid & ((1u << a.shift) - 1); c < q8; c += 1u << a.shift) {
+                const uint32_t at = (buf * LP_K + r) * PQ + c * 8;
+                if (on && c < d8) cp_async16(sK + at * 2, a.kx + row * a.kx_pitch + kh * a.kx_head + c * 8);
+                else if (on && c < d8 + r8) cp_async16(sK + at * 2, a.krot + row * a.rot_dim + (c - d8) * 8);
+                else *reinterpret_cast<uint4 *>(Ks + at) = z4;
+            }
         }
         for (uint32_t i = tid; i < LP_K * (VD / 8); i += LP_THREADS) {
             const uint32_t r = i / (VD / 8), c = i % (VD / 8), at = (buf * LP_K + r) * PV + c * 8;
@@ -607,25 +610,27 @@ __global__ void __launch_bounds__(LP_THREADS) tiled_attn_kernel(const TiledAttn 
     }
 }
 
-template <int VD>
+template <int VD, int KT, int MIN_CTAS>
 static int launch_ta(prism_cuda_ctx *ctx, const TiledAttn &p) {
     static bool configured[PRISM_MAX_DEVICES] = {false};
     if (!configured[ctx->device]) {
-        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(tiled_attn_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024));
+        PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(tiled_attn_kernel<VD, KT, MIN_CTAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024));
         configured[ctx->device] = true;
     }
-    launch_pdl(ctx, "tiled_attn_kernel", tiled_attn_kernel<VD>, dim3((p.n_rows + LP_Q - 1) / LP_Q, p.heads), LP_THREADS, tiled_attn_smem(p, VD), p);
+    launch_pdl(ctx, "tiled_attn_kernel", tiled_attn_kernel<VD, KT, MIN_CTAS>, dim3(p.heads, (p.n_rows + LP_Q - 1) / LP_Q), LP_THREADS, tiled_attn_smem(p, VD, KT), p);
     return after_launch(ctx, "tiled_attn_kernel");
 }
 bool tiled_attn_ok(uint32_t dim, uint32_t vdim) { return dim <= 256 && vdim <= 256; }
-int launch_tiled_attn(prism_cuda_ctx *ctx, const TiledAttn &p) {
+int launch_tiled_attn(prism_cuda_ctx *ctx, const TiledAttn &args) {
+    TiledAttn p = args;
+    p.shift = row_shift(round_up_u32(p.dim + p.rot_dim, 16) / 8);
     const uintptr_t ptrs = reinterpret_cast<uintptr_t>(p.kx) | reinterpret_cast<uintptr_t>(p.vx) | reinterpret_cast<uintptr_t>(p.krot);
     if (!tiled_attn_ok(p.dim + p.rot_dim, p.vdim) || (ptrs & 15) || p.kx_pitch % 8 || p.vx_pitch % 8 || p.kx_head % 8 || p.vx_head % 8 || p.rot_dim % 8 ||
         (p.rot_dim && p.dim % 8) || p.out_pitch % 2 || (p.gate && (p.gate_pitch % 2 || p.vdim % 2)))
         return fail(ctx, PRISM_E_ARG, "tiled attention: keys and values need 16-byte rows and heads of at most 256");
-    if (p.vdim <= 64) return launch_ta<64>(ctx, p);
-    if (p.vdim <= 128) return launch_ta<128>(ctx, p);
-    return launch_ta<256>(ctx, p);
+    if (p.vdim <= 64) return launch_ta<64, 64, 2>(ctx, p);
+    if (p.vdim <= 128) return launch_ta<128, 32, 2>(ctx, p);
+    return launch_ta<256, 64, 1>(ctx, p);
 }
 
 bool latent_expand_ok(const LatentArgs &a) {

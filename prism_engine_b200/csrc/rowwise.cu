@@ -54,7 +54,7 @@ __device__ __forceinline__ float as_act(float v, const bf16 *) { return __bfloat
 // Thread: V channels of a strip of tokens; with TAPS the last inputs stay in registers.  Only the first strip reaches
 // back before the portion, and the same threads leave the portion's last inputs in the ring after they have read what
 // was there.
-constexpr int CV_THREADS = 128, CV_STRIP = 16, CV_U = 8;
+constexpr int CV_THREADS = 128, CV_STRIP = 16, CV_U = 4;
 template <typename TA, int V, int TAPS>
 __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, const RowMap rows, uint32_t n, uint32_t strip) {
     pdl_launch_dependents();
@@ -75,11 +75,15 @@ __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, 
         if (pos < 0) return Vals<V>{};
         return u >= 0 ? ldv<V>(x + (size_t)u * a.x_pitch) : ldv<V>(ring + (size_t)((uint32_t)pos % a.taps) * a.channels);
     };
-    auto finish = [&](int32_t t, const Vals<V> &s, const Vals<V> &cur) {
+    auto finish = [&](TA *to, const Vals<V> &s, const Vals<V> &cur) {
         Vals<V> o;
 #pragma unroll
-        for (int i = 0; i < V; i++) o.v[i] = a.silu ? s.v[i] * sigmoid_f(s.v[i]) : cur.v[i] + s.v[i];
-        stv<V>(y + (size_t)t * a.y_pitch, o);
+        for (int i = 0; i < V; i++) {
+            if (!a.silu) o.v[i] = cur.v[i] + s.v[i];
+            else if (sizeof(TA) == 2) o.v[i] = s.v[i] * __fdividef(1.0f, 1.0f + __expf(-s.v[i]));  // rounded to 16 bits
+            else o.v[i] = s.v[i] * sigmoid_f(s.v[i]);
+        }
+        stv<V>(to, o);
     };
     if constexpr (TAPS > 0) {
         Vals<V> wr[TAPS], h[TAPS];  // h[j]: the input TAPS - 1 - j tokens ago
@@ -88,13 +92,15 @@ __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, 
         pdl_wait();
 #pragma unroll
         for (int j = 1; j < TAPS; j++) h[j] = earlier(t0 - TAPS + j);
+        const TA *xt = x + (size_t)t0 * a.x_pitch;
+        TA *yt = y + (size_t)t0 * a.y_pitch;
         for (int32_t t = t0; t < t1; t += CV_U) {
             Vals<V> in[CV_U];
 #pragma unroll
-            for (int k = 0; k < CV_U; k++)
-                if (t + k < t1) in[k] = ldv<V>(x + (size_t)(t + k) * a.x_pitch);
+            for (int k = 0; k < CV_U; k++, xt += a.x_pitch)
+                if (t + k < t1) in[k] = ldv<V>(xt);
 #pragma unroll
-            for (int k = 0; k < CV_U; k++) {
+            for (int k = 0; k < CV_U; k++, yt += a.y_pitch) {
                 if (t + k >= t1) break;
 #pragma unroll
                 for (int j = 0; j + 1 < TAPS; j++) h[j] = h[j + 1];
@@ -104,7 +110,7 @@ __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, 
                 for (int j = 0; j < TAPS; j++)
 #pragma unroll
                     for (int i = 0; i < V; i++) s.v[i] = fmaf(wr[j].v[i], h[j].v[i], s.v[i]);
-                finish(t + k, s, in[k]);
+                finish(yt, s, in[k]);
             }
         }
     } else {
@@ -116,7 +122,7 @@ __global__ void __launch_bounds__(CV_THREADS) conv_seq_kernel(const ConvArgs a, 
 #pragma unroll
                 for (int i = 0; i < V; i++) s.v[i] = fmaf(wj.v[i], h.v[i], s.v[i]);
             }
-            finish(t, s, ldv<V>(x + (size_t)t * a.x_pitch));
+            finish(y + (size_t)t * a.y_pitch, s, ldv<V>(x + (size_t)t * a.x_pitch));
         }
     }
     if (blockIdx.y == 0)
@@ -131,16 +137,17 @@ static int run_conv(prism_cuda_ctx *ctx, const ConvArgs &a, const RowMap &rows, 
         at |= reinterpret_cast<uintptr_t>(a.piece[i].x) | reinterpret_cast<uintptr_t>(a.piece[i].y);
         odd |= a.piece[i].channels | a.piece[i].c0;
     }
-    const bool vec = !(at & 15) && !(odd & 3);
+    const uint32_t v = (at & 15) || (odd & 3) ? 1 : 4;
     uint32_t blocks = 0;
-    for (uint32_t i = 0; i < a.pieces; i++) blocks += (a.piece[i].channels + CV_THREADS * (vec ? 4 : 1) - 1) / (CV_THREADS * (vec ? 4 : 1));
+    for (uint32_t i = 0; i < a.pieces; i++) blocks += (a.piece[i].channels + CV_THREADS * v - 1) / (CV_THREADS * v);
     const uint32_t strip = std::max((uint32_t)CV_STRIP, a.taps);
     const dim3 grid(blocks, (n + strip - 1) / strip);
-    if (!vec) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 1, 0>, grid, CV_THREADS, 0, a, rows, n, strip);
-    else if (a.taps == 2) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 2>, grid, CV_THREADS, 0, a, rows, n, strip);
-    else if (a.taps == 3) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 3>, grid, CV_THREADS, 0, a, rows, n, strip);
-    else if (a.taps == 4) launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 4>, grid, CV_THREADS, 0, a, rows, n, strip);
-    else launch_pdl(ctx, "conv_seq_kernel", conv_seq_kernel<TA, 4, 0>, grid, CV_THREADS, 0, a, rows, n, strip);
+    auto run = [&](auto kernel) { launch_pdl(ctx, "conv_seq_kernel", kernel, grid, dim3(CV_THREADS), 0, a, rows, n, strip); };
+    if (v == 1) run(conv_seq_kernel<TA, 1, 0>);
+    else if (a.taps == 2) run(conv_seq_kernel<TA, 4, 2>);
+    else if (a.taps == 3) run(conv_seq_kernel<TA, 4, 3>);
+    else if (a.taps == 4) run(conv_seq_kernel<TA, 4, 4>);
+    else run(conv_seq_kernel<TA, 4, 0>);
     return after_launch(ctx, "conv_seq_kernel");
 }
 int launch_conv_seq(prism_cuda_ctx *ctx, const ConvArgs &a, const RowMap &rows, uint32_t n_rows, bool act32) {
