@@ -284,17 +284,18 @@ constexpr uint32_t DC_SCALARS = 256;                              // floats: e[6
 constexpr size_t DC_ITEM = 4 * DC_C * DC_C * 2 + DC_SCALARS * 4;  // T hi, T lo, P hi, P lo, scalars
 
 // Rows of a chunk into shared memory, zeros past row nt and column `valid`; 2^sh threads take a row.
+template <int THREADS>
 __device__ __forceinline__ void load_rows(bf16 *dst, uint32_t pitch, uint32_t cols, const bf16 *src, uint32_t src_pitch, uint32_t nt, uint32_t valid,
                                           bool vec, uint32_t sh) {
     const uint32_t s = (uint32_t)__cvta_generic_to_shared(dst);
     if (vec) {
-        for (uint32_t r = threadIdx.x >> sh; r < DC_C; r += DL_THREADS >> sh)
+        for (uint32_t r = threadIdx.x >> sh; r < DC_C; r += THREADS >> sh)
             for (uint32_t c = (threadIdx.x & ((1u << sh) - 1)) * 8; c < cols; c += 8u << sh) {
                 if (r < nt && c < valid) cp_async16(s + (r * pitch + c) * 2, src + (size_t)r * src_pitch + c);
                 else *reinterpret_cast<uint4 *>(dst + r * pitch + c) = make_uint4(0, 0, 0, 0);
             }
     } else {
-        for (uint32_t i = threadIdx.x; i < DC_C * cols; i += DL_THREADS) {
+        for (uint32_t i = threadIdx.x; i < DC_C * cols; i += THREADS) {
             const uint32_t r = i / cols, c = i % cols;
             dst[r * pitch + c] = r < nt && c < valid ? src[(size_t)r * src_pitch + c] : __float2bfloat16_rn(0.0f);
         }
@@ -312,8 +313,8 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs 
     float *A = reinterpret_cast<float *>(dps), *X = A + DC_C * PA, *Y = X + DC_C * PA;  // X and Y share their place with Q and K
     bf16 *Q = reinterpret_cast<bf16 *>(X), *K = Q + DC_C * PD;
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(Q), sK = (uint32_t)__cvta_generic_to_shared(K);
-    load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
-    load_rows(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+    load_rows<DL_THREADS>(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+    load_rows<DL_THREADS>(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
     cp_async_commit();
     if (warp == 0) {  // running sums of the logarithms
         float carry = 0.0f;
@@ -471,8 +472,13 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prep_kernel(const DeltaArgs 
 }
 
 // Grid: (slice of 32 value columns, head).  The slice of the state lives in mma accumulators from the first chunk to
-// the last; nbuf 2: the next chunk loads under this one.
-__global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs a, int32_t slot, uint32_t dpad, uint32_t vec, uint32_t nbuf, uint32_t sh) {
+// the last; nbuf 2: the next chunk loads under this one.  Sixteen warps: 16 tokens x 8 value columns each, and of the
+// state 16 (for more than 128 rows 2 x 16) rows x 16 columns.
+constexpr int DC_THREADS = 512;
+// DP: the padded key size when it is a usual one, else 0.
+template <int DP>
+__global__ void __launch_bounds__(DC_THREADS) delta_chunk_kernel(const DeltaArgs a, int32_t slot, uint32_t dpad_, uint32_t vec, uint32_t nbuf, uint32_t sh) {
+    const uint32_t dpad = DP ? DP : dpad_;
     extern __shared__ __align__(16) uint8_t dcs[];
     pdl_launch_dependents();
     pdl_wait();
@@ -484,25 +490,26 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
     auto sm = [](const bf16 *p) { return (uint32_t)__cvta_generic_to_shared(p); };
     const uint32_t sSh = sm(Sh), sSl = sm(Sl), sWh = sm(Wh), sWl = sm(Wl), sUh = sm(Uh), sUl = sm(Ul), sHh = sm(Hh), sHl = sm(Hl);
     float *S = a.state + ((size_t)slot * a.heads + h) * a.dim * a.vdim;
-    float st[2][4][4];  // warp w holds rows 16 (w + 8 m) .. +16 of the key dimension
+    const uint32_t sw = warp & 7, s0 = (warp >> 3) * 16;
+    float st[2][2][4];  // rows 16 (sw + 8 m) .. +16 of the key dimension, value columns s0 .. +16
 #pragma unroll
     for (int m = 0; m < 2; m++)
 #pragma unroll
-        for (int n = 0; n < 4; n++)
+        for (int n = 0; n < 2; n++)
 #pragma unroll
             for (int i = 0; i < 4; i++) {
-                const uint32_t d = (warp + 8 * m) * 16 + g8 + 8 * (i >> 1), c = v0 + n * 8 + 2 * t4 + (i & 1);
+                const uint32_t d = (sw + 8 * m) * 16 + g8 + 8 * (i >> 1), c = v0 + s0 + n * 8 + 2 * t4 + (i & 1);
                 st[m][n][i] = d < a.dim && c < a.vdim ? S[(size_t)d * a.vdim + c] : 0.0f;
             }
     const uint32_t n_mt = dpad / 16;
     auto load_chunk = [&](uint32_t r0, uint32_t buf) {
         const uint32_t nt = min((uint32_t)DC_C, a.rows - r0);
         bf16 *Q = tiles + buf * TILE, *K = Q + DC_C * PD, *V = K + DC_C * PD, *TP = V + DC_C * DC_PV, *sc = TP + 4 * DC_C * DC_PT;
-        load_rows(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
-        load_rows(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
-        load_rows(V, DC_PV, DL_VS, reinterpret_cast<const bf16 *>(a.v) + (size_t)r0 * a.pitch + h * a.vdim + v0, a.pitch, nt, a.vdim - v0, vec, 2);
+        load_rows<DC_THREADS>(Q, PD, dpad, reinterpret_cast<const bf16 *>(a.q) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+        load_rows<DC_THREADS>(K, PD, dpad, reinterpret_cast<const bf16 *>(a.k) + (size_t)r0 * a.pitch + kh * a.dim, a.pitch, nt, a.dim, vec, sh);
+        load_rows<DC_THREADS>(V, DC_PV, DL_VS, reinterpret_cast<const bf16 *>(a.v) + (size_t)r0 * a.pitch + h * a.vdim + v0, a.pitch, nt, a.vdim - v0, vec, 2);
         const uint8_t *item = reinterpret_cast<const uint8_t *>(a.chunk_scratch) + ((size_t)(r0 / DC_C) * a.heads + h) * DC_ITEM;
-        for (uint32_t i = tid; i < 4 * DC_C * 8; i += DL_THREADS)
+        for (uint32_t i = tid; i < 4 * DC_C * 8; i += DC_THREADS)
             cp_async16(sm(TP) + ((i >> 3) * DC_PT + (i & 7) * 8) * 2, item + (size_t)i * 16);
         if (tid < DC_SCALARS / 4) cp_async16(sm(sc) + tid * 16, item + 4 * DC_C * DC_C * 2 + tid * 16);
         cp_async_commit();
@@ -521,14 +528,14 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
         constexpr uint32_t LO = DC_C * DC_PT * 2;  // bytes from the high to the low part
 #pragma unroll
         for (int m = 0; m < 2; m++)
-            if (warp + 8 * m < n_mt) {
+            if (sw + 8 * m < n_mt) {
 #pragma unroll
-                for (int n = 0; n < 4; n++)
+                for (int n = 0; n < 2; n++)
 #pragma unroll
                     for (int i = 0; i < 2; i++) {
                         uint32_t hi, lo;
                         split_bf16(st[m][n][2 * i], st[m][n][2 * i + 1], hi, lo);
-                        const uint32_t at = ((warp + 8 * m) * 16 + g8 + 8 * i) * DC_PV + n * 8 + 2 * t4;
+                        const uint32_t at = ((sw + 8 * m) * 16 + g8 + 8 * i) * DC_PV + s0 + n * 8 + 2 * t4;
                         *reinterpret_cast<uint32_t *>(Sh + at) = hi;
                         *reinterpret_cast<uint32_t *>(Sl + at) = lo;
                     }
@@ -536,123 +543,108 @@ __global__ void __launch_bounds__(DL_THREADS) delta_chunk_kernel(const DeltaArgs
         cp_async_wait<0>();
         __syncthreads();  // this chunk and the state are there; every warp is done with the previous chunk
         if (nbuf == 2 && r0 + DC_C < a.rows) load_chunk(r0 + DC_C, buf ^ 1);
-        const uint32_t i0 = (warp & 3) * 16, c0 = (warp >> 2) * 16;  // rows and value columns of this warp
-        float ks[2][4] = {}, qs[2][4] = {}, kl[2][4] = {}, ql[2][4] = {};  // products with the state's high and low parts
+        const uint32_t i0 = (warp & 3) * 16, c0 = (warp >> 2) * 8;  // rows and value columns of this warp
+        float ks[4] = {}, qs[4] = {}, kl[4] = {}, ql[4] = {};       // products with the state's high and low parts
+#pragma unroll(DP ? DP / 16 : 2)
         for (uint32_t d = 0; d < dpad; d += 16) {
-            uint32_t ak[4], aq[4], b[4];
-            ldsm_x4(ak, sK + ((i0 + (lane & 15)) * PD + d + (lane >> 4) * 8) * 2);
-            ldsm_x4(aq, sQ + ((i0 + (lane & 15)) * PD + d + (lane >> 4) * 8) * 2);
-            ldsm_x4_t(b, sSh + ((d + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2);
-            mma_bf16(ks[0], ak, b[0], b[1]);
-            mma_bf16(ks[1], ak, b[2], b[3]);
-            mma_bf16(qs[0], aq, b[0], b[1]);
-            mma_bf16(qs[1], aq, b[2], b[3]);
-            ldsm_x4_t(b, sSl + ((d + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2);
-            mma_bf16(kl[0], ak, b[0], b[1]);
-            mma_bf16(kl[1], ak, b[2], b[3]);
-            mma_bf16(ql[0], aq, b[0], b[1]);
-            mma_bf16(ql[1], aq, b[2], b[3]);
+            uint32_t ak[4], aq[4], bh[2], bl[2];
+            const uint32_t at = ((i0 + (lane & 15)) * PD + d + (lane >> 4) * 8) * 2, bt = ((d + (lane & 15)) * DC_PV + c0) * 2;
+            ldsm_x4(ak, sK + at);
+            ldsm_x4(aq, sQ + at);
+            ldsm_x2_t(bh, sSh + bt);
+            ldsm_x2_t(bl, sSl + bt);
+            mma_bf16(ks, ak, bh[0], bh[1]);
+            mma_bf16(qs, aq, bh[0], bh[1]);
+            mma_bf16(kl, ak, bl[0], bl[1]);
+            mma_bf16(ql, aq, bl[0], bl[1]);
         }
-#pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                ks[n][i] += kl[n][i];
-                qs[n][i] += ql[n][i];
-            }
-#pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                const uint32_t row = i0 + g8 + 8 * i, at = row * DC_PV + c0 + n * 8 + 2 * t4;
-                const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(V + at));
-                const float e = sc[row];
-                uint32_t hi, lo;
-                split_bf16(fmaf(-e, ks[n][2 * i], v.x), fmaf(-e, ks[n][2 * i + 1], v.y), hi, lo);
-                *reinterpret_cast<uint32_t *>(Wh + at) = hi;
-                *reinterpret_cast<uint32_t *>(Wl + at) = lo;
-            }
+        const uint32_t row = i0 + g8, at0 = row * DC_PV + c0 + 2 * t4, at1 = at0 + 8 * DC_PV;  // this lane's two rows
+        {
+            const float2 va = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(V + at0)), vb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(V + at1));
+            const float ea = sc[row], eb = sc[row + 8];
+            uint32_t hi, lo;
+            split_bf16(fmaf(-ea, ks[0] + kl[0], va.x), fmaf(-ea, ks[1] + kl[1], va.y), hi, lo);
+            *reinterpret_cast<uint32_t *>(Wh + at0) = hi;
+            *reinterpret_cast<uint32_t *>(Wl + at0) = lo;
+            split_bf16(fmaf(-eb, ks[2] + kl[2], vb.x), fmaf(-eb, ks[3] + kl[3], vb.y), hi, lo);
+            *reinterpret_cast<uint32_t *>(Wh + at1) = hi;
+            *reinterpret_cast<uint32_t *>(Wl + at1) = lo;
+        }
         __syncthreads();
-        // a lower triangular matrix (high and low parts at m) times columns c0 .. +16 of a right-hand side
-        auto tri = [&](float (&o)[2][4], uint32_t m, uint32_t bh, uint32_t bl) {
-            float p[2][4] = {}, q[2][4] = {};
+        // a lower triangular matrix (high and low parts at m) times columns c0 .. +8 of a right-hand side
+        auto tri = [&](float (&o)[4], uint32_t m, uint32_t bh, uint32_t bl) {
+            float p[4] = {}, q[4] = {};
             for (uint32_t j = 0; j <= i0; j += 16) {
-                uint32_t xh[4], xl[4], b[4];
-                const uint32_t at = ((i0 + (lane & 15)) * DC_PT + j + (lane >> 4) * 8) * 2, bt = ((j + (lane & 15)) * DC_PV + c0 + (lane >> 4) * 8) * 2;
+                uint32_t xh[4], xl[4], yh[2], yl[2];
+                const uint32_t at = ((i0 + (lane & 15)) * DC_PT + j + (lane >> 4) * 8) * 2, bt = ((j + (lane & 15)) * DC_PV + c0) * 2;
                 ldsm_x4(xh, m + at);
                 ldsm_x4(xl, m + LO + at);
-                ldsm_x4_t(b, bh + bt);
-                mma_bf16(o[0], xh, b[0], b[1]);
-                mma_bf16(o[1], xh, b[2], b[3]);
-                mma_bf16(p[0], xl, b[0], b[1]);
-                mma_bf16(p[1], xl, b[2], b[3]);
-                ldsm_x4_t(b, bl + bt);
-                mma_bf16(q[0], xh, b[0], b[1]);
-                mma_bf16(q[1], xh, b[2], b[3]);
+                ldsm_x2_t(yh, bh + bt);
+                ldsm_x2_t(yl, bl + bt);
+                mma_bf16(o, xh, yh[0], yh[1]);
+                mma_bf16(p, xl, yh[0], yh[1]);
+                mma_bf16(q, xh, yl[0], yl[1]);
             }
 #pragma unroll
-            for (int n = 0; n < 2; n++)
-#pragma unroll
-                for (int i = 0; i < 4; i++) o[n][i] += p[n][i] + q[n][i];
+            for (int i = 0; i < 4; i++) o[i] += p[i] + q[i];
         };
-        float u[2][4] = {};
+        float u[4] = {};
         tri(u, sT, sWh, sWl);
 #pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                const uint32_t row = i0 + g8 + 8 * i, at = row * DC_PV + c0 + n * 8 + 2 * t4;
-                const float w = sc[2 * DC_C + row];
-                uint32_t hi, lo;
-                split_bf16(u[n][2 * i], u[n][2 * i + 1], hi, lo);
-                *reinterpret_cast<uint32_t *>(Uh + at) = hi;
-                *reinterpret_cast<uint32_t *>(Ul + at) = lo;
-                split_bf16(u[n][2 * i] * w, u[n][2 * i + 1] * w, hi, lo);
-                *reinterpret_cast<uint32_t *>(Hh + at) = hi;
-                *reinterpret_cast<uint32_t *>(Hl + at) = lo;
-            }
+        for (int i = 0; i < 2; i++) {
+            const uint32_t at = i ? at1 : at0;
+            const float w = sc[2 * DC_C + row + 8 * i];
+            uint32_t hi, lo;
+            split_bf16(u[2 * i], u[2 * i + 1], hi, lo);
+            *reinterpret_cast<uint32_t *>(Uh + at) = hi;
+            *reinterpret_cast<uint32_t *>(Ul + at) = lo;
+            split_bf16(u[2 * i] * w, u[2 * i + 1] * w, hi, lo);
+            *reinterpret_cast<uint32_t *>(Hh + at) = hi;
+            *reinterpret_cast<uint32_t *>(Hl + at) = lo;
+        }
         __syncthreads();
-        float o[2][4] = {};
+        float o[4] = {};
         tri(o, sP, sUh, sUl);
 #pragma unroll
-        for (int n = 0; n < 2; n++)
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const uint32_t row = i0 + g8 + 8 * (i >> 1), c = v0 + c0 + n * 8 + 2 * t4 + (i & 1);
-                if (row < nt && c < a.vdim) a.o32[(size_t)(r0 + row) * a.heads * a.vdim + h * a.vdim + c] = fmaf(sc[DC_C + row], qs[n][i], o[n][i]);
-            }
+        for (int i = 0; i < 4; i++) {
+            const uint32_t t = row + 8 * (i >> 1), c = v0 + c0 + 2 * t4 + (i & 1);
+            if (t < nt && c < a.vdim) a.o32[(size_t)(r0 + t) * a.heads * a.vdim + h * a.vdim + c] = fmaf(sc[DC_C + t], qs[i] + ql[i], o[i]);
+        }
         const float gc = sc[3 * DC_C];
 #pragma unroll
         for (int m = 0; m < 2; m++)
-            if (warp + 8 * m < n_mt) {
+            if (sw + 8 * m < n_mt) {
+                float low[2][4] = {};
 #pragma unroll
-                for (int n = 0; n < 4; n++)
+                for (int n = 0; n < 2; n++)
 #pragma unroll
                     for (int i = 0; i < 4; i++) st[m][n][i] *= gc;
+#pragma unroll
                 for (uint32_t j = 0; j < DC_C; j += 16) {
                     uint32_t ak[4], b[4];
-                    ldsm_x4_t(ak, sK + ((j + (lane >> 4) * 8 + (lane & 7)) * PD + (warp + 8 * m) * 16 + ((lane >> 3) & 1) * 8) * 2);
-#pragma unroll
-                    for (int n = 0; n < 2; n++) {
-                        const uint32_t bt = ((j + (lane & 15)) * DC_PV + n * 16 + (lane >> 4) * 8) * 2;
-                        ldsm_x4_t(b, sHh + bt);
-                        mma_bf16(st[m][2 * n], ak, b[0], b[1]);
-                        mma_bf16(st[m][2 * n + 1], ak, b[2], b[3]);
-                        ldsm_x4_t(b, sHl + bt);
-                        mma_bf16(st[m][2 * n], ak, b[0], b[1]);
-                        mma_bf16(st[m][2 * n + 1], ak, b[2], b[3]);
-                    }
+                    const uint32_t bt = ((j + (lane & 15)) * DC_PV + s0 + (lane >> 4) * 8) * 2;
+                    ldsm_x4_t(ak, sK + ((j + (lane >> 4) * 8 + (lane & 7)) * PD + (sw + 8 * m) * 16 + ((lane >> 3) & 1) * 8) * 2);
+                    ldsm_x4_t(b, sHh + bt);
+                    mma_bf16(st[m][0], ak, b[0], b[1]);
+                    mma_bf16(st[m][1], ak, b[2], b[3]);
+                    ldsm_x4_t(b, sHl + bt);
+                    mma_bf16(low[0], ak, b[0], b[1]);
+                    mma_bf16(low[1], ak, b[2], b[3]);
                 }
+#pragma unroll
+                for (int n = 0; n < 2; n++)
+#pragma unroll
+                    for (int i = 0; i < 4; i++) st[m][n][i] += low[n][i];
             }
         if (nbuf == 2) buf ^= 1;
     }
 #pragma unroll
     for (int m = 0; m < 2; m++)
 #pragma unroll
-        for (int n = 0; n < 4; n++)
+        for (int n = 0; n < 2; n++)
 #pragma unroll
             for (int i = 0; i < 4; i++) {
-                const uint32_t d = (warp + 8 * m) * 16 + g8 + 8 * (i >> 1), c = v0 + n * 8 + 2 * t4 + (i & 1);
+                const uint32_t d = (sw + 8 * m) * 16 + g8 + 8 * (i >> 1), c = v0 + s0 + n * 8 + 2 * t4 + (i & 1);
                 if (d < a.dim && c < a.vdim) S[(size_t)d * a.vdim + c] = st[m][n][i];
             }
 }
@@ -668,7 +660,9 @@ static int configure(prism_cuda_ctx *ctx) {
     PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_seq_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
     PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_seq_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
     PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
-    PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
+    PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_chunk_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
+    PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_chunk_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
+    PRISM_CUDA_TRY(ctx, cudaFuncSetAttribute(delta_chunk_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)DL_SMEM_MAX));
     configured[ctx->device] = true;
     return PRISM_OK;
 }
@@ -687,7 +681,10 @@ int launch_delta_seq(prism_cuda_ctx *ctx, const DeltaArgs &a, const RowMap &rows
         PRISM_TRY(after_launch(ctx, "delta_prep_kernel"));
         const size_t tile = qk + (size_t)(DC_C * DC_PV + 4 * DC_C * DC_PT) * 2 + DC_SCALARS * 4, rest = (size_t)(2 * dpad + 6 * DC_C) * DC_PV * 2;
         const uint32_t nbuf = 2 * tile + rest <= DL_SMEM_MAX ? 2 : 1;
-        launch_pdl(ctx, "delta_chunk_kernel", delta_chunk_kernel, grid, DL_THREADS, nbuf * tile + rest, a, rows.slot0, dpad, vec, nbuf, sh);
+        auto chunk = [&](auto kernel) { launch_pdl(ctx, "delta_chunk_kernel", kernel, grid, DC_THREADS, nbuf * tile + rest, a, rows.slot0, dpad, vec, nbuf, sh); };
+        if (dpad == 64) chunk(delta_chunk_kernel<64>);
+        else if (dpad == 128) chunk(delta_chunk_kernel<128>);
+        else chunk(delta_chunk_kernel<0>);
         PRISM_TRY(after_launch(ctx, "delta_chunk_kernel"));
     } else {
         const size_t smem = (size_t)a.dim * (2 + DL_VS) * 4;

@@ -85,6 +85,14 @@ static void name_conv(LayeredModel *m, const std::string &name, uint32_t channel
     d.mean = 0.2f;
 }
 
+// A tensor that a checkpoint may carry although no sublayer reads it.
+static void name_unused(LayeredModel *m, const std::string &name, uint64_t rows, uint64_t cols) {
+    LayeredDst &d = m->names[name];
+    d.rows = rows;
+    d.cols = cols;
+    d.bound = true;
+}
+
 static uint32_t ring_size(const LayeredModel *m, uint32_t window) {
     return window ? (uint32_t)std::min<uint64_t>(m->c.max_seq, (uint64_t)window - 1 + m->chunk) : m->c.max_seq;
 }
@@ -308,6 +316,13 @@ static int build_sequential_layer(prism_cuda_engine *e, LayeredLayer &ly, uint32
         m->act_pitch = std::max(m->act_pitch, ly.down.k_pad);
         PRISM_TRY(build_sublayer(e, p, "2", ly.in2, ly.seg_gate2, ly.gate2_b, ly.canon2, ly.ring2));
         m->proj_pitch = std::max(m->proj_pitch, ly.in2.n_tiles * 128);
+    } else {
+        name_unused(m, p + "norm2", D, 1);
+        if (m->c.canon_taps) name_unused(m, p + "canon2", D, m->c.canon_taps);
+        if (m->c.gated_residual) {
+            name_unused(m, p + "rg2", D, D);
+            name_unused(m, p + "rg2.b", D, 1);
+        }
     }
     if (m->c.depth_average) PRISM_TRY(name_vector(e, p + "dwa", i + 2, ly.avg, 0.5f));
     return PRISM_OK;
@@ -419,6 +434,9 @@ static int build_model(prism_cuda_engine *e, const prism_layer_config *layers) {
         PRISM_TRY(model_alloc(e, m->rows_scratch.ml, ml * m->rows_scratch.rows_cap));
     }
     m->slot_pos.assign(c.max_batch, -1);
+    PRISM_CUDA_TRY(e->ctx, cudaStreamCreateWithFlags(&m->side, cudaStreamNonBlocking));
+    PRISM_CUDA_TRY(e->ctx, cudaEventCreateWithFlags(&m->fork, cudaEventDisableTiming));
+    PRISM_CUDA_TRY(e->ctx, cudaEventCreateWithFlags(&m->join, cudaEventDisableTiming));
     return PRISM_OK;
 }
 
@@ -428,6 +446,9 @@ void layered_destroy(prism_cuda_engine *e) {
     cudaFree(m->ex_lat);
     cudaFree(m->ex_krot);
     cudaFree(m->ex_kv);
+    if (m->fork) cudaEventDestroy(m->fork);
+    if (m->join) cudaEventDestroy(m->join);
+    if (m->side) cudaStreamDestroy(m->side);
     delete m;
     e->lm = nullptr;
 }
@@ -709,8 +730,37 @@ static int feed_forward(prism_cuda_engine *e, LayeredLayer &ly, const DenseIn &i
     return launch_moe_gemm_tc5(ctx, ly.down, plan, act, yo, pairs);
 }
 
-static int forward_sequential(prism_cuda_engine *e, const RowMap &rows, uint32_t n, bool seq) {
+// All mixers of a layer.  In a prompt portion the second of a pair runs on a stream of its own: its chunks follow one
+// another on a part of the GPU.
+static int run_mixers(prism_cuda_engine *e, LayeredLayer &ly, const RowMap &rows, uint32_t n, bool seq) {
     prism_cuda_ctx *ctx = e->ctx;
+    LayeredModel *m = e->lm;
+    auto whole = [&](LayeredMixer &mx) -> int {
+        PRISM_TRY(run_mixer(e, ly, mx, rows, n, seq));
+        if (mx.c.mixer != PRISM_MIXER_LIGHTNING) return PRISM_OK;
+        DenseIn h{};
+        h.x = at(m, m->cat, mx.col); h.pitch = m->cat_pitch;
+        lightning_norm(m, ly, mx, h);
+        return launch_dense_norm(ctx, h, at(m, m->cat, mx.col), m->cat_pitch, n, m->act32);
+    };
+    if (!seq || ly.mix.size() != 2 || ly.mix[0].c.mixer == ly.mix[1].c.mixer || n <= DENSE_GEMV_ROWS) {  // mixers of a kind share scratch
+        for (LayeredMixer &mx : ly.mix) PRISM_TRY(whole(mx));
+        return PRISM_OK;
+    }
+    const cudaStream_t main = ctx->stream;
+    PRISM_CUDA_TRY(ctx, cudaEventRecord(m->fork, main));
+    PRISM_CUDA_TRY(ctx, cudaStreamWaitEvent(m->side, m->fork, 0));
+    ctx->stream = m->side;
+    const int rc = whole(ly.mix[1]);
+    ctx->stream = main;
+    PRISM_TRY(rc);
+    PRISM_CUDA_TRY(ctx, cudaEventRecord(m->join, m->side));
+    PRISM_TRY(whole(ly.mix[0]));
+    PRISM_CUDA_TRY(ctx, cudaStreamWaitEvent(main, m->join, 0));
+    return PRISM_OK;
+}
+
+static int forward_sequential(prism_cuda_engine *e, const RowMap &rows, uint32_t n, bool seq) {
     LayeredModel *m = e->lm;
     const uint32_t D = m->c.width, L = m->c.num_layers;
     DenseIn in{};  // what the sublayers read: the convolved norm, and the norm itself
@@ -729,15 +779,7 @@ static int forward_sequential(prism_cuda_engine *e, const RowMap &rows, uint32_t
         DenseOut outs[DENSE_MAX_SEGS];
         in_outs(m, ly, outs);
         PRISM_TRY(linear(e, ly.in, in, outs, n, nullptr, 0));
-        for (LayeredMixer &mx : ly.mix) {
-            PRISM_TRY(run_mixer(e, ly, mx, rows, n, seq));
-            if (mx.c.mixer == PRISM_MIXER_LIGHTNING) {
-                DenseIn h{};
-                h.x = at(m, m->cat, mx.col); h.pitch = m->cat_pitch;
-                lightning_norm(m, ly, mx, h);
-                PRISM_TRY(launch_dense_norm(ctx, h, at(m, m->cat, mx.col), m->cat_pitch, n, m->act32));
-            }
-        }
+        PRISM_TRY(run_mixers(e, ly, rows, n, seq));
         DenseIn oi{};
         oi.x = m->cat; oi.pitch = m->cat_pitch;
         const bool pair = ly.mix.size() > 1;

@@ -82,6 +82,8 @@ struct LayeredModel {
     uint32_t aux_pitch = 0, y_pitch = 0, act_pitch = 0, conv_pitch = 0, o32_width = 0;
     size_t pairs_cap = 0;                          // rows of the experts' buffers
     MoePlan plan{};                                // buffers; experts and top are the layer's
+    cudaStream_t side = nullptr;                   // the second mixer of a pair, in prompt portions
+    cudaEvent_t fork = nullptr, join = nullptr;
     // expanded keys and values of a prompt portion, grown on demand
     bf16 *ex_lat = nullptr, *ex_krot = nullptr, *ex_kv = nullptr;
     size_t ex_lat_n = 0, ex_krot_n = 0, ex_kv_n = 0;

@@ -487,7 +487,8 @@ def test_errors_are_reported(backend):
     eng = U.engine(backend, cfg, lacking, max_seq=40)
     with pytest.raises(p.PrismCudaError, match="l2.mlp.e4.down"):
         eng.generate([1, 2], 1)
-    for bad in ("l2.mlp.e5.down", "l1.norm2", "l0.mlp.up"):
+    eng.set_tensor("l1.norm2", U.bits(w["l0.norm1"]))  # of a layer without feed-forward: taken, not needed
+    for bad in ("l2.mlp.e5.down", "l1.mlp.router", "l0.mlp.up"):
         with pytest.raises(p.PrismCudaError, match="miss"):
             eng.set_tensor(bad, U.bits(w["l0.norm1"]))
     with pytest.raises(p.PrismCudaError, match="needs"):
