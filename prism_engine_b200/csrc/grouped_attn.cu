@@ -35,10 +35,8 @@ int launch_grouped_append(prism_cuda_ctx *ctx, const GroupedArgs &a, const void 
     return after_launch(ctx, "grouped_append_kernel");
 }
 
-// Grid: (splits, key/value head x part of its query heads, row); a cluster along x shares the row's keys.  `lpk`
-// lanes share a key in the scores, one thread owns eight value columns of some keys in the weighted sum; GR
-// query heads go together.  The CTAs of a cluster exchange maxima, sums and partial outputs through shared memory.
 constexpr int GA_THREADS = 256, GA_KT = 128, GA_PRE = 4;  // value vectors a thread requests before the scores
+// Eight consecutive values as they are in memory.
 template <typename TA>
 struct Raw8;
 template <>
@@ -68,6 +66,9 @@ struct Raw8<float> {
     }
 };
 
+// Grid: (splits, key/value head x part of its query heads, row); a cluster along x shares the row's keys.  `lpk`
+// lanes share a key in the scores, one thread owns eight value columns of some keys in the weighted sum; GR
+// query heads go together.  The CTAs of a cluster exchange maxima, sums and partial outputs through shared memory.
 template <typename TA, int GR>
 __global__ void __launch_bounds__(GA_THREADS) grouped_rows_kernel(const GroupedArgs a, const TA *__restrict__ q, const TA *__restrict__ k,
                                                                   const TA *__restrict__ v, uint32_t pitch, TA *__restrict__ out, uint32_t out_pitch,
